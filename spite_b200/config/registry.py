@@ -54,7 +54,8 @@ def config_from_dict(d: dict):
 
 
 def load_config(folder):
-    """Read `<folder>/config.json` and return the typed configuration it names."""
+    """Read `<folder>/config.json` and return the typed configuration it names.  A configuration class whose file leaves a
+    size to the shape of a tensor has `with_tensor_shapes({name: shape})`, which is given what the folder holds."""
     path = Path(folder) / "config.json"
     if not path.is_file():
         raise ConfigError(f"{path} not found")
@@ -62,4 +63,9 @@ def load_config(folder):
         d = json.loads(path.read_text())
     except json.JSONDecodeError as e:
         raise ConfigError(f"{path}: not valid JSON ({e})") from None
-    return config_from_dict(d)
+    config = config_from_dict(d)
+    if hasattr(config, "with_tensor_shapes"):
+        # a size that the configuration leaves to a tensor's shape
+        from ..weights.safetensors_io import checkpoint_shapes
+        config = config.with_tensor_shapes(checkpoint_shapes(folder))
+    return config

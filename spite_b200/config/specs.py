@@ -98,6 +98,7 @@ class ModelPlan:
     logit_scale: float = 1.0              # logits are multiplied by this,
     logit_softcap: float | None = None    # then squashed to cap * tanh(logit / cap)
     position_table: int | None = None     # learned position vectors [this many, hidden], added (unscaled) to the embedding
+    streams: int | None = None            # so many residual streams instead of one (arrangements that serve them)
     junctions: tuple[PartSpec, ...] = ()  # parts of the family "junction" that `JunctionCall`s of the order name
 
     def layer_calls(self):
@@ -113,6 +114,11 @@ class ModelPlan:
             raise ConfigError("logit_softcap must be positive")
         if self.position_table is not None and self.position_table < self.max_positions:
             raise ConfigError(f"{self.position_table} learned position vectors cannot serve {self.max_positions} positions")
+        if self.streams is not None:
+            if self.streams < 1 or self.junctions or self.position_table is not None:
+                raise ConfigError("several residual streams: at least one, without junctions and position vectors")
+            if self.final_norm.kind != "rms_norm":
+                raise ConfigError("several residual streams end in an RMS norm of their sum")
         for call in self.order:
             if isinstance(call, JunctionCall) and not 0 <= call.junction < len(self.junctions):
                 raise ConfigError(f"run order names junction {call.junction}, model has {len(self.junctions)}")

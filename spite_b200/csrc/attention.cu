@@ -5,6 +5,8 @@
 //    the rotating part pair up), per-head RMS norm after or before it with or without gains,
 //    the temperature factor of layers without rotation, and the append of k and v to
 //    their pages, in one pass over the projection's output (one warp per head).
+//  * turn_heads: the heads' results on their way to the output projection, turned back by the query's position
+//    where the values were cached rotated by their own, scaled, and laid into columns of a wider row.
 //  * paged_attention: one warp per (token, query head) walks the visible keys in
 //    tiles of 32, keeps a running maximum and sum (all in float32) and gathers the
 //    values.  It serves prompt portions and decoded tokens alike, since every key of
@@ -45,6 +47,10 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkPrepareParams p
     if (p.write_cache && !p.q_only) {
         page = b.block_table[(size_t)b.seg_of_token[t] * b.table_width + pos / c.page_size];
         if (page >= c.n_pages) page = -1;                     // the host never lets this happen
+        // A captured step pads its rows with copies of its first row.  Behind a recurrent layer a copy's row is not the
+        // first row's (the state moved on once, with the first row), so a copy appends nothing: the first row does.
+        if (t > 0 && pos == b.positions[0] && page == b.block_table[(size_t)b.seg_of_token[0] * b.table_width + pos / c.page_size])
+            page = -1;
     }
     // the temperature factor of this position (llama4.rs:177-183)
     float temp = 1.f;
@@ -59,7 +65,9 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkPrepareParams p
     constexpr bool halves = HALVES;
     // cos and sin of a position's angles are the same for every head: the block computes each once (the exact
     // sincosf of an angle of thousands of radians is the most expensive thing here) and its warps read them
-    __shared__ float cs_s[128], sn_s[128];
+    __shared__ float cs_s[128], sn_s[128], vc_s[128], vs_s[128];
+    const int vrot = p.v_inv_freq ? p.v_rotary_dim : 0;
+    for (int i = threadIdx.x; 2 * i < vrot; i += blockDim.x) sincosf((float)pos * p.v_inv_freq[i], &vs_s[i], &vc_s[i]);
     for (int i = threadIdx.x; 2 * i < rot; i += blockDim.x) {
         sincosf((float)pos * p.inv_freq[i], &sn_s[i], &cs_s[i]);
         sn_s[i] *= p.rot_amplitude; cs_s[i] *= p.rot_amplitude;
@@ -99,6 +107,19 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkPrepareParams p
         if (is_v) {
             const T* other = p.v_other ? (const T*)p.v_other + (size_t)t * p.v_other_stride +
                                          (size_t)(head - nq - nkv) * p.v_other_head : nullptr;
+            if (vrot > 0) {
+                const bool vh = p.v_pairing == SPITE_PAIR_HALVES;
+                for (int i = lane; 2 * i < hd; i += 32) {
+                    const bool turns = 2 * i < vrot;
+                    const int f0 = turns && vh ? i : 2 * i, f1 = turns && vh ? i + vrot / 2 : 2 * i + 1;
+                    float a = to_f32(in[f0]), bb = to_f32(in[f1]);
+                    if (bias) { a += bias[f0]; bb += bias[f1]; }
+                    const float cv = turns ? vc_s[i] : 1.f, sv = turns ? vs_s[i] : 0.f;
+                    dst[f0] = from_f32<T>(a * cv - bb * sv);
+                    dst[f1] = from_f32<T>(bb * cv + a * sv);
+                }
+                continue;
+            }
             for (int i = lane; 2 * i < hd; i += 32) {
                 float a, bb;
                 load_pair(in + 2 * i, a, bb);
@@ -159,6 +180,38 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkPrepareParams p
             if (halves) { dst[e0[r]] = from_f32<T>(a); dst[e1[r]] = from_f32<T>(bb); }
             else store_pair(dst + e0[r], a, bb);
         }
+    }
+}
+
+// out[t, h * size + e] = scale * x[t, h, e] for e < size, the pairs of the first `rot` elements turned back by the
+// token's position: the pair (u, v) becomes (u cos a + v sin a, v cos a - u sin a), a = pos * inv_freq[i].  x has rows of
+// heads * head_dim elements, out rows of out_stride.  grid (tokens, head chunks): a block computes the angles once.
+template <typename T>
+__global__ void __launch_bounds__(128) turn_heads_kernel(const T* __restrict__ x, T* __restrict__ out, long long out_stride,
+                                                         const int* __restrict__ positions, const float* __restrict__ inv_freq,
+                                                         int rot, int pairing, int heads, int head_dim, int size, float scale,
+                                                         int heads_per_block) {
+    pdl_wait();
+    pdl_launch_dependents();
+    __shared__ float cs_s[128], sn_s[128];
+    const int t = blockIdx.x;
+    for (int i = threadIdx.x; 2 * i < rot; i += blockDim.x) {
+        sincosf((float)positions[t] * inv_freq[i], &sn_s[i], &cs_s[i]);
+    }
+    __syncthreads();
+    const int h0 = blockIdx.y * heads_per_block, h1 = min(heads, h0 + heads_per_block);
+    const bool halves = pairing == SPITE_PAIR_HALVES;
+    const int pairs = (size + 1) / 2;
+    for (int e = threadIdx.x; e < (h1 - h0) * pairs; e += blockDim.x) {
+        const int h = h0 + e / pairs, i = e % pairs;
+        const T* in = x + ((size_t)t * heads + h) * head_dim;
+        T* o = out + (size_t)t * out_stride + (size_t)h * size;
+        const bool turns = 2 * i < rot;
+        const int e0 = turns && halves ? i : 2 * i, e1 = turns && halves ? i + rot / 2 : 2 * i + 1;
+        const float u = to_f32(in[e0]), v = e1 < size ? to_f32(in[e1]) : 0.f;
+        const float c = turns ? cs_s[i] : 1.f, s = turns ? sn_s[i] : 0.f;
+        o[e0] = from_f32<T>((u * c + v * s) * scale);
+        if (e1 < size) o[e1] = from_f32<T>((v * c - u * s) * scale);
     }
 }
 
@@ -272,6 +325,8 @@ SPITE_API int spite_qk_prepare(int dtype, const QkPrepareParams* given, const St
     if (p->q_only && (p->v_other || p->gates_out)) return SPITE_BAD_ARG;
     if (p->qkv_stride < (long long)heads * c->head_dim || (p->qkv_stride & 1)) return SPITE_BAD_ARG;
     if (p->gates_out && p->qkv_stride < (long long)heads * c->head_dim + p->num_heads) return SPITE_BAD_ARG;
+    if (p->v_inv_freq && (p->v_other || p->q_only || p->v_rotary_dim < 2 || p->v_rotary_dim % 2 || p->v_rotary_dim > c->head_dim ||
+                          (p->v_pairing != SPITE_PAIR_NEIGHBOURS && p->v_pairing != SPITE_PAIR_HALVES))) return SPITE_BAD_ARG;
     if (p->v_other && (p->v_mix_dim < 0 || p->v_mix_dim > c->head_dim || p->v_other_head < p->v_mix_dim)) return SPITE_BAD_ARG;
     // few tokens: four heads a block, so that the step still fills the device; many: a block per token
     const bool many = b->n_tokens >= 1024;
@@ -290,6 +345,30 @@ SPITE_API int spite_qk_prepare(int dtype, const QkPrepareParams* given, const St
         if (halves) SPITE_LAUNCH((qk_prepare_kernel<__nv_bfloat16, true>), grid, threads, 0, st, *p, *b, *c, heads_per_block);
         else SPITE_LAUNCH((qk_prepare_kernel<__nv_bfloat16, false>), grid, threads, 0, st, *p, *b, *c, heads_per_block);
     }
+    return spite_launch_status();
+}
+
+SPITE_API int spite_turn_heads(int dtype, const void* x, void* out, long long out_stride, const int* positions,
+                               const float* inv_freq, int rotary_dim, int pairing, int n_tokens, int heads, int head_dim,
+                               int size, float scale, void* stream) {
+    if (!x || !out || n_tokens < 0 || heads < 1 || size < 1 || head_dim < size || !(scale == scale)) return SPITE_BAD_ARG;
+    if (out_stride < (long long)heads * size) return SPITE_BAD_ARG;
+    if (inv_freq && (!positions || rotary_dim < 2 || rotary_dim % 2 || rotary_dim > size)) return SPITE_BAD_ARG;
+    if (pairing != SPITE_PAIR_NEIGHBOURS && pairing != SPITE_PAIR_HALVES) return SPITE_BAD_ARG;
+    if (dtype != SPITE_DT_F32 && dtype != SPITE_DT_BF16) return SPITE_BAD_ARG;
+    if (inv_freq && rotary_dim > 256) return SPITE_UNSUPPORTED;
+    if (n_tokens == 0) return SPITE_OK;
+    const int hpb = n_tokens >= 1024 ? 32 : 4;                // few tokens: more blocks
+    dim3 grid(n_tokens, (heads + hpb - 1) / hpb);
+    if (grid.y > 65535) return SPITE_UNSUPPORTED;
+    const int rot = inv_freq ? rotary_dim : 0;
+    cudaStream_t st = (cudaStream_t)stream;
+    if (dtype == SPITE_DT_F32)
+        SPITE_LAUNCH(turn_heads_kernel<float>, grid, 128, 0, st, (const float*)x, (float*)out, out_stride, positions, inv_freq, rot,
+                     pairing, heads, head_dim, size, scale, hpb);
+    else
+        SPITE_LAUNCH(turn_heads_kernel<__nv_bfloat16>, grid, 128, 0, st, (const __nv_bfloat16*)x, (__nv_bfloat16*)out, out_stride,
+                     positions, inv_freq, rot, pairing, heads, head_dim, size, scale, hpb);
     return spite_launch_status();
 }
 

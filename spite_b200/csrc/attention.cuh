@@ -63,6 +63,11 @@ struct QkPrepareParams {
     int q_only;                 // the rows of qkv hold the q heads alone: this layer reads keys and values that another layer cached
     int norm_dim;               // > 0: a q or k head has this many elements (the rest of its head_dim are padding zeros): the
                                 // per-head norm's mean is taken over them (0: over head_dim)
+    // rotated values: element i < v_rotary_dim / 2 of a value head pairs with its partner by v_pairing (SPITE_PAIR_*) and the
+    // pair turns by position * v_inv_freq[i] before it is cached (null: values are cached as they are)
+    const float* v_inv_freq;
+    int v_rotary_dim;
+    int v_pairing;
 };
 
 struct AttentionParams {

@@ -6,12 +6,12 @@
 // h[m, :] = table[token[m], :] * scale    (crates/spite-models/src/llama/llama4.rs:118-119; scale 1 there)
 template <typename T>
 __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict__ tokens,
-                             float* __restrict__ h, int d, int vocab, float scale) {
+                             float* __restrict__ h, int d, int vocab, float scale, int copies) {
     pdl_wait();
     pdl_launch_dependents();
-    const int m = blockIdx.x;
+    const int m = blockIdx.x / copies;                      // (a model with several residual streams starts them alike)
     const int tok = tokens[m];
-    float* out = h + (size_t)m * d;
+    float* out = h + (size_t)blockIdx.x * d;
     if (tok < 0 || tok >= vocab) {          // the host rejects such ids before the launch
         for (int i = threadIdx.x; i < d; i += blockDim.x) out[i] = 0.f;
         return;
@@ -244,15 +244,16 @@ SPITE_API int spite_transform_logits(float* logits, long long n, float scale, fl
 }
 
 SPITE_API int spite_embed(int dtype, const void* table, const int* tokens, float* h,
-                          int n_tokens, int d, int vocab, float scale, void* stream) {
-    if (!table || !tokens || !h || n_tokens < 0 || d <= 0 || vocab <= 0 || !(scale == scale)) return SPITE_BAD_ARG;
+                          int n_tokens, int d, int vocab, float scale, int copies, void* stream) {
+    if (!table || !tokens || !h || n_tokens < 0 || d <= 0 || vocab <= 0 || copies < 1 || !(scale == scale)) return SPITE_BAD_ARG;
+    if ((long long)n_tokens * copies > 0x7fffffffLL) return SPITE_UNSUPPORTED;
     if (n_tokens == 0) return SPITE_OK;
     cudaStream_t st = (cudaStream_t)stream;
     const int threads = d >= 1024 ? 256 : 128;
     if (dtype == SPITE_DT_F32)
-        SPITE_LAUNCH(embed_kernel<float>, n_tokens, threads, 0, st, (const float*)table, tokens, h, d, vocab, scale);
+        SPITE_LAUNCH(embed_kernel<float>, n_tokens * copies, threads, 0, st, (const float*)table, tokens, h, d, vocab, scale, copies);
     else if (dtype == SPITE_DT_BF16)
-        SPITE_LAUNCH(embed_kernel<__nv_bfloat16>, n_tokens, threads, 0, st, (const __nv_bfloat16*)table, tokens, h, d, vocab, scale);
+        SPITE_LAUNCH(embed_kernel<__nv_bfloat16>, n_tokens * copies, threads, 0, st, (const __nv_bfloat16*)table, tokens, h, d, vocab, scale, copies);
     else
         return SPITE_BAD_ARG;
     return spite_launch_status();
@@ -495,8 +496,8 @@ SPITE_API int spite_fill_rows(float* out, const float* vec, int n_rows, int d, i
 template <typename TX, typename TO>
 __global__ void __launch_bounds__(128) head_norm_gate_kernel(const TX* __restrict__ x, const TX* __restrict__ gates,
                                                              long long gate_stride, const float* __restrict__ gain,
-                                                             TO* __restrict__ out, int n_tokens, int heads, int size, float eps,
-                                                             int gate_silu, int gain_per_head) {
+                                                             TO* __restrict__ out, long long out_stride, int n_tokens, int heads,
+                                                             int size, float eps, int gate_silu, int gain_per_head) {
     pdl_wait();
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31;
@@ -515,7 +516,7 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const TX* __restric
     }
     const TX* g = gates ? gates + (size_t)m * gate_stride + (size_t)h * size : nullptr;
     const float* w = gain ? gain + (gain_per_head ? (size_t)h * size : 0) : nullptr;
-    TO* o = out + base;
+    TO* o = out + (size_t)m * out_stride + (size_t)h * size;
     for (int j = lane; j < size; j += 32) {
         float v = to_f32(in[j]) * mul;
         if (w) v *= w[j];
@@ -530,10 +531,10 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const TX* __restric
 // x_dtype: type of x and gates; out_dtype: type of out (x may be the float32 result of a recurrence while out feeds a
 // bfloat16 product); out may be x.
 SPITE_API int spite_head_norm_gate(int x_dtype, int out_dtype, const void* x, const void* gates, long long gate_stride,
-                                   const float* gain, void* out, int n_tokens, int heads, int size, float eps, int gate_silu,
-                                   int gain_per_head, void* stream) {
+                                   const float* gain, void* out, long long out_stride, int n_tokens, int heads, int size,
+                                   float eps, int gate_silu, int gain_per_head, void* stream) {
     if (!x || !out || n_tokens < 0 || heads < 1 || size < 1 || !(eps == eps) || eps < 0.f) return SPITE_BAD_ARG;
-    if (gates && gate_stride < (long long)heads * size) return SPITE_BAD_ARG;
+    if ((gates && gate_stride < (long long)heads * size) || out_stride < (long long)heads * size) return SPITE_BAD_ARG;
     if (x_dtype != SPITE_DT_F32 && x_dtype != SPITE_DT_BF16) return SPITE_BAD_ARG;
     if (out_dtype != SPITE_DT_F32 && out_dtype != SPITE_DT_BF16) return SPITE_BAD_ARG;
     if (x_dtype == SPITE_DT_BF16 && out_dtype == SPITE_DT_F32) return SPITE_UNSUPPORTED;
@@ -544,13 +545,13 @@ SPITE_API int spite_head_norm_gate(int x_dtype, int out_dtype, const void* x, co
     cudaStream_t st = (cudaStream_t)stream;
     if (x_dtype == SPITE_DT_F32 && out_dtype == SPITE_DT_F32)
         SPITE_LAUNCH((head_norm_gate_kernel<float, float>), (int)blocks, 128, 0, st, (const float*)x, (const float*)gates,
-                     gate_stride, gain, (float*)out, n_tokens, heads, size, eps, gate_silu, gain_per_head);
+                     gate_stride, gain, (float*)out, out_stride, n_tokens, heads, size, eps, gate_silu, gain_per_head);
     else if (x_dtype == SPITE_DT_F32)
         SPITE_LAUNCH((head_norm_gate_kernel<float, __nv_bfloat16>), (int)blocks, 128, 0, st, (const float*)x, (const float*)gates,
-                     gate_stride, gain, (__nv_bfloat16*)out, n_tokens, heads, size, eps, gate_silu, gain_per_head);
+                     gate_stride, gain, (__nv_bfloat16*)out, out_stride, n_tokens, heads, size, eps, gate_silu, gain_per_head);
     else
         SPITE_LAUNCH((head_norm_gate_kernel<__nv_bfloat16, __nv_bfloat16>), (int)blocks, 128, 0, st, (const __nv_bfloat16*)x,
-                     (const __nv_bfloat16*)gates, gate_stride, gain, (__nv_bfloat16*)out, n_tokens, heads, size, eps, gate_silu, gain_per_head);
+                     (const __nv_bfloat16*)gates, gate_stride, gain, (__nv_bfloat16*)out, out_stride, n_tokens, heads, size, eps, gate_silu, gain_per_head);
     return spite_launch_status();
 }
 
@@ -603,6 +604,7 @@ struct ShortConvParams {
     int n_segments, channels, taps, copy_columns;
     int activation;             // 0: none, 1: silu
     int max_seg_len;
+    const float* bias;          // [channels] added to a channel's sum before the activation, or null
 };
 
 constexpr int CONV_TB = 16;
@@ -634,6 +636,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
     } else {
         const int taps = p.taps;
         float w[CONV_MAX_TAPS], win[CONV_MAX_TAPS - 1], old[CONV_MAX_TAPS - 1];
+        const float bias = p.bias ? p.bias[c] : 0.f;
 #pragma unroll
         for (int j = 0; j < CONV_MAX_TAPS; ++j)               // the taps right-aligned: w[CONV_MAX_TAPS - 1] is the current token's
             w[j] = j >= CONV_MAX_TAPS - taps ? p.w[(size_t)c * taps + j - (CONV_MAX_TAPS - taps)] : 0.f;
@@ -659,7 +662,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
             float acc = 0.f;
 #pragma unroll
             for (int j = 0; j < CONV_MAX_TAPS - 1; ++j) acc = fmaf(w[j], win[j], acc);
-            acc = fmaf(w[CONV_MAX_TAPS - 1], cur, acc);
+            acc = fmaf(w[CONV_MAX_TAPS - 1], cur, acc) + bias;
             if (p.activation == 1) acc = acc / (1.0f + expf(-acc));
             y[i - i0] = acc;
             out[(size_t)(t0 + i) * p.out_stride + c] = from_f32<T>(acc);
@@ -706,4 +709,333 @@ SPITE_API int spite_short_conv(int out_dtype, const ShortConvParams* p, void* st
     if (out_dtype == SPITE_DT_F32) SPITE_LAUNCH(short_conv_kernel<float>, grid, 128, 0, (cudaStream_t)stream, *p);
     else SPITE_LAUNCH(short_conv_kernel<__nv_bfloat16>, grid, 128, 0, (cudaStream_t)stream, *p);
     return spite_launch_status();
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Token shift: what a mixer reads that blends every token with the one before it, in `n_mixes` ways at once:
+//     out[g, m, :] = x[m, :] + (x'[m, :] - x[m, :]) * mu[g, :]
+// x' is the row before (for a segment's first token the row in the request's slot, all zeros at the start of a
+// sequence); the slot then receives the segment's last row.  Also lists where every mix's rows start in the order
+// [mix, token] (offsets_out[g] = g * tokens, for a product of one group per mix).
+struct TokenShiftParams {
+    const void* x;              // [tokens, d] (T)
+    const float* mu;            // [n_mixes, d]
+    void* out;                  // [n_mixes, tokens, d] (T)
+    float* state;               // state + slot * slot_stride: [d]
+    long long slot_stride;
+    const int* seg_of_token;    // [tokens]
+    const int* cu_seqlens;      // [segments + 1]
+    const int* slots;           // [segments]
+    int* offsets_out;           // [n_mixes + 1] or null
+    int n_tokens, d, n_mixes;
+};
+
+constexpr int SHIFT_MAX_MIXES = 8;
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) token_shift_kernel(const TokenShiftParams p) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t = blockIdx.x, d = p.d;
+    if (p.offsets_out && t == 0 && blockIdx.y == 0 && (int)threadIdx.x <= p.n_mixes) p.offsets_out[threadIdx.x] = threadIdx.x * p.n_tokens;
+    const int s = p.seg_of_token[t], t0 = p.cu_seqlens[s], t1 = p.cu_seqlens[s + 1];
+    const int slot = p.slots[s];
+    // a captured step's padding row (a copy of the first row) leaves the slot alone; its results are never read
+    const bool copy = s > 0 && slot == p.slots[0];
+    float* st = p.state + (size_t)slot * p.slot_stride;
+    const T* cur = (const T*)p.x + (size_t)t * d;
+    const T* last = (const T*)p.x + (size_t)(t1 - 1) * d;
+    T* out = (T*)p.out + (size_t)t * d;
+    const size_t plane = (size_t)p.n_tokens * d;
+    constexpr int W = VEC ? 4 : 1;
+    for (int c = W * (blockIdx.y * blockDim.x + threadIdx.x); c < d; c += W * gridDim.y * blockDim.x) {
+        float x[W], b[W];
+        if constexpr (VEC) { const float4 v = load4(cur + c); x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w; }
+        else x[0] = to_f32(cur[c]);
+        if (t > t0) {
+            if constexpr (VEC) { const float4 v = load4(cur - d + c); b[0] = v.x; b[1] = v.y; b[2] = v.z; b[3] = v.w; }
+            else b[0] = to_f32(cur[c - d]);
+        } else {
+            // the thread that reads an element of the slot is the one that renews it
+#pragma unroll
+            for (int i = 0; i < W; ++i) {
+                b[i] = copy ? 0.f : st[c + i];
+                if (!copy) st[c + i] = to_f32(last[c + i]);
+            }
+        }
+#pragma unroll 1
+        for (int g = 0; g < p.n_mixes; ++g) {
+            const float* mu = p.mu + (size_t)g * d + c;
+            T* o = out + (size_t)g * plane + c;
+            if constexpr (VEC) {
+                const float4 m = *(const float4*)mu;
+                store4(o, fmaf(b[0] - x[0], m.x, x[0]), fmaf(b[1] - x[1], m.y, x[1]), fmaf(b[2] - x[2], m.z, x[2]),
+                       fmaf(b[3] - x[3], m.w, x[3]));
+            } else {
+                o[0] = from_f32<T>(fmaf(b[0] - x[0], mu[0], x[0]));
+            }
+        }
+    }
+}
+
+SPITE_API int spite_token_shift(int dtype, const TokenShiftParams* p, void* stream) {
+    if (!p || !p->x || !p->mu || !p->out || !p->state || !p->seg_of_token || !p->cu_seqlens || !p->slots) return SPITE_BAD_ARG;
+    if (p->n_tokens < 0 || p->d < 1 || p->n_mixes < 1 || p->slot_stride < p->d) return SPITE_BAD_ARG;
+    if (dtype != SPITE_DT_F32 && dtype != SPITE_DT_BF16) return SPITE_BAD_ARG;
+    if (p->n_mixes > SHIFT_MAX_MIXES) return SPITE_UNSUPPORTED;
+    if (p->n_tokens == 0) return SPITE_OK;
+    const bool vec = p->d % 4 == 0 && ((((uintptr_t)p->x | (uintptr_t)p->mu | (uintptr_t)p->out) & 15) == 0);
+    const int per = vec ? 4 : 1;
+    const int threads = (p->d + per - 1) / per >= 256 ? 256 : 128;
+    dim3 grid(p->n_tokens, p->n_tokens < 64 ? (p->d + per * threads - 1) / (per * threads) : 1);
+    cudaStream_t st = (cudaStream_t)stream;
+    if (dtype == SPITE_DT_F32) {
+        if (vec) SPITE_LAUNCH((token_shift_kernel<float, true>), grid, threads, 0, st, *p);
+        else SPITE_LAUNCH((token_shift_kernel<float, false>), grid, threads, 0, st, *p);
+    } else {
+        if (vec) SPITE_LAUNCH((token_shift_kernel<__nv_bfloat16, true>), grid, threads, 0, st, *p);
+        else SPITE_LAUNCH((token_shift_kernel<__nv_bfloat16, false>), grid, threads, 0, st, *p);
+    }
+    return spite_launch_status();
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// A recurrence's output gated first and normed after, in equal parts:
+//     v = x[m, :] * silu(z[m, :]);   out[m, e] = v[e] / sqrt(mean of v^2 over e's part + eps) * gain[e]
+// x float32 [tokens, groups * size], z float32 with rows of z_stride.  A block serves one (token, part); a part's values
+// stay in shared memory between the sum and the scaling.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) gate_group_norm_kernel(const float* __restrict__ x, const float* __restrict__ z,
+                                                              long long z_stride, const float* __restrict__ gain,
+                                                              T* __restrict__ out, int groups, int size, float eps) {
+    extern __shared__ __align__(16) float part[];
+    __shared__ float scratch[33];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int m = blockIdx.x, g = blockIdx.y;
+    const float* xr = x + ((size_t)m * groups + g) * size;
+    const float* zr = z + (size_t)m * z_stride + (size_t)g * size;
+    const float* w = gain + (size_t)g * size;
+    T* o = out + ((size_t)m * groups + g) * size;
+    constexpr int W = VEC ? 4 : 1;
+    float s = 0.f;
+    for (int c = W * threadIdx.x; c < size; c += W * blockDim.x) {
+        if constexpr (VEC) {
+            const float4 a = *(const float4*)(xr + c), b = *(const float4*)(zr + c);
+            float4 v;
+            v.x = a.x * (b.x / (1.0f + expf(-b.x))); v.y = a.y * (b.y / (1.0f + expf(-b.y)));
+            v.z = a.z * (b.z / (1.0f + expf(-b.z))); v.w = a.w * (b.w / (1.0f + expf(-b.w)));
+            *(float4*)(part + c) = v;
+            s += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+        } else {
+            const float v = xr[c] * (zr[c] / (1.0f + expf(-zr[c])));
+            part[c] = v;
+            s += v * v;
+        }
+    }
+    s = block_sum(s, scratch);
+    const float mul = 1.0f / sqrtf(s / (float)size + eps);
+    for (int c = W * threadIdx.x; c < size; c += W * blockDim.x) {      // (a thread reads what it wrote)
+        if constexpr (VEC) {
+            const float4 v = *(const float4*)(part + c), b = *(const float4*)(w + c);
+            store4(o + c, v.x * mul * b.x, v.y * mul * b.y, v.z * mul * b.z, v.w * mul * b.w);
+        } else {
+            o[c] = from_f32<T>(part[c] * mul * w[c]);
+        }
+    }
+}
+
+template <typename K>
+static int raise_smem_limit(K kernel, size_t bytes) {
+    if (bytes <= 48 * 1024) return SPITE_OK;
+    return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) == cudaSuccess ? SPITE_OK
+                                                                                                             : SPITE_LAUNCH_FAILED;
+}
+
+SPITE_API int spite_gate_group_norm(int out_dtype, const float* x, const float* z, long long z_stride, const float* gain, void* out,
+                                    int n_tokens, int groups, int size, float eps, void* stream) {
+    if (!x || !z || !gain || !out || n_tokens < 0 || groups < 1 || size < 1 || !(eps > 0.f)) return SPITE_BAD_ARG;
+    if (z_stride < (long long)groups * size) return SPITE_BAD_ARG;
+    if (out_dtype != SPITE_DT_F32 && out_dtype != SPITE_DT_BF16) return SPITE_BAD_ARG;
+    const size_t bytes = (size_t)size * sizeof(float);
+    if (groups > 65535 || bytes > 200 * 1024) return SPITE_UNSUPPORTED;
+    if (n_tokens == 0) return SPITE_OK;
+    const bool vec = size % 4 == 0 && z_stride % 4 == 0 && ((((uintptr_t)x | (uintptr_t)z | (uintptr_t)gain | (uintptr_t)out) & 15) == 0);
+    const int work = vec ? size / 4 : size;
+    const int threads = work <= 32 ? 32 : work <= 64 ? 64 : work <= 128 ? 128 : 256;
+    dim3 grid(n_tokens, groups);
+    cudaStream_t st = (cudaStream_t)stream;
+#define SPITE_GGN(T, V)                                                                                                     \
+    if (raise_smem_limit(gate_group_norm_kernel<T, V>, bytes) != SPITE_OK) return SPITE_LAUNCH_FAILED;                      \
+    SPITE_LAUNCH((gate_group_norm_kernel<T, V>), grid, threads, bytes, st, x, z, z_stride, gain, (T*)out, groups, size, eps)
+    if (out_dtype == SPITE_DT_F32) { if (vec) { SPITE_GGN(float, true); } else { SPITE_GGN(float, false); } }
+    else { if (vec) { SPITE_GGN(__nv_bfloat16, true); } else { SPITE_GGN(__nv_bfloat16, false); } }
+#undef SPITE_GGN
+    return spite_launch_status();
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Several residual streams (hyper-connections).  x float32 [tokens, S, d].  One kernel does everything that happens between
+// two sublayers:
+//   with y:      v = (y[m, :] + bias) * scale;   x_t <- sum_s mix[s, t] x_s + w_out[t] v        (all from the old streams)
+//   with w_in:   u = sum_s w_in[s] x_s;   next_out[i, :] = u / sqrt(mean(u^2) + eps) * gain   (without a gain: u itself)
+// `rows` (with next_out): only these tokens are served, next_out's row i is token rows[i].  `write_back` 0: the renewed
+// streams are used for u and not stored (the last read of a step).  A block serves one token, a thread the same columns of
+// all streams; u stays in shared memory between the sum and the scaling.
+struct StreamsParams {
+    float* x;
+    const float* y;             // [tokens, d] or null
+    const float* bias;          // [d] or null
+    const float* scale;         // [d] or null
+    const float* mix;           // [S, S], [from, to] (with y)
+    const float* w_out;         // [S] (with y)
+    const float* w_in;          // [S] (with next_out)
+    const float* gain;          // [d] or null
+    void* next_out;             // [rows, d] (T or float32) or null
+    const int* rows;            // or null
+    int n_rows, d, streams, write_back;
+    float eps;
+};
+
+constexpr int MAX_STREAMS = 32;
+
+template <typename T, int S, bool VEC>                     // S 0: the number of streams is known at run time only
+__global__ void __launch_bounds__(256) streams_kernel(const StreamsParams p) {
+    extern __shared__ __align__(16) float u_s[];
+    __shared__ float scratch[33];
+    __shared__ float coef[MAX_STREAMS * MAX_STREAMS + 2 * MAX_STREAMS];
+    const int n = S ? S : p.streams, d = p.d;
+    // (weights only: nothing an earlier kernel of the step writes)
+    if (p.y) {
+        for (int i = threadIdx.x; i < n * n; i += blockDim.x) coef[i] = p.mix[i];
+        for (int i = threadIdx.x; i < n; i += blockDim.x) coef[n * n + i] = p.w_out[i];
+    }
+    if (p.next_out) for (int i = threadIdx.x; i < n; i += blockDim.x) coef[n * n + n + i] = p.w_in[i];
+    pdl_wait();
+    pdl_launch_dependents();
+    __syncthreads();
+    const int m = p.rows ? p.rows[blockIdx.x] : blockIdx.x;
+    float* xr = p.x + (size_t)m * n * d;
+    const float* yr = p.y ? p.y + (size_t)m * d : nullptr;
+    const float* mix = coef;
+    const float* w_out = coef + n * n;
+    const float* w_in = coef + n * n + n;
+    constexpr int W = VEC ? 4 : 1;
+    constexpr int R = S ? S : MAX_STREAMS, UN = S ? S : 1;
+    float sum = 0.f;
+    for (int c = W * threadIdx.x; c < d; c += W * blockDim.x) {
+        float old[R][W], v[W], u[W];
+#pragma unroll UN
+        for (int s = 0; s < R; ++s) {
+            if (s >= n) break;
+            if constexpr (VEC) { const float4 f = *(const float4*)(xr + (size_t)s * d + c); old[s][0] = f.x; old[s][1] = f.y; old[s][2] = f.z; old[s][3] = f.w; }
+            else old[s][0] = xr[(size_t)s * d + c];
+        }
+#pragma unroll
+        for (int i = 0; i < W; ++i) u[i] = 0.f;
+        if (yr) {
+            if constexpr (VEC) { const float4 f = *(const float4*)(yr + c); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+            else v[0] = yr[c];
+#pragma unroll
+            for (int i = 0; i < W; ++i) {
+                if (p.bias) v[i] += p.bias[c + i];
+                if (p.scale) v[i] *= p.scale[c + i];
+            }
+#pragma unroll UN
+            for (int t = 0; t < R; ++t) {
+                if (t >= n) break;
+                float a[W];
+#pragma unroll
+                for (int i = 0; i < W; ++i) a[i] = w_out[t] * v[i];
+#pragma unroll UN
+                for (int s = 0; s < R; ++s) {
+                    if (s >= n) break;
+                    const float f = mix[s * n + t];
+#pragma unroll
+                    for (int i = 0; i < W; ++i) a[i] = fmaf(f, old[s][i], a[i]);
+                }
+                if (p.write_back) {
+                    if constexpr (VEC) *(float4*)(xr + (size_t)t * d + c) = make_float4(a[0], a[1], a[2], a[3]);
+                    else xr[(size_t)t * d + c] = a[0];
+                }
+                if (p.next_out) {
+#pragma unroll
+                    for (int i = 0; i < W; ++i) u[i] = fmaf(w_in[t], a[i], u[i]);
+                }
+            }
+        } else {
+#pragma unroll UN
+            for (int s = 0; s < R; ++s) {
+                if (s >= n) break;
+#pragma unroll
+                for (int i = 0; i < W; ++i) u[i] = fmaf(w_in[s], old[s][i], u[i]);
+            }
+        }
+        if (!p.next_out) continue;
+        if constexpr (VEC) *(float4*)(u_s + c) = make_float4(u[0], u[1], u[2], u[3]);
+        else u_s[c] = u[0];
+#pragma unroll
+        for (int i = 0; i < W; ++i) sum = fmaf(u[i], u[i], sum);
+    }
+    if (!p.next_out) return;
+    float mul = 1.f;
+    if (p.gain) {
+        sum = block_sum(sum, scratch);
+        mul = 1.0f / sqrtf(sum / (float)d + p.eps);
+    }
+    T* o = (T*)p.next_out + (size_t)blockIdx.x * d;
+    for (int c = W * threadIdx.x; c < d; c += W * blockDim.x) {         // (a thread reads what it wrote)
+        if constexpr (VEC) {
+            float4 f = *(const float4*)(u_s + c);
+            if (p.gain) {
+                const float4 g = *(const float4*)(p.gain + c);
+                f = make_float4(f.x * mul * g.x, f.y * mul * g.y, f.z * mul * g.z, f.w * mul * g.w);
+            }
+            store4(o + c, f.x, f.y, f.z, f.w);
+        } else {
+            o[c] = from_f32<T>(p.gain ? u_s[c] * mul * p.gain[c] : u_s[c]);
+        }
+    }
+}
+
+template <typename T, int S>
+static int launch_streams(const StreamsParams& p, bool vec, cudaStream_t st) {
+    const size_t bytes = p.next_out ? (size_t)p.d * sizeof(float) : 0;
+    const int work = vec ? p.d / 4 : p.d;
+    const int threads = work <= 32 ? 32 : work <= 64 ? 64 : work <= 128 ? 128 : 256;
+    if constexpr (S > 0) {
+        if (vec) {
+            if (raise_smem_limit(streams_kernel<T, S, true>, bytes) != SPITE_OK) return SPITE_LAUNCH_FAILED;
+            SPITE_LAUNCH((streams_kernel<T, S, true>), p.n_rows, threads, bytes, st, p);
+            return spite_launch_status();
+        }
+    }
+    if (raise_smem_limit(streams_kernel<T, S, false>, bytes) != SPITE_OK) return SPITE_LAUNCH_FAILED;
+    SPITE_LAUNCH((streams_kernel<T, S, false>), p.n_rows, threads, bytes, st, p);
+    return spite_launch_status();
+}
+
+SPITE_API int spite_streams(int out_dtype, const StreamsParams* p, void* stream) {
+    if (!p || !p->x || p->n_rows < 0 || p->d < 1 || p->streams < 1) return SPITE_BAD_ARG;
+    if (!p->y && !p->next_out) return SPITE_BAD_ARG;
+    if (p->y && (!p->mix || !p->w_out)) return SPITE_BAD_ARG;
+    if (p->next_out && !p->w_in) return SPITE_BAD_ARG;
+    if (p->gain && !(p->eps > 0.f)) return SPITE_BAD_ARG;
+    if (p->rows && (!p->next_out || (p->y && p->write_back))) return SPITE_BAD_ARG;     // (a row may be named twice)
+    if (out_dtype != SPITE_DT_F32 && out_dtype != SPITE_DT_BF16) return SPITE_BAD_ARG;
+    if (p->streams > MAX_STREAMS || (size_t)p->d * sizeof(float) > 200 * 1024) return SPITE_UNSUPPORTED;
+    if (p->n_rows == 0) return SPITE_OK;
+    const bool vec = p->d % 4 == 0 && ((((uintptr_t)p->x | (uintptr_t)p->y | (uintptr_t)p->gain | (uintptr_t)p->next_out) & 15) == 0);
+    cudaStream_t st = (cudaStream_t)stream;
+#define SPITE_STREAMS_T(T)                                        \
+    switch (p->streams) {                                         \
+        case 1: return launch_streams<T, 1>(*p, vec, st);         \
+        case 2: return launch_streams<T, 2>(*p, vec, st);         \
+        case 3: return launch_streams<T, 3>(*p, vec, st);         \
+        case 4: return launch_streams<T, 4>(*p, vec, st);         \
+        default: return launch_streams<T, 0>(*p, false, st);      \
+    }
+    if (out_dtype == SPITE_DT_F32) { SPITE_STREAMS_T(float) }
+    SPITE_STREAMS_T(__nv_bfloat16)
+#undef SPITE_STREAMS_T
 }

@@ -30,23 +30,38 @@ struct GemmParams {
     int n_groups, M, N, K;
     int epilogue;
     int scale_by_a_row;
-    int activation;       // SPITE_ACT_*: applied by EPI_STORE to the scaled sum before it is rounded
+    int activation;       // SPITE_ACT_*: applied by EPI_STORE to the scaled sum (plus bias) before it is rounded
+    const float* bias;    // [N] or null: added by EPI_STORE to the scaled sum before the activation (one group)
+    float act_pos, act_neg;   // SPITE_ACT_XIELU: the coefficients of its two branches
 };
 
 #define SPITE_ACT_NONE 0
 #define SPITE_ACT_RELU2 1        // relu(y)^2
 #define SPITE_ACT_GELU_TANH 2    // 0.5 y (1 + tanh(sqrt(2/pi) (y + 0.044715 y^3)))
+#define SPITE_ACT_XIELU 3        // y > 0: act_pos y^2 + y / 2; else act_neg (e^y - 1 - y) + y / 2
+#define SPITE_ACT_TANH 4
 
-__device__ __forceinline__ float apply_activation(int act, float y) {
+__device__ __forceinline__ float apply_activation(const GemmParams& p, float y) {
+    const int act = p.activation;
     if (act == SPITE_ACT_RELU2) { y = fmaxf(y, 0.f); y *= y; }
     else if (act == SPITE_ACT_GELU_TANH) y = 0.5f * y * (1.0f + tanhf(0.7978845608028654f * (y + 0.044715f * y * y * y)));
+    else if (act == SPITE_ACT_XIELU) {
+        const float n = fminf(y, 0.f);                       // (no branch per element)
+        const float pos = fmaxf(y, 0.f);
+        y = fmaf(p.act_pos * pos, pos, fmaf(p.act_neg, expm1f(n) - n, 0.5f * y));
+    } else if (act == SPITE_ACT_TANH) y = tanhf(y);
     return y;
 }
+// The same for output column n: the bias first.
+__device__ __forceinline__ float finish_store(const GemmParams& p, float y, int n) {
+    return apply_activation(p, p.bias ? y + p.bias[n] : y);
+}
 
-// An activation goes with the plain store only.
+// An activation goes with the plain store only, a bias with the plain store of a product of one group.
 static inline bool activation_ok(const GemmParams* p) {
-    return p->activation == SPITE_ACT_NONE ||
-           ((p->activation == SPITE_ACT_RELU2 || p->activation == SPITE_ACT_GELU_TANH) && p->epilogue == EPI_STORE);
+    if (p->activation < SPITE_ACT_NONE || p->activation > SPITE_ACT_TANH) return false;
+    if (p->bias && (p->epilogue != EPI_STORE || p->group_offsets)) return false;
+    return p->activation == SPITE_ACT_NONE || p->epilogue == EPI_STORE;
 }
 
 __device__ __forceinline__ float silu_f32(float g) { return g / (1.0f + expf(-g)); }

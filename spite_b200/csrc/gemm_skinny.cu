@@ -253,7 +253,7 @@ __global__ void __launch_bounds__(WARPS * 32, (NT <= 1 ? 2 : 1)) gemm_skinny_ker
             const int crow = p.c_rows ? p.c_rows[li] : li;
             const float sc = p.row_scale ? p.row_scale[p.scale_by_a_row ? arow : li] : 1.f;
             const size_t o = (size_t)crow * p.ldc + n;
-            if (EPI == EPI_STORE) ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(apply_activation(p.activation, v * sc));
+            if (EPI == EPI_STORE) ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(finish_store(p, v * sc, n));
             else if (EPI == EPI_STORE_F32) ((float*)p.C)[o] = v * sc;
             else if (EPI == EPI_ADD_F32) ((float*)p.C)[o] += v * sc;
             else ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(silu_f32(v * sc) * (v2 * sc));

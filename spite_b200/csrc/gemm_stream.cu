@@ -350,7 +350,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const GemmParams p
                 const int crow = p.c_rows ? p.c_rows[li] : li;
                 const float sc = p.row_scale ? p.row_scale[p.scale_by_a_row ? ar : li] : 1.f;
                 const size_t o = (size_t)crow * p.ldc + n;
-                if (EPI == EPI_STORE) ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(apply_activation(p.activation, v * sc));
+                if (EPI == EPI_STORE) ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(finish_store(p, v * sc, n));
                 else if (EPI == EPI_STORE_F32) ((float*)p.C)[o] = v * sc;
                 else if (EPI == EPI_ADD_F32) ((float*)p.C)[o] += v * sc;
                 else ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(silu_f32(v * sc) * (v2 * sc));

@@ -37,7 +37,17 @@ __device__ __forceinline__ void drain_accumulator_row(const GemmParams& p, int l
             __nv_bfloat16* dst = (__nv_bfloat16*)p.C + o;
             float y[32];
 #pragma unroll
-            for (int i = 0; i < 32; ++i) y[i] = DUAL ? silu_f32(v[i] * sc) * (u[i] * sc) : apply_activation(p.activation, v[i] * sc);
+            for (int i = 0; i < 32; ++i) y[i] = DUAL ? silu_f32(v[i] * sc) * (u[i] * sc) : v[i] * sc;
+            if (!DUAL && p.bias) {
+                const float* b = p.bias + n;
+#pragma unroll
+                for (int i = 0; i < 32; ++i)
+                    if (n + i < p.N) y[i] += b[i];
+            }
+            if (!DUAL && p.activation != SPITE_ACT_NONE) {
+#pragma unroll
+                for (int i = 0; i < 32; ++i) y[i] = apply_activation(p, y[i]);
+            }
             if (full && ((uintptr_t)dst & 15) == 0) {
 #pragma unroll
                 for (int i = 0; i < 32; i += 8) {

@@ -311,7 +311,7 @@ gemm_tc_experts_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_c
                         const float s = __shfl_sync(0xffffffffu, sc, t);
                         if (c0 + t < it.rows && n_ok) {
                             const float y = old[t] + v[t] * s;
-                            if (EPI == EPI_STORE) ((__nv_bfloat16*)p.C)[(size_t)r * p.ldc + n] = __float2bfloat16_rn(apply_activation(p.activation, y));
+                            if (EPI == EPI_STORE) ((__nv_bfloat16*)p.C)[(size_t)r * p.ldc + n] = __float2bfloat16_rn(apply_activation(p, y));
                             else ((float*)p.C)[(size_t)r * p.ldc + n] = y;
                         }
                     }

@@ -89,6 +89,9 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentPrepare
     // asked for before the sums, used after them (thread i: gate column i, pair i of the shared key part)
     int page = -1;
     if (p.write_cache) page = b.block_table[(size_t)b.seg_of_token[t] * b.table_width + pos / c.page_size];
+    // (a captured step's padding row, a copy of the first row, appends nothing: behind a recurrent layer it is not that row)
+    if (page >= 0 && t > 0 && pos == b.positions[0] && page == b.block_table[(size_t)b.seg_of_token[0] * b.table_width + pos / c.page_size])
+        page = -1;
     const float* kr = kv + p.kv_rank;
     const int first_gate = p.q_rank + p.kv_rank + p.rot_dim;
     float gate_in = 0.f, kr0 = 0.f, kr1 = 0.f;

@@ -1,0 +1,377 @@
+// Recurrent mixers whose state is a matrix per head that decays and takes one outer product a token, carried from token to
+// token in float32 in the request's state slot.  One walk serves two designs:
+//
+//   state space (Mamba-2):   dt = softplus(a + dt_bias),  S <- exp(-exp(A_log) dt) S + dt k v^T,   o = S^T q + D v
+//                            (one decay a head and token; q and k shared by a group of heads; read after the write)
+//   decaying memory (RWKV):  o = S^T q + (sum_i q_i u_i k_i) v,   S <- diag(w) S + k v^T,   w = exp(-exp(z + w0))
+//                            (a decay per key channel; the token itself enters the read-out through the bonus u)
+//
+// S is [dim keys, vdim values], zeros at the start of a sequence.  Everything is float32.
+//
+// Unlike a delta rule, what a token writes does not depend on the state, so the walk is bound by what its warps can issue,
+// not by one token's chain.  A warp is LR lanes along the keys times 32 / LR lanes along the values; a lane holds RP = 4 RPV
+// key rows (as packed pairs, for the two-at-a-time multiply-adds of sm_100) of CC value columns.  TB = LR / CC tokens form a
+// batch: their inputs arrive in one stage of a shared-memory ring by asynchronous copies two batches ahead, one barrier a
+// batch, and their partial read-outs (TB * CC a lane) are summed over the LR lanes by a halving exchange that leaves every
+// lane one finished number.  The order of the sums depends on the head's sizes alone, so the result does not depend on
+// how a sequence was cut into steps.
+//
+// The slot holds S transposed: value column j's keys are contiguous, [vdim, dim4] with dim4 = dim rounded up to a multiple
+// of four (the padding stays zero), so that a lane's rows are whole 16-byte groups and a warp's loads whole lines.
+#include "common.cuh"
+
+struct ScanParams {
+    const float* q; const float* k; const float* v;       // first element of token 0's q, k [kv_heads * dim], v [heads * vdim]
+    long long q_stride, k_stride, v_stride;               // floats between two tokens' rows
+    const float* w; long long w_stride;                   // decay per key channel [tokens, heads * dim], or null: per head
+    const float* scalars;                                 // [tokens, heads, 2]: (decay, dt) without w; (bonus, unused) with w
+    const float* skip;                                    // [heads] the factor D on v in the read-out, or null
+    float* out; long long out_stride;                     // [tokens, heads * vdim]
+    float* state; long long slot_stride;                  // state + slot * slot_stride + head * vdim * dim4
+    const int* cu_seqlens; const int* slots;
+    int n_segments, n_tokens, heads, kv_heads, dim, vdim;
+};
+
+namespace {
+
+typedef unsigned long long f2;                            // two packed floats
+
+__device__ __forceinline__ f2 pack2(float lo, float hi) {
+    f2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ void unpack2(f2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
+    f2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
+    f2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
+__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
+    const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(d), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+    const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(d), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
+
+constexpr int RING = 3;
+
+template <int LR, int RPV, int CC, bool CH>
+struct Shape {
+    static constexpr int TB = LR / CC;                    // tokens a batch
+    static constexpr int DP = LR * RPV * 4;               // key rows a warp covers
+    static constexpr int WC = 32 / LR * CC;               // value columns a warp covers
+    static constexpr int ROWS = CH ? 3 : 2;               // q, k (and w) of a token
+    static __host__ __device__ constexpr int token_floats(int warps) { return ROWS * DP + ((WC * warps + 3) & ~3) + 4; }
+};
+
+// grid (ceil(vdim / (WC * warps)), heads, segments)
+template <int LR, int RPV, int CC, bool CH>
+__global__ void __launch_bounds__(128) scan_kernel(const ScanParams p, const int wide) {
+    using SH = Shape<LR, RPV, CC, CH>;
+    constexpr int TB = SH::TB, DP = SH::DP, WC = SH::WC, NP = RPV * 2;
+    extern __shared__ __align__(16) float ring[];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    const int r = lane % LR, cl = lane / LR;
+    const int seg = blockIdx.z, head = blockIdx.y;
+    const int dim = p.dim, vdim = p.vdim, dim4 = (dim + 3) & ~3;
+    const int BC = WC * warps, c0 = blockIdx.x * BC;
+    const int tok_floats = SH::token_floats(warps);
+    // rows beyond dim stay zero in every stage (q and k; a decay there multiplies zeros)
+    if (DP > dim) {
+        const int gap = DP - dim;
+        for (int e = threadIdx.x; e < RING * TB * SH::ROWS * gap; e += blockDim.x) {
+            const int slot = e / (SH::ROWS * gap), i = e % (SH::ROWS * gap);
+            ring[(size_t)slot * tok_floats + (i / gap) * DP + dim + i % gap] = 0.f;
+        }
+    }
+    pdl_wait();
+    const int t0 = p.cu_seqlens[seg], t1 = p.cu_seqlens[seg + 1];
+    if (t0 >= t1) return;
+    const int slot = p.slots[seg];
+    if (seg > 0 && slot == p.slots[0]) {                  // a captured step's padding row (a copy of the first row): the state
+        for (int e = threadIdx.x; e < (t1 - t0) * BC; e += blockDim.x)      // moves on once; the copy's results are never read
+            if (c0 + e % BC < vdim) p.out[(size_t)(t0 + e / BC) * p.out_stride + (size_t)head * vdim + c0 + e % BC] = 0.f;
+        return;
+    }
+    const int kvh = head / (p.heads / p.kv_heads);
+    const float* qp = p.q + (size_t)kvh * dim;
+    const float* kp = p.k + (size_t)kvh * dim;
+    const float* vp = p.v + (size_t)head * vdim + c0;
+    const float* wp = CH ? p.w + (size_t)head * dim : nullptr;
+    const float* sp = p.scalars + 2 * head;
+
+    const int n_cols = min(BC, vdim - c0);
+    const int n_batches = (t1 - t0 + TB - 1) / TB;
+    auto issue = [&](int b) {
+        const int tb = t0 + b * TB, n = min(TB, t1 - tb);
+        float* stage = ring + (size_t)(b % RING) * TB * tok_floats;
+        if (b < n_batches) {
+            if (wide) {                                   // whole 16-byte groups everywhere
+                const int d4 = dim >> 2, v4 = n_cols >> 2, per = SH::ROWS * d4 + v4 + 1;
+                for (int e = threadIdx.x; e < per; e += blockDim.x) {
+                    const float* src;
+                    long long stride;
+                    int dst;
+                    if (e < d4) { src = qp + 4 * e; stride = p.q_stride; dst = 4 * e; }
+                    else if (e < 2 * d4) { src = kp + 4 * (e - d4); stride = p.k_stride; dst = DP + 4 * (e - d4); }
+                    else if (CH && e < 3 * d4) { src = wp + 4 * (e - 2 * d4); stride = p.w_stride; dst = 2 * DP + 4 * (e - 2 * d4); }
+                    else if (e < SH::ROWS * d4 + v4) { src = vp + 4 * (e - SH::ROWS * d4); stride = p.v_stride; dst = SH::ROWS * DP + 4 * (e - SH::ROWS * d4); }
+                    else { src = sp; stride = 2 * p.heads; dst = tok_floats - 4; }
+                    src += (size_t)tb * stride;
+                    float* d = stage + dst;
+                    if (e == per - 1) {
+                        for (int tt = 0; tt < n; ++tt, src += stride, d += tok_floats) { cp_async4(d, src); cp_async4(d + 1, src + 1); }
+                    } else {
+                        for (int tt = 0; tt < n; ++tt, src += stride, d += tok_floats) cp_async16(d, src);
+                    }
+                }
+            } else {
+                const int per = SH::ROWS * dim + n_cols + 2;
+                for (int e = threadIdx.x; e < per; e += blockDim.x) {
+                    const float* src;
+                    long long stride;
+                    int dst;
+                    if (e < dim) { src = qp + e; stride = p.q_stride; dst = e; }
+                    else if (e < 2 * dim) { src = kp + e - dim; stride = p.k_stride; dst = DP + e - dim; }
+                    else if (CH && e < 3 * dim) { src = wp + e - 2 * dim; stride = p.w_stride; dst = 2 * DP + e - 2 * dim; }
+                    else if (e < SH::ROWS * dim + n_cols) { src = vp + e - SH::ROWS * dim; stride = p.v_stride; dst = SH::ROWS * DP + e - SH::ROWS * dim; }
+                    else { const int i = e - SH::ROWS * dim - n_cols; src = sp + i; stride = 2 * p.heads; dst = tok_floats - 4 + i; }
+                    src += (size_t)tb * stride;
+                    float* d = stage + dst;
+                    for (int tt = 0; tt < n; ++tt, src += stride, d += tok_floats) cp_async4(d, src);
+                }
+            }
+        }
+        cp_commit();
+    };
+#pragma unroll 1
+    for (int b = 0; b < RING - 1; ++b) issue(b);
+
+    // the state: value column j = c0 + warp * WC + cl * CC + c, key rows 4 (r + LR i) .. + 3
+    float* st = p.state + (size_t)slot * p.slot_stride + (size_t)head * vdim * dim4;
+    const int j0 = warp * WC + cl * CC;                   // within the block's columns
+    f2 S[NP][CC];
+#pragma unroll
+    for (int c = 0; c < CC; ++c)
+#pragma unroll
+        for (int i = 0; i < RPV; ++i) {
+            const int row = 4 * (r + LR * i);
+            float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (row < dim4 && j0 + c < n_cols) f = *(const float4*)(st + (size_t)(c0 + j0 + c) * dim4 + row);
+            S[2 * i][c] = pack2(f.x, f.y); S[2 * i + 1][c] = pack2(f.z, f.w);
+        }
+
+    const float skip = p.skip ? p.skip[head] : 0.f;
+    auto token = [&](const float* in, float* o) {
+        f2 q[NP], k[NP], w[CH ? NP : 1];
+#pragma unroll
+        for (int i = 0; i < RPV; ++i) {
+            const int row = 4 * (r + LR * i);
+            const ulonglong2 a = *(const ulonglong2*)(in + row), b = *(const ulonglong2*)(in + DP + row);
+            q[2 * i] = a.x; q[2 * i + 1] = a.y; k[2 * i] = b.x; k[2 * i + 1] = b.y;
+            if constexpr (CH) {
+                const ulonglong2 d = *(const ulonglong2*)(in + 2 * DP + row);
+                w[2 * i] = d.x; w[2 * i + 1] = d.y;
+            }
+        }
+        f2 decay = 0;
+        float dt = 1.f;
+        if constexpr (!CH) { const float2 s = *(const float2*)(in + tok_floats - 4); decay = pack2(s.x, s.x); dt = s.y; }
+#pragma unroll
+        for (int c = 0; c < CC; ++c) {
+            const float v = CH ? in[SH::ROWS * DP + j0 + c] : dt * in[SH::ROWS * DP + j0 + c];
+            const f2 v2 = pack2(v, v);
+            f2 acc = 0;
+#pragma unroll
+            for (int i = 0; i < NP; ++i) {
+                if constexpr (CH) {
+                    acc = fma2(q[i], S[i][c], acc);
+                    S[i][c] = fma2(w[i], S[i][c], mul2(k[i], v2));
+                } else {
+                    S[i][c] = fma2(k[i], v2, mul2(decay, S[i][c]));
+                    acc = fma2(q[i], S[i][c], acc);
+                }
+            }
+            float lo, hi;
+            unpack2(acc, lo, hi);
+            o[c] = lo + hi;
+        }
+    };
+
+#pragma unroll 1
+    for (int b = 0; b < n_batches; ++b) {
+        cp_wait<RING - 2>();
+        __syncthreads();                                  // batch b has landed, and every thread is done with batch b - 1
+        issue(b + RING - 1);                              // (into the stage that batch b - 1 had)
+        const float* in = ring + (size_t)(b % RING) * TB * tok_floats;
+        const int tb = t0 + b * TB, n = min(TB, t1 - tb);
+        float o[TB * CC];
+        if (n == TB) {
+#pragma unroll
+            for (int tt = 0; tt < TB; ++tt) token(in + (size_t)tt * tok_floats, o + tt * CC);
+        } else {
+#pragma unroll
+            for (int tt = 0; tt < TB; ++tt) {
+                if (tt < n) token(in + (size_t)tt * tok_floats, o + tt * CC);
+                else
+#pragma unroll
+                    for (int c = 0; c < CC; ++c) o[tt * CC + c] = 0.f;
+            }
+        }
+        // sums over the LR lanes of the keys; lane r keeps number r = (token r / CC, column r % CC)
+#pragma unroll
+        for (int h = LR / 2; h >= 1; h >>= 1) {
+            const bool up = (r & h) != 0;
+#pragma unroll
+            for (int i = 0; i < h; ++i) {
+                const float give = up ? o[i] : o[i + h], keep = up ? o[i + h] : o[i];
+                o[i] = keep + __shfl_xor_sync(0xffffffffu, give, h);
+            }
+        }
+        const int tt = r / CC, j = j0 + r % CC;
+        if (tt < n && j < n_cols) {
+            const float* tok = in + (size_t)tt * tok_floats;
+            const float v = tok[SH::ROWS * DP + j];
+            p.out[(size_t)(tb + tt) * p.out_stride + (size_t)head * vdim + c0 + j] = fmaf(CH ? tok[tok_floats - 4] : skip, v, o[0]);
+        }
+    }
+    cp_wait<0>();
+#pragma unroll
+    for (int c = 0; c < CC; ++c)
+#pragma unroll
+        for (int i = 0; i < RPV; ++i) {
+            const int row = 4 * (r + LR * i);
+            if (row < dim4 && j0 + c < n_cols) {
+                float4 f;
+                unpack2(S[2 * i][c], f.x, f.y); unpack2(S[2 * i + 1][c], f.z, f.w);
+                *(float4*)(st + (size_t)(c0 + j0 + c) * dim4 + row) = f;
+            }
+        }
+    pdl_launch_dependents();                              // (late: the next kernel's blocks would only sit and wait)
+}
+
+// ---- what a token brings besides q, k and v
+// state space: scalars[t, h] = (exp(-exp(A_log[h]) dt), dt), dt = softplus(a[t, h] + dt_bias[h])
+__global__ void __launch_bounds__(128) state_space_gates_kernel(const float* __restrict__ a, long long stride,
+                                                                const float* __restrict__ a_log, const float* __restrict__ dt_bias,
+                                                                float* __restrict__ scalars, long long n, int heads) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    const long long t = i / heads;
+    const int h = (int)(i % heads);
+    const float z = a[t * stride + h] + dt_bias[h];
+    const float dt = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+    *(float2*)(scalars + 2 * i) = make_float2(expf(-expf(a_log[h]) * dt), dt);
+}
+
+// decaying memory: w[t, h, i] = exp(-exp(z + w0)) in place, scalars[t, h, 0] = sum_i q_i u_i k_i.  One warp per (token, head).
+__global__ void __launch_bounds__(128) memory_gates_kernel(float* __restrict__ w, long long w_stride, const float* __restrict__ w0,
+                                                           const float* __restrict__ q, long long q_stride,
+                                                           const float* __restrict__ k, long long k_stride,
+                                                           const float* __restrict__ u, float* __restrict__ scalars, long long rows,
+                                                           int heads, int dim) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31;
+    const long long row = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (row >= rows) return;
+    const long long t = row / heads;
+    const int h = (int)(row % heads);
+    float* wr = w + t * w_stride + (size_t)h * dim;
+    const float* qr = q + t * q_stride + (size_t)h * dim;
+    const float* kr = k + t * k_stride + (size_t)h * dim;
+    float s = 0.f;
+    for (int i = lane; i < dim; i += 32) {
+        wr[i] = expf(-expf(wr[i] + w0[h * dim + i]));
+        s = fmaf(qr[i] * u[h * dim + i], kr[i], s);
+    }
+    s = warp_sum(s);
+    if (lane == 0) *(float2*)(scalars + 2 * row) = make_float2(s, 0.f);
+}
+
+template <int LR, int RPV, int CC, bool CH>
+int launch_scan(const ScanParams& p, int wide, cudaStream_t st) {
+    using SH = Shape<LR, RPV, CC, CH>;
+    // four warps a block, fewer where a step has so few (segment, head) pairs that more and smaller blocks spread better
+    int warps = 4;
+    while (warps > 1 && ((long long)((p.vdim + SH::WC * warps - 1) / (SH::WC * warps)) * p.heads * p.n_segments < 148 ||
+                         SH::WC * (warps / 2) >= p.vdim)) warps /= 2;
+    const size_t bytes = (size_t)RING * SH::TB * SH::token_floats(warps) * sizeof(float);
+    auto kernel = scan_kernel<LR, RPV, CC, CH>;
+    if (bytes > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess)
+        return SPITE_LAUNCH_FAILED;
+    dim3 grid((p.vdim + SH::WC * warps - 1) / (SH::WC * warps), p.heads, p.n_segments);
+    // A step of single tokens is launched as a programmatic dependent; a longer walk in the ordinary way: started early, its
+    // blocks would take the multiprocessors that the kernel before frees first, several to one, for the whole walk.
+    if (p.n_tokens == p.n_segments) SPITE_LAUNCH(kernel, grid, 32 * warps, bytes, st, p, wide);
+    else kernel<<<grid, 32 * warps, bytes, st>>>(p, wide);
+    return spite_launch_status();
+}
+
+template <bool CH>
+int choose_scan(const ScanParams& p, cudaStream_t st) {
+    const auto al = [](const void* x) { return ((uintptr_t)x & 15) == 0; };
+    const int wide = p.dim % 4 == 0 && p.vdim % 4 == 0 && p.q_stride % 4 == 0 && p.k_stride % 4 == 0 && p.v_stride % 4 == 0 &&
+                     al(p.q) && al(p.k) && al(p.v) && (!CH || (p.w_stride % 4 == 0 && al(p.w)));
+    if (p.dim <= 32) return launch_scan<8, 1, 2, CH>(p, wide, st);
+    if (p.dim <= 64) return launch_scan<8, 2, 2, CH>(p, wide, st);
+    if (p.dim <= 128) return launch_scan<16, 2, 2, CH>(p, wide, st);
+    if (p.dim <= 256) return launch_scan<16, 4, 2, CH>(p, wide, st);
+    return launch_scan<32, 4, 4, CH>(p, wide, st);
+}
+
+int check_scan(const ScanParams* p) {
+    if (!p || !p->q || !p->k || !p->v || !p->out || !p->state || !p->cu_seqlens || !p->slots || !p->scalars) return SPITE_BAD_ARG;
+    if (p->n_segments < 0 || p->n_tokens < 0 || p->heads < 1 || p->kv_heads < 1 || p->heads % p->kv_heads || p->dim < 1 || p->vdim < 1)
+        return SPITE_BAD_ARG;
+    const long long dim4 = (p->dim + 3) & ~3;
+    if (p->slot_stride < (long long)p->heads * p->vdim * dim4 || p->out_stride < (long long)p->heads * p->vdim) return SPITE_BAD_ARG;
+    if (p->q_stride < 1 || p->k_stride < 1 || p->v_stride < 1) return SPITE_BAD_ARG;
+    if (p->slot_stride % 4 || ((uintptr_t)p->state & 15)) return SPITE_UNSUPPORTED;      // the state moves in 16-byte groups
+    if (p->dim > 512 || p->heads > 65535 || p->n_segments > 65535) return SPITE_UNSUPPORTED;
+    return SPITE_OK;
+}
+
+}  // namespace
+
+// `a` [tokens, heads] with rows of a_stride: the projection's step columns; p->scalars is filled here
+SPITE_API int spite_state_space_scan(const ScanParams* p, const float* a, long long a_stride, const float* a_log,
+                                     const float* dt_bias, void* stream) {
+    const int chk = check_scan(p);
+    if (chk != SPITE_OK) return chk;
+    if (!a || !a_log || !dt_bias || p->w || a_stride < p->heads) return SPITE_BAD_ARG;
+    if (p->n_segments == 0 || p->n_tokens == 0) return SPITE_OK;
+    cudaStream_t st = (cudaStream_t)stream;
+    const long long n = (long long)p->n_tokens * p->heads;
+    SPITE_LAUNCH(state_space_gates_kernel, (int)((n + 127) / 128), 128, 0, st, a, a_stride, a_log, dt_bias, (float*)p->scalars, n, p->heads);
+    if (cudaGetLastError() != cudaSuccess) return SPITE_LAUNCH_FAILED;
+    return choose_scan<false>(*p, st);
+}
+
+// p->w holds the decay's pre-activations on entry and the decays afterwards; `u` and `w0` [heads * dim]
+SPITE_API int spite_decay_scan(const ScanParams* p, const float* w0, const float* u, void* stream) {
+    const int chk = check_scan(p);
+    if (chk != SPITE_OK) return chk;
+    if (!w0 || !u || !p->w || p->w_stride < (long long)p->heads * p->dim || p->kv_heads != p->heads || p->skip) return SPITE_BAD_ARG;
+    if (p->n_segments == 0 || p->n_tokens == 0) return SPITE_OK;
+    cudaStream_t st = (cudaStream_t)stream;
+    const long long rows = (long long)p->n_tokens * p->heads;
+    if ((rows + 3) / 4 > 0x7fffffffLL) return SPITE_UNSUPPORTED;
+    SPITE_LAUNCH(memory_gates_kernel, (int)((rows + 3) / 4), 128, 0, st, (float*)p->w, p->w_stride, w0, p->q, p->q_stride, p->k,
+                 p->k_stride, u, (float*)p->scalars, rows, p->heads, p->dim);
+    if (cudaGetLastError() != cudaSuccess) return SPITE_LAUNCH_FAILED;
+    return choose_scan<true>(*p, st);
+}

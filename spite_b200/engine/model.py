@@ -15,6 +15,7 @@ from ..config import ConfigError, JunctionCall, ModelPlan, load_config
 from ..kernels import build as kernel_build
 from ..parts import BuildContext, ParamSpec, build_part
 from ..parts.base import _REGISTRIES
+from ..parts.streams import ResidualStreams
 from ..weights import bind_tensors, load_bound_tensors
 from ..weights.random_init import tensor_seed
 
@@ -51,8 +52,9 @@ class Model:
         self.embed_table = None
         self.head_weight = None
         self.position_table = None
+        self._ones = None if plan.streams is None else torch.ones(plan.streams, dtype=torch.float32, device=self.device)
         #: if set, called as `layer_tap(i, h)` after the i-th layer run of the order with the float32 residual
-        #: stream (for comparing a model layer by layer; the step then cannot be captured in a graph)
+        #: stream (the sum of the streams, if there are several; for comparing a model layer by layer; the step then cannot be captured in a graph)
         self.layer_tap = None
         self._check_caches()
 
@@ -186,6 +188,8 @@ class Model:
                      build=True) -> "Model":
         """The same from checkpoint tensors in memory ({checkpoint tensor name: tensor}, the names and
         layouts a model.safetensors of this architecture would have)."""
+        if hasattr(config, "with_tensor_shapes"):
+            config = config.with_tensor_shapes({n: tuple(t.shape) for n, t in checkpoint_tensors.items()})
         model = cls.from_config(config, dtype=dtype, device=device, kernels=kernels)
         if build and kernels is None:
             kernel_build.ensure_built(model.kernel_libraries())
@@ -198,12 +202,14 @@ class Model:
         k = self.kernels
         p = self.plan
         batch.shared.clear()
-        h = torch.empty((batch.n_tokens, p.hidden_size), dtype=torch.float32, device=self.device)
-        if self.position_table is None:
-            k.embed(self.embed_table, batch.token_ids, h, scale=p.embedding_scale)
+        if p.streams is not None:
+            x = torch.empty((batch.n_tokens, p.streams, p.hidden_size), dtype=torch.float32, device=self.device)
+            k.embed(self.embed_table, batch.token_ids, x, scale=p.embedding_scale, copies=p.streams)
+            h = ResidualStreams(k, x)
         else:
-            k.embed(self.embed_table, batch.token_ids, h, scale=p.embedding_scale,
-                    position_table=self.position_table, positions=batch.positions)
+            h = torch.empty((batch.n_tokens, p.hidden_size), dtype=torch.float32, device=self.device)
+            more = {} if self.position_table is None else dict(position_table=self.position_table, positions=batch.positions)
+            k.embed(self.embed_table, batch.token_ids, h, scale=p.embedding_scale, **more)
         h0 = None
         if self.junctions:                       # the embedding's output, which the junctions mix back in
             h0 = torch.empty_like(h)
@@ -215,13 +221,16 @@ class Model:
                 continue
             self.blocks[call.layer].forward(h, batch, storage.layer_cache(call.cache, call.write_cache))
             if self.layer_tap is not None:
-                self.layer_tap(runs, h)
+                self.layer_tap(runs, h if p.streams is None else h.total())
             runs += 1
         R = batch.logit_rows.numel()
         logits = torch.empty((R, p.vocab_size), dtype=torch.float32, device=self.device)
         if R:
             x = torch.empty((R, p.hidden_size), dtype=self.dtype, device=self.device)
-            self.final_norm.forward(h, x, rows=batch.logit_rows)
+            if p.streams is None:
+                self.final_norm.forward(h, x, rows=batch.logit_rows)
+            else:
+                h.enter(self._ones, self.final_norm, x, rows=batch.logit_rows, last=True)
             k.linear(x, self.head_weight, logits)
             if p.logit_scale != 1.0 or p.logit_softcap is not None:
                 k.transform_logits(logits, scale=p.logit_scale, softcap=p.logit_softcap)

@@ -50,8 +50,9 @@ class KernelSet:
         return {}
 
     # ---- elementwise
-    def embed(self, table, token_ids, out_h, *, scale=1.0, position_table=None, positions=None):
-        """out_h[m, :] (float32) = table[token_ids[m], :] (T) * scale; with a `position_table` [P, d] (T)
+    def embed(self, table, token_ids, out_h, *, scale=1.0, position_table=None, positions=None, copies=1):
+        """out_h[m, :] (float32) = table[token_ids[m], :] (T) * scale; with `copies` n, out_h is [M, n, d] and every row is
+        written n times (the start of several residual streams); with a `position_table` [P, d] (T)
         and `positions` [M] int32, + position_table[positions[m], :] (the factor applies to the token's row only)."""
         raise NotImplementedError
 
@@ -80,13 +81,14 @@ class KernelSet:
         """out (T) = h (float32), element by element: what a sublayer without a norm in front of it reads."""
         raise NotImplementedError
 
-    def short_conv(self, x, w, out, batch, state, *, channels, activation=None, state_offset=0):
+    def short_conv(self, x, w, out, batch, state, *, channels, activation=None, state_offset=0, bias=None):
         """A short causal convolution over time on the first `channels` columns of a projection's float32 output x
         [M, >= channels + c]: out[t, ch] = act(sum_j w[ch, j] * x[t - taps + 1 + j, ch]) within each segment, w float32
         [channels, taps]; rows before a segment's first token come from the request's slot, state[slot, state_offset :
         state_offset + (taps - 1) * channels] (float32 [taps - 1, channels], oldest first; zeros at the start of a
         sequence), which then receives the sequence's last taps - 1 rows of x.  The c = out.shape[1] - channels columns behind
         the channels are passed on unchanged.  out [M, channels + c] is T or float32; `activation` None or "silu".
+        `bias` float32 [channels] is added to a channel's sum before the activation.
         With one tap nothing is carried and `state` may be None."""
         raise NotImplementedError
 
@@ -94,21 +96,60 @@ class KernelSet:
         """out[m, :] (float32 [M, d]) = vec (float32 [d]), or += vec: a bias laid down for a product that adds to it."""
         raise NotImplementedError
 
-    def head_norm_gate(self, x, out, *, heads, size, gates=None, gate_column=0, gain=None, eps=None, gate_activation="sigmoid"):
+    def head_norm_gate(self, x, out, *, heads, size, gates=None, gate_column=0, gain=None, eps=None, gate_activation="sigmoid",
+                       out_column=None):
         """What stands between a mixer's heads and its output projection.  x [M, heads * size] (T, or float32: the
         result of a recurrence), out [M, heads * size] (T; may be x):
         out[m, h, j] = x[m, h, j] * r * gain[h * size + j] * sigmoid(gates[m, gate_column + h * size + j]) with
         r = rsqrt(mean_j x[m, h, :]^2 + eps) if `eps` is given (a norm of every head without a gain of its own), else 1;
         `gates` (a 2-D tensor of x's type, the gate columns of a wider product) and `gain` (float32) may be left out.
-        `gate_activation` "silu": the factor is z * sigmoid(z) of the gate column z instead of sigmoid(z)."""
+        `gate_activation` "silu": the factor is z * sigmoid(z) of the gate column z instead of sigmoid(z).
+        `out_column` c: out is a wider 2-D tensor and the result goes into its columns from c on."""
+        raise NotImplementedError
+
+    def turn_heads(self, x, out, batch, *, heads, size, rotation=None, scale=1.0, out_column=0):
+        """The other way from a mixer's heads to its output projection, for heads whose values were cached rotated by their
+        own position: out[m, out_column + h * size + e] (T, a 2-D tensor) = scale * (x[m, h, :size] turned back)[e], every pair
+        of `rotation` by minus the angle that the token's position turns it by (None: not turned).  x [M, heads * head_dim]
+        (T) with head_dim >= size: what lies behind a head's first `size` elements is left out."""
+        raise NotImplementedError
+
+    def gate_group_norm(self, x, z, gain, out, *, groups, eps, z_column=0):
+        """A gate first, a norm behind it: v = x[m, :] * silu(z[m, z_column:]); out[m, e] (T) = v[e] / sqrt(mean of v^2 over e's
+        part + eps) * gain[e], `groups` equal parts; x float32 [M, n], z float32 [M, >= z_column + n], gain float32 [n]."""
+        raise NotImplementedError
+
+    def token_shift(self, x, mu, out, batch, state, *, state_offset=0, offsets_out=None):
+        """out[g, m, :] (T) = x[m, :] + (x'[m, :] - x[m, :]) * mu[g, :] with x' the row of the token before in the sequence: for
+        a segment's first token the row in its request's slot (float32, state[slot, state_offset : state_offset + d]; zeros
+        at the start of a sequence), which then receives the segment's last row.  x [M, d] (T), mu float32 [n, d], out
+        [n, M, d]; `offsets_out` (int32 [n + 1]) receives g * M: the groups of a `batched_linear` over out."""
+        raise NotImplementedError
+
+    # ---- several residual streams
+    def streams(self, x, *, y=None, bias=None, scale=None, mix=None, w_out=None, w_in=None, gain=None, eps=None, next_out=None,
+                rows=None, write_back=True):
+        """Everything between two sublayers of a model with n residual streams x float32 [M, n, d] (hyper-connections).
+        With the sublayer's output y float32 [M, d]: v = (y + bias) * scale, and all streams at once from the old ones
+        x_t <- sum_s mix[s, t] x_s + w_out[t] v (mix [n, n], [from, to]).  With `next_out` [rows, d] (T or float32): what the
+        next sublayer reads, u = sum_s w_in[s] x_s of the streams just made, next_out = u / sqrt(mean(u^2) + eps) * gain (u
+        itself without a gain).  `rows` int32: only these tokens (row i of next_out is token rows[i]); `write_back` False:
+        the new streams are used for u and not stored.  All coefficients float32."""
         raise NotImplementedError
 
     # ---- matrix products: y = x W^T with W [out, in]
-    def linear(self, x, w, out, *, accumulate=False, row_scale=None, activation=None):
+    def linear(self, x, w, out, *, accumulate=False, row_scale=None, activation=None, bias=None, act_params=None):
         """out[M, N] = x[M, K] @ w[N, K]^T.  `out` is T, or float32 (logits); with
         `accumulate` it is float32 and the product is added to it (residual stream).
         `row_scale` [M] float32 multiplies the product's rows.  `activation` (with an output of type T):
-        "relu2": out = relu(s y)^2; "gelu_tanh": out = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))), z = s y."""
+        "relu2": out = relu(s y)^2; "gelu_tanh": out = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))), z = s y; "tanh";
+        "xielu" with `act_params` (a, b): a z^2 + z / 2 for z > 0, else b (e^z - 1 - z) + z / 2.  `bias` float32 [N] (with an
+        output of type T) is added to the scaled product before the activation: z = s y + bias."""
+        raise NotImplementedError
+
+    def batched_linear(self, x, w, offsets, out):
+        """out[g, M, N] (float32) = x[g, M, K] @ w[g, N, K]^T: one product per group on rows of its own; offsets int32 [G + 1]
+        on the device holds g * M."""
         raise NotImplementedError
 
     def linear_swiglu(self, x, w_gate_up, out, *, row_scale=None):
@@ -146,7 +187,7 @@ class KernelSet:
 
     # ---- attention
     def qk_prepare(self, qkv, q_out, batch, cache, *, num_heads, rotation, qk_norm, temperature,
-                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None):
+                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None, value_rotation=None):
         """Encode positions of q and k, normalise, scale q, append k and v to the cache.
         `bias` float32 [(nq + 2 nkv) hd]: added to the projection's columns before anything else.  `q_only`: a row of
         qkv holds the q heads alone (and `bias` theirs): the layer reads keys and values that another layer cached.
@@ -158,7 +199,9 @@ class KernelSet:
         value becomes (1 - lam) v + lam * other[m, column + g * head stride + i] before it is cached.
         `gates_out` float32 [M, nq]: receives sigmoid(qkv[m, (nq + 2 nkv) hd + h]), the columns after the heads.
         `norm_dim`: a q or k head has this many elements and zeros behind them up to hd (a cache row wider than the key):
-        the per-head norm takes its mean over them."""
+        the per-head norm takes its mean over them.
+        `value_rotation`: a `parts.Rotation` over the leading elements of a value head: a value turns by its own position
+        before it is cached."""
         raise NotImplementedError
 
     def paged_attention(self, q, out, batch, cache, *, num_heads, window, softmax_scale, cache_settled=False,
@@ -228,6 +271,27 @@ class KernelSet:
         g = exp(-exp(a_log[h]) * softplus(a + dt_bias[h])); S <- g S; u = beta (v - S^T k); S <- S + k u^T; out = S^T q.
         All float32.  `split_rows`: more lanes share a value column's key rows (the same sums in another order; for steps
         with long segments); None leaves the choice to the kernel set."""
+        raise NotImplementedError
+
+    @staticmethod
+    def scan_state_size(dim: int, vdim: int) -> int:
+        """Floats of one head's state in the two scans below: value column by value column, its keys padded to a multiple of four."""
+        return vdim * (-(-dim // 4) * 4)
+
+    def state_space_scan(self, q, k, v, step, out, batch, state, *, heads, kv_heads, dim, vdim, a_log, dt_bias, skip,
+                         state_offset=0):
+        """A state space with one decay per head and token (Mamba-2), for every segment of the step from the matrices its
+        request's slot holds (zeros: the start of a sequence); the slot receives the matrices after the segment's last
+        token.  Per head h: dt = softplus(step + dt_bias[h]); S <- exp(-exp(a_log[h]) dt) S + dt k v^T; out = S^T q + skip[h] v.
+        q, k, v, step are pairs (float32 tensor [M, *], first column) of widths kv_heads * dim (twice), heads * vdim and heads;
+        head h reads q and k of head h // (heads / kv_heads); out float32 [M, heads * vdim]; state float32 [slots, *], head h's
+        S at state[slot, state_offset + h * scan_state_size(dim, vdim)], transposed ([vdim, keys]).  All float32."""
+        raise NotImplementedError
+
+    def decay_scan(self, r, k, v, w, out, batch, state, *, heads, dim, vdim, w0, u, state_offset=0):
+        """A memory that decays per key channel (RWKV), walked and kept as above: out = S^T r + (sum_i r_i u_i k_i) v, then
+        S <- diag(exp(-exp(w + w0))) S + k v^T.  w float32 [M, heads * dim] holds the decay's pre-activations and is
+        overwritten with the decays; w0, u float32 [heads * dim]."""
         raise NotImplementedError
 
     # ---- mixture of experts

@@ -42,6 +42,7 @@ LIBRARIES = {
     "latent": (["latent.cu"], []),
     "recurrent": (["recurrent.cu"], []),
     "delta": (["delta.cu"], []),
+    "scan": (["scan.cu"], []),
     "sampling": (["sampling.cu"], []),
 }
 

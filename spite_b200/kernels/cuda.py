@@ -20,7 +20,7 @@ _STATUS = {-1: "malformed argument", -2: "size not supported by this kernel", -3
 
 EPI_STORE, EPI_STORE_F32, EPI_ADD_F32, EPI_SWIGLU = 0, 1, 2, 3
 _WINDOW = {"full": 0, "chunk": 1, "sliding": 2}
-_ACTIVATION = {None: 0, "relu2": 1, "gelu_tanh": 2}
+_ACTIVATION = {None: 0, "relu2": 1, "gelu_tanh": 2, "xielu": 3, "tanh": 4}
 
 
 class GemmParams(C.Structure):
@@ -29,7 +29,8 @@ class GemmParams(C.Structure):
                 ("row_scale", C.c_void_p),
                 ("lda", C.c_longlong), ("ldc", C.c_longlong), ("w_group_stride", C.c_longlong),
                 ("n_groups", C.c_int), ("M", C.c_int), ("N", C.c_int), ("K", C.c_int),
-                ("epilogue", C.c_int), ("scale_by_a_row", C.c_int), ("activation", C.c_int)]
+                ("epilogue", C.c_int), ("scale_by_a_row", C.c_int), ("activation", C.c_int),
+                ("bias", C.c_void_p), ("act_pos", C.c_float), ("act_neg", C.c_float)]
 
 
 class StepTokens(C.Structure):
@@ -51,7 +52,8 @@ class QkPrepareParams(C.Structure):
                 ("qkv_stride", C.c_longlong), ("rot_amplitude", C.c_float),
                 ("v_other", C.c_void_p), ("v_other_stride", C.c_longlong), ("v_other_head", C.c_int),
                 ("v_mix_dim", C.c_int), ("v_mix", C.c_float), ("gates_out", C.c_void_p),
-                ("bias", C.c_void_p), ("q_only", C.c_int), ("norm_dim", C.c_int)]
+                ("bias", C.c_void_p), ("q_only", C.c_int), ("norm_dim", C.c_int),
+                ("v_inv_freq", C.c_void_p), ("v_rotary_dim", C.c_int), ("v_pairing", C.c_int)]
 
 
 class AttentionParams(C.Structure):
@@ -81,7 +83,31 @@ class ShortConvParams(C.Structure):
     _fields_ = [("x", C.c_void_p), ("x_stride", C.c_longlong), ("w", C.c_void_p), ("out", C.c_void_p),
                 ("out_stride", C.c_longlong), ("state", C.c_void_p), ("slot_stride", C.c_longlong),
                 ("cu_seqlens", C.c_void_p), ("slots", C.c_void_p), ("n_segments", C.c_int), ("channels", C.c_int),
-                ("taps", C.c_int), ("copy_columns", C.c_int), ("activation", C.c_int), ("max_seg_len", C.c_int)]
+                ("taps", C.c_int), ("copy_columns", C.c_int), ("activation", C.c_int), ("max_seg_len", C.c_int),
+                ("bias", C.c_void_p)]
+
+
+class TokenShiftParams(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("mu", C.c_void_p), ("out", C.c_void_p), ("state", C.c_void_p),
+                ("slot_stride", C.c_longlong), ("seg_of_token", C.c_void_p), ("cu_seqlens", C.c_void_p),
+                ("slots", C.c_void_p), ("offsets_out", C.c_void_p), ("n_tokens", C.c_int), ("d", C.c_int),
+                ("n_mixes", C.c_int)]
+
+
+class StreamsParams(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("y", C.c_void_p), ("bias", C.c_void_p), ("scale", C.c_void_p), ("mix", C.c_void_p),
+                ("w_out", C.c_void_p), ("w_in", C.c_void_p), ("gain", C.c_void_p), ("next_out", C.c_void_p),
+                ("rows", C.c_void_p), ("n_rows", C.c_int), ("d", C.c_int), ("streams", C.c_int), ("write_back", C.c_int),
+                ("eps", C.c_float)]
+
+
+class ScanParams(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p),
+                ("q_stride", C.c_longlong), ("k_stride", C.c_longlong), ("v_stride", C.c_longlong),
+                ("w", C.c_void_p), ("w_stride", C.c_longlong), ("scalars", C.c_void_p), ("skip", C.c_void_p),
+                ("out", C.c_void_p), ("out_stride", C.c_longlong), ("state", C.c_void_p), ("slot_stride", C.c_longlong),
+                ("cu_seqlens", C.c_void_p), ("slots", C.c_void_p), ("n_segments", C.c_int), ("n_tokens", C.c_int),
+                ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int)]
 
 
 class DeltaParams(C.Structure):
@@ -323,10 +349,12 @@ class CudaKernels(KernelSet):
         return t
 
     # ------------------------------------------------------------------ elementwise
-    def embed(self, table, token_ids, out_h, *, scale=1.0, position_table=None, positions=None):
+    def embed(self, table, token_ids, out_h, *, scale=1.0, position_table=None, positions=None, copies=1):
         self._t(table, self.dtype, "table"); self._t(token_ids, torch.int32, "token_ids")
         self._t(out_h, torch.float32, "out_h")
         V, d = table.shape
+        if out_h.numel() != token_ids.numel() * copies * d or (copies != 1 and position_table is not None):
+            raise KernelError("embed: the output does not fit")
         if position_table is not None:
             self._t(position_table, self.dtype, "position_table"); self._t(positions, torch.int32, "positions")
             if position_table.shape[1] != d or positions.numel() != token_ids.numel():
@@ -340,7 +368,7 @@ class CudaKernels(KernelSet):
             return
         st = self._lib("elementwise").spite_embed(
             self._dt, C.c_void_p(table.data_ptr()), C.c_void_p(token_ids.data_ptr()),
-            C.c_void_p(out_h.data_ptr()), token_ids.numel(), d, V, C.c_float(scale), self._stream())
+            C.c_void_p(out_h.data_ptr()), token_ids.numel(), d, V, C.c_float(scale), int(copies), self._stream())
         self._count("elementwise", 1)
         _check(st, "embed")
 
@@ -405,7 +433,7 @@ class CudaKernels(KernelSet):
         self._count("elementwise", 1)
         _check(st, "cast_rows")
 
-    def short_conv(self, x, w, out, batch, state, *, channels, activation=None, state_offset=0):
+    def short_conv(self, x, w, out, batch, state, *, channels, activation=None, state_offset=0, bias=None):
         self._t(x, torch.float32, "x"); self._t(w, torch.float32, "w"); self._t(out, None, "out")
         if state is None and w.shape[1] == 1:
             state = x[:1]                                       # one tap: nothing is carried, and the kernel touches no slot
@@ -416,6 +444,8 @@ class CudaKernels(KernelSet):
         taps = w.shape[1]
         if w.shape[0] != channels or out.shape[0] != M or out.shape[1] < channels or x.shape[1] < out.shape[1]:
             raise KernelError("short_conv: shapes do not fit")
+        if bias is not None and self._t(bias, torch.float32, "bias").numel() != channels:
+            raise KernelError("short_conv: one bias per channel")
         if activation not in (None, "silu"):
             raise KernelError(f"short_conv: unknown activation {activation!r}")
         slot_stride = state[0].numel()
@@ -426,7 +456,7 @@ class CudaKernels(KernelSet):
                             state=state.data_ptr() + 4 * int(state_offset), slot_stride=slot_stride,
                             cu_seqlens=batch.cu_seqlens.data_ptr(), slots=batch.slots.data_ptr(), n_segments=n_seg,
                             channels=int(channels), taps=int(taps), copy_columns=out.shape[1] - int(channels),
-                            activation=1 if activation == "silu" else 0, max_seg_len=int(batch.max_seg_len))
+                            activation=1 if activation == "silu" else 0, max_seg_len=int(batch.max_seg_len), bias=_ptr(bias))
         st = self._lib("elementwise").spite_short_conv(_DT[out.dtype], C.byref(p), self._stream())
         self._count("elementwise", 1)
         _check(st, "short_conv")
@@ -441,15 +471,17 @@ class CudaKernels(KernelSet):
         self._count("elementwise", 1)
         _check(st, "fill_rows")
 
-    def head_norm_gate(self, x, out, *, heads, size, gates=None, gate_column=0, gain=None, eps=None, gate_activation="sigmoid"):
+    def head_norm_gate(self, x, out, *, heads, size, gates=None, gate_column=0, gain=None, eps=None, gate_activation="sigmoid",
+                       out_column=None):
         self._t(x, None, "x"); self._t(out, self.dtype, "out")
         if gate_activation not in ("sigmoid", "silu"):
             raise KernelError(f"head_norm_gate: unknown gate activation {gate_activation!r}")
         if x.dtype not in (self.dtype, torch.float32):
             raise KernelError(f"head_norm_gate: x must be {self.dtype} or float32")
         M = x.shape[0]
-        if tuple(x.shape) != (M, heads * size) or tuple(out.shape) != (M, heads * size):
+        if tuple(x.shape) != (M, heads * size) or (out_column is None and tuple(out.shape) != (M, heads * size)):
             raise KernelError("head_norm_gate: x and out must be [tokens, heads * size]")
+        o_ptr = self._columns(out, out_column or 0, heads * size, M, "head_norm_gate: out")
         g_ptr, g_stride = None, 0
         if gates is not None:
             self._t(gates, x.dtype, "gates")
@@ -460,10 +492,68 @@ class CudaKernels(KernelSet):
             raise KernelError("head_norm_gate: the gain must have heads * size elements")
         st = self._lib("elementwise").spite_head_norm_gate(
             _DT[x.dtype], self._dt, C.c_void_p(x.data_ptr()), C.c_void_p(g_ptr), C.c_longlong(g_stride),
-            C.c_void_p(_ptr(gain)), C.c_void_p(out.data_ptr()), M, int(heads), int(size), C.c_float(eps or 0.0),
+            C.c_void_p(_ptr(gain)), C.c_void_p(o_ptr), C.c_longlong(out.shape[1]), M, int(heads), int(size), C.c_float(eps or 0.0),
             int(gate_activation == "silu"), 1, self._stream())
         self._count("elementwise", 1)
         _check(st, "head_norm_gate")
+
+    @staticmethod
+    def _columns(t, column, width, rows, what):
+        """Address of column `column` of the 2-D tensor `t`, whose rows must have `width` columns from there on."""
+        if t.dim() != 2 or t.shape[0] != rows or column < 0 or column + width > t.shape[1]:
+            raise KernelError(f"{what} must be [tokens, *] with {width} columns from column {column} on")
+        return t.data_ptr() + int(column) * t.element_size()
+
+    def token_shift(self, x, mu, out, batch, state, *, state_offset=0, offsets_out=None):
+        self._t(x, self.dtype, "x"); self._t(mu, torch.float32, "mu"); self._t(out, self.dtype, "out")
+        self._t(state, torch.float32, "state")
+        M, d = x.shape
+        n = mu.shape[0]
+        slot_stride = state[0].numel()
+        if mu.shape[1] != d or tuple(out.shape) != (n, M, d) or state_offset < 0 or state_offset + d > slot_stride:
+            raise KernelError("token_shift: shapes do not fit")
+        if offsets_out is not None and self._t(offsets_out, torch.int32, "offsets_out").numel() != n + 1:
+            raise KernelError("token_shift: one offset per mix and one behind them")
+        p = TokenShiftParams(x=x.data_ptr(), mu=mu.data_ptr(), out=out.data_ptr(), state=state.data_ptr() + 4 * int(state_offset),
+                             slot_stride=slot_stride, seg_of_token=batch.seg_of_token.data_ptr(),
+                             cu_seqlens=batch.cu_seqlens.data_ptr(), slots=batch.slots.data_ptr(), offsets_out=_ptr(offsets_out),
+                             n_tokens=M, d=d, n_mixes=n)
+        st = self._lib("elementwise").spite_token_shift(self._dt, C.byref(p), self._stream())
+        self._count("elementwise", 1)
+        _check(st, "token_shift")
+
+    def gate_group_norm(self, x, z, gain, out, *, groups, eps, z_column=0):
+        self._t(x, torch.float32, "x"); self._t(z, torch.float32, "z"); self._t(gain, torch.float32, "gain")
+        self._t(out, self.dtype, "out")
+        M, n = x.shape
+        if n % groups or tuple(out.shape) != (M, n) or gain.numel() != n:
+            raise KernelError("gate_group_norm: shapes do not fit")
+        z_ptr = self._columns(z, z_column, n, M, "gate_group_norm: z")
+        st = self._lib("elementwise").spite_gate_group_norm(
+            self._dt, C.c_void_p(x.data_ptr()), C.c_void_p(z_ptr), C.c_longlong(z.shape[1]), C.c_void_p(gain.data_ptr()),
+            C.c_void_p(out.data_ptr()), M, int(groups), n // int(groups), C.c_float(eps), self._stream())
+        self._count("elementwise", 1)
+        _check(st, "gate_group_norm")
+
+    def streams(self, x, *, y=None, bias=None, scale=None, mix=None, w_out=None, w_in=None, gain=None, eps=None, next_out=None,
+                rows=None, write_back=True):
+        self._t(x, torch.float32, "x")
+        M, n, d = x.shape
+        for name, t, numel in (("y", y, M * d), ("bias", bias, d), ("scale", scale, d), ("mix", mix, n * n), ("w_out", w_out, n),
+                               ("w_in", w_in, n), ("gain", gain, d)):
+            if t is not None and self._t(t, torch.float32, name).numel() != numel:
+                raise KernelError(f"streams: {name} has {t.numel()} elements, {numel} are needed")
+        R = M
+        if rows is not None:
+            R = self._t(rows, torch.int32, "rows").numel()
+        if next_out is not None and (next_out.dtype not in _DT or tuple(self._t(next_out, None, "next_out").shape) != (R, d)):
+            raise KernelError("streams: next_out must be [rows, width]")
+        p = StreamsParams(x=x.data_ptr(), y=_ptr(y), bias=_ptr(bias), scale=_ptr(scale), mix=_ptr(mix), w_out=_ptr(w_out),
+                          w_in=_ptr(w_in), gain=_ptr(gain), next_out=_ptr(next_out), rows=_ptr(rows), n_rows=R, d=d, streams=n,
+                          write_back=int(bool(write_back)), eps=float(eps or 0.0))
+        st = self._lib("elementwise").spite_streams(_DT[next_out.dtype] if next_out is not None else 0, C.byref(p), self._stream())
+        self._count("elementwise", 1)
+        _check(st, "streams")
 
     def clear_pages(self, kv, page_ids):
         self._t(kv, None, "cache")
@@ -627,7 +717,7 @@ class CudaKernels(KernelSet):
         words[5] = 0
         return code
 
-    def linear(self, x, w, out, *, accumulate=False, row_scale=None, activation=None):
+    def linear(self, x, w, out, *, accumulate=False, row_scale=None, activation=None, bias=None, act_params=None):
         self._t(x, self.dtype, "x"); self._t(w, self.dtype, "w"); self._t(out, None, "out")
         M, K = x.shape
         N = w.shape[0]
@@ -645,9 +735,15 @@ class CudaKernels(KernelSet):
             raise KernelError(f"linear: output type {out.dtype} not supported")
         if activation not in _ACTIVATION or (activation is not None and epi != EPI_STORE):
             raise KernelError(f"linear: activation {activation!r} needs a plain store in the activation type")
+        if bias is not None and (epi != EPI_STORE or self._t(bias, torch.float32, "bias").numel() != N):
+            raise KernelError("linear: a bias goes with a plain store and has one element per output column")
+        if (activation == "xielu") != (act_params is not None):
+            raise KernelError("linear: act_params are the two coefficients of the activation 'xielu'")
+        pos, neg = act_params or (0.0, 0.0)
         p = GemmParams(A=x.data_ptr(), W=w.data_ptr(), C=out.data_ptr(), a_rows=None, c_rows=None,
                        group_offsets=None, row_scale=_ptr(row_scale), lda=K, ldc=N, w_group_stride=0,
-                       n_groups=1, M=M, N=N, K=K, epilogue=epi, scale_by_a_row=0, activation=_ACTIVATION[activation])
+                       n_groups=1, M=M, N=N, K=K, epilogue=epi, scale_by_a_row=0, activation=_ACTIVATION[activation],
+                       bias=_ptr(bias), act_pos=float(pos), act_neg=float(neg))
         self._gemm(p, "linear", M)
 
     def linear_swiglu(self, x, w_gate_up, out, *, row_scale=None):
@@ -721,6 +817,18 @@ class CudaKernels(KernelSet):
                        w_group_stride=N * K, n_groups=G, M=M, N=N, K=K, epilogue=EPI_STORE, scale_by_a_row=0)
         self._gemm(p, "grouped_linear_rows", M, gather_src=None if a_sorted else a)
 
+    def batched_linear(self, x, w, offsets, out):
+        self._t(x, self.dtype, "x"); self._t(w, self.dtype, "w"); self._t(out, torch.float32, "out")
+        self._t(offsets, torch.int32, "offsets")
+        G, M, K = x.shape
+        N = w.shape[1]
+        if w.shape[0] != G or w.shape[2] != K or tuple(out.shape) != (G, M, N) or offsets.numel() != G + 1:
+            raise KernelError("batched_linear: shapes do not fit")
+        p = GemmParams(A=x.data_ptr(), W=w.data_ptr(), C=out.data_ptr(), a_rows=None, c_rows=None,
+                       group_offsets=offsets.data_ptr(), row_scale=None, lda=K, ldc=N, w_group_stride=N * K,
+                       n_groups=G, M=G * M, N=N, K=K, epilogue=EPI_STORE_F32, scale_by_a_row=0)
+        self._gemm(p, "batched_linear", M)
+
     # ------------------------------------------------------------------ attention
     def _step_tokens(self, batch, group):
         bt = batch.block_tables[group]
@@ -734,7 +842,7 @@ class CudaKernels(KernelSet):
                           page_size=kv.shape[3], num_kv_heads=kv.shape[2], head_dim=kv.shape[4])
 
     def qk_prepare(self, qkv, q_out, batch, cache, *, num_heads, rotation, qk_norm, temperature,
-                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None):
+                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None, value_rotation=None):
         self._t(qkv, self.dtype, "qkv"); self._t(q_out, self.dtype, "q_out")
         head_dim = cache.kv.shape[4]
         n_cols = (num_heads + (0 if q_only else 2 * cache.kv.shape[2])) * head_dim
@@ -765,6 +873,12 @@ class CudaKernels(KernelSet):
             rotary_dim = int(rotation.rotary_dim or head_dim)
             if inv_freq.numel() != rotary_dim // 2:
                 raise KernelError(f"qk_prepare: {inv_freq.numel()} frequencies for {rotary_dim} rotating elements")
+        v_freq, v_dims, v_pairing = None, 0, 0
+        if value_rotation is not None:
+            f = self._t(value_rotation.inv_freq, torch.float32, "inv_freq")
+            v_freq, v_dims, v_pairing = f.data_ptr(), 2 * f.numel(), self._PAIRING[value_rotation.pairing]
+            if value_rotation.amplitude != 1.0 or (value_rotation.rotary_dim or v_dims) != v_dims:
+                raise KernelError("qk_prepare: values turn by a pure rotation")
         eps, before, q_gain, k_gain = 0.0, 0, None, None
         if qk_norm is not None:
             eps, before = float(qk_norm.eps), int(qk_norm.before_rotation)
@@ -780,12 +894,32 @@ class CudaKernels(KernelSet):
                             write_cache=int(cache.write), qkv_stride=qkv.shape[1], rot_amplitude=amplitude,
                             v_other=v_other, v_other_stride=v_stride, v_other_head=int(v_head), v_mix_dim=int(v_dim),
                             v_mix=float(v_lam), gates_out=_ptr(gates_out), bias=_ptr(bias), q_only=int(bool(q_only)),
-                            norm_dim=int(norm_dim or 0))
+                            norm_dim=int(norm_dim or 0), v_inv_freq=v_freq, v_rotary_dim=v_dims, v_pairing=v_pairing)
         b, c = self._step_tokens(batch, cache.group), self._paged(cache)
         st = self._lib("attention").spite_qk_prepare(self._dt, C.byref(p), C.byref(b), C.byref(c), self._stream())
         self._count("attention", 1)
         _check(st, "qk_prepare")
 
+    _PAIRING = {"neighbours": 0, "halves": 1}
+
+    def turn_heads(self, x, out, batch, *, heads, size, rotation=None, scale=1.0, out_column=0):
+        self._t(x, self.dtype, "x"); self._t(out, self.dtype, "out")
+        M = x.shape[0]
+        if x.shape[1] % heads or x.shape[1] // heads < size:
+            raise KernelError("turn_heads: x must be [tokens, heads * head_dim] with head_dim >= size")
+        o_ptr = self._columns(out, out_column, heads * size, M, "turn_heads: out")
+        freq, dims, pairing = None, 0, 0
+        if rotation is not None:
+            freq = self._t(rotation.inv_freq, torch.float32, "inv_freq")
+            dims, pairing = 2 * freq.numel(), self._PAIRING[rotation.pairing]
+            if rotation.amplitude != 1.0:
+                raise KernelError("turn_heads: heads turn back by a pure rotation")
+        st = self._lib("attention").spite_turn_heads(
+            self._dt, C.c_void_p(x.data_ptr()), C.c_void_p(o_ptr), C.c_longlong(out.shape[1]),
+            C.c_void_p(batch.positions.data_ptr()), C.c_void_p(_ptr(freq)), int(dims), pairing, M, int(heads),
+            x.shape[1] // heads, int(size), C.c_float(scale), self._stream())
+        self._count("attention", 1)
+        _check(st, "turn_heads")
 
     def paged_attention(self, q, out, batch, cache, *, num_heads, window, softmax_scale, cache_settled=False,
                         sink_logit=None, head_sinks=None, head_slopes=None, head_gates=None, out_by_head=False,
@@ -1030,6 +1164,57 @@ class CudaKernels(KernelSet):
         st = self._lib("delta").spite_delta_scan(C.byref(p), C.c_int(int(bool(split_rows))), self._stream())
         self._count("delta", 2)
         _check(st, "delta_scan")
+
+    def _scan(self, what, q, k, v, out, batch, state, *, heads, kv_heads, dim, vdim, state_offset):
+        """The argument block that both scans share; q, k, v are (float32 tensor [M, *], first column)."""
+        self._t(out, torch.float32, "out"); self._t(state, torch.float32, "state")
+        M = out.shape[0]
+        slot_stride = state[0].numel()
+        if tuple(out.shape) != (M, heads * vdim) or heads % kv_heads or state_offset < 0 \
+                or state_offset + heads * self.scan_state_size(dim, vdim) > slot_stride:
+            raise KernelError(f"{what}: shapes do not fit")
+        at = []
+        for name, (t, column), width in (("q", q, kv_heads * dim), ("k", k, kv_heads * dim), ("v", v, heads * vdim)):
+            self._t(t, torch.float32, name)
+            at.append((self._columns(t, column, width, M, f"{what}: {name}"), t.shape[1]))
+        scalars = torch.empty((M, heads, 2), dtype=torch.float32, device=out.device)
+        p = ScanParams(q=at[0][0], k=at[1][0], v=at[2][0], q_stride=at[0][1], k_stride=at[1][1], v_stride=at[2][1],
+                       w=None, w_stride=0, scalars=scalars.data_ptr(), skip=None, out=out.data_ptr(), out_stride=out.shape[1],
+                       state=state.data_ptr() + 4 * int(state_offset), slot_stride=slot_stride,
+                       cu_seqlens=batch.cu_seqlens.data_ptr(), slots=batch.slots.data_ptr(),
+                       n_segments=batch.cu_seqlens.numel() - 1, n_tokens=M, heads=int(heads), kv_heads=int(kv_heads),
+                       dim=int(dim), vdim=int(vdim))
+        return p, scalars
+
+    def state_space_scan(self, q, k, v, step, out, batch, state, *, heads, kv_heads, dim, vdim, a_log, dt_bias, skip,
+                         state_offset=0):
+        p, scalars = self._scan("state_space_scan", q, k, v, out, batch, state, heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim,
+                                state_offset=state_offset)
+        for name, t in (("a_log", a_log), ("dt_bias", dt_bias), ("skip", skip)):
+            if self._t(t, torch.float32, name).numel() != heads:
+                raise KernelError(f"state_space_scan: {name} has one element per head")
+        t, column = step
+        self._t(t, torch.float32, "step")
+        a = self._columns(t, column, heads, out.shape[0], "state_space_scan: step")
+        p.skip = skip.data_ptr()
+        st = self._lib("scan").spite_state_space_scan(C.byref(p), C.c_void_p(a), C.c_longlong(t.shape[1]),
+                                                      C.c_void_p(a_log.data_ptr()), C.c_void_p(dt_bias.data_ptr()), self._stream())
+        self._count("scan", 2)
+        _check(st, "state_space_scan")
+
+    def decay_scan(self, r, k, v, w, out, batch, state, *, heads, dim, vdim, w0, u, state_offset=0):
+        p, scalars = self._scan("decay_scan", r, k, v, out, batch, state, heads=heads, kv_heads=heads, dim=dim, vdim=vdim,
+                                state_offset=state_offset)
+        self._t(w, torch.float32, "w")
+        if tuple(w.shape) != (out.shape[0], heads * dim):
+            raise KernelError("decay_scan: w must be [tokens, heads * dim]")
+        for name, t in (("w0", w0), ("u", u)):
+            if self._t(t, torch.float32, name).numel() != heads * dim:
+                raise KernelError(f"decay_scan: {name} has one element per head and key channel")
+        p.w, p.w_stride = w.data_ptr(), w.shape[1]
+        st = self._lib("scan").spite_decay_scan(C.byref(p), C.c_void_p(w0.data_ptr()), C.c_void_p(u.data_ptr()), self._stream())
+        self._count("scan", 2)
+        _check(st, "decay_scan")
 
     # ------------------------------------------------------------------ mixture of experts
     def moe_identity(self, x, routing, first_identity, out, *, accumulate=True):

@@ -7,7 +7,8 @@ temperature factor, a value size that differs from the key size, a sink in
 the softmax (an extra term exp(sink) in the sum, with nothing behind it; one score for all heads or a learned
 one per head), a bias that grows with the distance between query and key, a gate on every head's output (one
 number a head, or one for every element of the concatenated heads), biases on the four projections, the
-blending of the values with those of another layer, and keys and values that are not the layer's own but those
+blending of the values with those of another layer, values cached rotated by their own position (and every head's
+result turned back by the query's), and keys and values that are not the layer's own but those
 another layer cached are constructor parameters.
 
 Formulas: crates/spite-models/src/llama/llama4.rs:126-207 (projections, rotation
@@ -36,7 +37,8 @@ class PagedAttention(Mixer):
                  position: PartSpec, window=("full", 0), qk_norm_eps=None, qk_norm_gain=False,
                  qk_norm_before_rotation=False, temperature_tuning=None, softmax_scale=None,
                  value_dim=None, sink_logit=None, head_sinks=False, distance_slopes=None, head_gate=False,
-                 value_mix=None, bias=False, output_gate=False, kv_shared=False, conv_taps=None, score_softcap=None):
+                 value_mix=None, bias=False, output_gate=False, kv_shared=False, conv_taps=None, score_softcap=None,
+                 value_rotation: PartSpec | None = None):
         """`head_dim` is the size of a query and a key head, `value_dim` that of a value head (default: the
         same).  `sink_logit`, if given, is the score of a sink: a term exp(sink) in every softmax's sum that adds
         nothing to the output, p_j = exp(s_j) / (exp(sink) + sum exp(s_j')); with `head_sinks` the score is a
@@ -53,7 +55,10 @@ class PagedAttention(Mixer):
         `conv_taps` n: q, k and v pass a causal convolution over time of n taps per channel (`q_conv`, `k_conv`, `v_conv`
         [channels, n], the last column the current token's) directly behind their projections, before norm and
         rotation; a request's last n - 1 projected rows are kept in its state slot.  `score_softcap` c: a scaled score s
-        becomes c tanh(s / c) before the softmax."""
+        becomes c tanh(s / c) before the softmax.
+        `value_rotation`, a position part that rotates the whole value head: value j turns by its position j before it is
+        cached, and a head's result at position i is turned back by i before the output projection (so a value
+        enters turned by its distance, and nothing else of the attention knows about it)."""
         super().__init__(ctx)
         self.conv_taps = None if conv_taps is None else int(conv_taps)
         if self.conv_taps is not None and (self.conv_taps < 1 or self.conv_taps > 8):
@@ -106,6 +111,13 @@ class PagedAttention(Mixer):
         may_pad = rot is None or rot.rotary_dim is not None
         if self.kd % 2 and not may_pad:
             raise ConfigError(f"head_dim {head_dim} must be even where heads rotate or are normed")
+        self.value_rotation = None
+        if value_rotation is not None:
+            self.value_rotation = build_part("position", value_rotation, ctx).rotation()
+            if self.value_rotation is not None and 2 * self.value_rotation.inv_freq.numel() != self.vd:
+                raise ConfigError(f"a rotation of {2 * self.value_rotation.inv_freq.numel()} elements for value heads of {self.vd}")
+            if kv_shared or value_mix or self.output_gate:
+                raise ConfigError("rotated values cannot be combined with borrowed or blended values or a gate per element")
         hd = max(self.kd, self.vd)
         step = 16 if self.vd != self.kd and ctx.dtype == torch.bfloat16 and hd <= 128 else 2
         self.hd = -(-hd // step) * step
@@ -202,8 +214,9 @@ class PagedAttention(Mixer):
             self.head_sinks = params["sinks"].to(torch.float32).contiguous()
         if self.value_mix == "blend":
             self.value_lambda = float(params["value_mix"].to(torch.float32))
-        # the output projection's columns, head by head, with zero columns for the padding
-        self.wo = self._pad_heads(params["o_proj"].to(dt).t().contiguous(), self.nq, self.vd).t().contiguous()
+        # the output projection's columns, head by head, with zero columns for the padding (heads that are turned back leave
+        # their padding behind on the way)
+        self.wo = params["o_proj"].to(dt).contiguous() if self.value_rotation is not None else self._pad_heads(params["o_proj"].to(dt).t().contiguous(), self.nq, self.vd).t().contiguous()
         if self.qk_norm_gain:
             def gain(name):                                      # (zeros for the padding of a head)
                 g = torch.zeros((self.hd,), dtype=torch.float32, device=params[name].device)
@@ -212,7 +225,7 @@ class PagedAttention(Mixer):
             self.qk_norm = QkNorm(self.qk_norm_eps, self.qk_norm_before_rotation, gain("q_norm"), gain("k_norm"))
 
     def weight_bytes(self):
-        return (self.wqkv.numel() + self.wo.numel()) * self.wqkv.element_size()
+        return (self.wqkv.numel() + (0 if self.wo is None else self.wo.numel())) * self.wqkv.element_size()
 
     def cache_request(self):
         state = None
@@ -220,7 +233,28 @@ class PagedAttention(Mixer):
             state = FixedState(((self.conv_taps - 1) * (self.nq + 2 * self.nkv) * self.hd,), torch.float32)
         return PagedKV(self.window, self.nkv, self.hd), state
 
+    @property
+    def heads_size(self):
+        return None if self.has_bias else self.nq * self.vd
+
+    def heads(self, x, out, column, batch, cache, scale=1.0):
+        o = self._attend(x, batch, cache)
+        self.k.turn_heads(o, out, batch, heads=self.nq, size=self.vd, rotation=self.value_rotation, scale=scale, out_column=column)
+
     def forward(self, x, h, batch, cache, accumulate=True):
+        o = self._attend(x, batch, cache)
+        k = self.k
+        if self.value_rotation is not None:
+            a = torch.empty((x.shape[0], self.nq * self.vd), dtype=x.dtype, device=x.device)
+            k.turn_heads(o, a, batch, heads=self.nq, size=self.vd, rotation=self.value_rotation)
+            o = a
+        if self.o_bias is not None:
+            k.fill_rows(h, self.o_bias, accumulate=accumulate)
+            accumulate = True
+        k.linear(o, self.wo, h, accumulate=accumulate)
+
+    def _attend(self, x, batch, cache):
+        """The heads' results [M, heads * cache row], gated if the layer has gates."""
         M = x.shape[0]
         k = self.k
         qkv = torch.empty((M, self.wqkv.shape[0]), dtype=x.dtype, device=x.device)
@@ -254,6 +288,8 @@ class PagedAttention(Mixer):
             if cache.write:
                 raise ConfigError("a layer without keys and values of its own was given a cache to write")
             extra["q_only"] = True
+        if self.value_rotation is not None:
+            extra["value_rotation"] = self.value_rotation
         k.qk_prepare(qkv, q, batch, cache, num_heads=self.nq, rotation=self.position.rotation(),
                      qk_norm=self.qk_norm, temperature=self.temperature, **extra)
         o = torch.empty_like(q)
@@ -272,7 +308,4 @@ class PagedAttention(Mixer):
                           softmax_scale=self.softmax_scale, cache_settled=True, sink_logit=self.sink_logit, **more)
         if self.output_gate:
             k.head_norm_gate(o, o, heads=self.nq, size=self.hd, gates=qkv, gate_column=self.head_columns)
-        if self.o_bias is not None:
-            k.fill_rows(h, self.o_bias, accumulate=accumulate)
-            accumulate = True
-        k.linear(o, self.wo, h, accumulate=accumulate)
+        return o

@@ -12,6 +12,7 @@ Kinds of parts and what each must provide:
                  leading elements of a head rotate) or None
   mixer          `cache_request()`, `forward(x, h, batch, cache)`: adds its output into h
   feed_forward   `forward(x, h, batch)`: adds its output into h
+  connection     how a sublayer hangs on several residual streams (`streams.py`)
   block          `places` (name -> family of each part it is made of),
                  `forward(h, batch, cache)`: one layer on the residual stream h
   junction       `forward(h, h0, batch, step)`: rewrites h between two layers; h0 is the
@@ -31,7 +32,7 @@ import torch
 from ..config.specs import ConfigError, PartSpec
 
 _REGISTRIES: dict[str, dict[str, type]] = {
-    "norm": {}, "position": {}, "mixer": {}, "feed_forward": {}, "block": {}, "junction": {},
+    "norm": {}, "position": {}, "mixer": {}, "feed_forward": {}, "block": {}, "junction": {}, "connection": {},
 }
 
 
@@ -67,6 +68,10 @@ def register_junction(kind):
     return _register("junction", kind)
 
 
+def register_connection(kind):
+    return _register("connection", kind)
+
+
 def registered(family: str) -> list[str]:
     return sorted(_REGISTRIES[family])
 
@@ -87,6 +92,20 @@ def build_part(family: str, spec: PartSpec, ctx: BuildContext):
         return reg[spec.kind](ctx, **spec.params)
     except TypeError as e:
         raise ConfigError(f"{family} {spec.kind!r}: bad parameters {sorted(spec.params)} ({e})") from None
+
+
+_SIDE_STREAMS: dict = {}      # one side stream per device, shared by the layers
+
+
+def side_stream(x):
+    """The device's side stream for work that runs beside the main stream within a layer; None without a GPU.  The caller
+    forks it from the main stream and joins it again before the layer ends."""
+    if not x.is_cuda:
+        return None
+    side = _SIDE_STREAMS.get(x.device)
+    if side is None:
+        side = _SIDE_STREAMS[x.device] = torch.cuda.Stream(device=x.device)
+    return side
 
 
 @dataclass(frozen=True)
@@ -161,6 +180,20 @@ class Mixer(Part):
     #: stream's shape that holds nothing yet) with its output instead of adding to it.  An arrangement that norms a
     #: sublayer's output before it joins the stream asks for this; for parts without it the arrangement zeroes the buffer.
     can_store = False
+    #: width of the concatenated heads in front of the output projection, for mixers whose forward is
+    #: `heads` followed by one product with the parameter `o_proj` [hidden, heads_size]; None: not such a mixer
+    heads_size = None
+
+    def heads(self, x, out, column, batch, cache, scale=1.0):
+        """The mixer up to its output projection: the heads, times `scale`, into the columns of the 2-D tensor `out` (the
+        activation type) from `column` on.  An arrangement that puts several mixers' heads through one product uses it."""
+        raise NotImplementedError
+
+    def drop_output_projection(self):
+        """The output projection is somebody else's now (after `bind`): forget the copy."""
+        for name in ("wo", "w_out"):
+            if hasattr(self, name):
+                setattr(self, name, None)
 
     def cache_request(self):
         """(PagedKV | None, FixedState | None): what one cache of this mixer holds."""
@@ -172,6 +205,9 @@ class Mixer(Part):
 
 class FeedForward(Part):
     can_store = False            # as for mixers
+    #: float32 [hidden]: a bias on the output that an arrangement may add itself (fused with what it does to the output):
+    #: `forward(..., accumulate=False, add_bias=False)` then leaves it out
+    output_bias = None
 
     def forward(self, x, h, batch):
         raise NotImplementedError

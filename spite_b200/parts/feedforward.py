@@ -7,13 +7,12 @@ input, SwiGLU experts, unweighted sum).
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..config.specs import ConfigError
-from .base import FeedForward, ParamSpec, register_feed_forward
-
-
-_SIDE_STREAMS: dict = {}      # one side stream per device, shared by the layers
+from .base import FeedForward, ParamSpec, register_feed_forward, side_stream
 
 
 @register_feed_forward("dense_swiglu")
@@ -163,46 +162,63 @@ class MoESigmoidPrescaled(FeedForward):
             k.grouped_linear_accumulate(a, self.w_down, routing.sorted_rows[slot], routing.offsets[slot], h)
 
     def _side_stream(self, x):
-        if not x.is_cuda or not self.router_beside_shared:
-            return None
-        side = _SIDE_STREAMS.get(x.device)
-        if side is None:
-            side = _SIDE_STREAMS[x.device] = torch.cuda.Stream(device=x.device)
-        return side
+        return side_stream(x) if self.router_beside_shared else None
 
 
 @register_feed_forward("dense_activation")
 class DenseActivation(FeedForward):
     """h += down( act(up x) ) without a gate; `activation` "relu2": act(z) = relu(z)^2; "gelu_tanh":
-    act(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))); applied to the float32 sums of the first product
-    before they are rounded."""
+    act(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))); "xielu" with two learned numbers p, q (parameter `act` [2]):
+    softplus(p) z^2 + z / 2 for z > 0, (1/2 + softplus(q)) (e^z - 1 - z) + z / 2 for z <= 0; applied to the float32 sums of
+    the first product before they are rounded.  `bias`: both projections add one (`up_bias`, `down_bias`); the first
+    joins the activation in the product's epilogue."""
     graph_safe = True
     can_store = True
     kernel_libraries = ("gemm_simt",)
 
-    ACTIVATIONS = ("relu2", "gelu_tanh")
+    ACTIVATIONS = ("relu2", "gelu_tanh", "xielu")
 
-    def __init__(self, ctx, hidden_size: int, intermediate_size: int, activation: str = "relu2"):
+    def __init__(self, ctx, hidden_size: int, intermediate_size: int, activation: str = "relu2", bias: bool = False):
         super().__init__(ctx)
         if activation not in self.ACTIVATIONS:
             raise ConfigError(f"unknown activation {activation!r}; known: {', '.join(self.ACTIVATIONS)}")
-        self.d, self.f, self.activation = int(hidden_size), int(intermediate_size), activation
-        self.w_up = self.w_down = None
+        self.d, self.f, self.activation, self.bias = int(hidden_size), int(intermediate_size), activation, bool(bias)
+        self.w_up = self.w_down = self.up_bias = self.output_bias = self.act_params = None
 
     def param_specs(self):
-        return {"up_proj": ParamSpec((self.f, self.d)), "down_proj": ParamSpec((self.d, self.f))}
+        specs = {"up_proj": ParamSpec((self.f, self.d)), "down_proj": ParamSpec((self.d, self.f))}
+        if self.bias:
+            specs.update({"up_bias": ParamSpec((self.f,)), "down_bias": ParamSpec((self.d,))})
+        if self.activation == "xielu":
+            specs["act"] = ParamSpec((2,))
+        return specs
 
     def bind(self, params):
         dt = self.ctx.dtype
         self.w_up = params["up_proj"].to(dt).contiguous()
         self.w_down = params["down_proj"].to(dt).contiguous()
+        if self.bias:
+            self.up_bias = params["up_bias"].to(torch.float32).contiguous()
+            self.output_bias = params["down_bias"].to(torch.float32).contiguous()
+        if self.activation == "xielu":
+            p, q = (float(v) for v in params["act"].to(torch.float32).cpu())
+            softplus = lambda v: max(v, 0.0) + math.log1p(math.exp(-abs(v)))
+            self.act_params = (softplus(p), 0.5 + softplus(q))
 
     def weight_bytes(self):
         return (self.w_up.numel() + self.w_down.numel()) * self.w_down.element_size()
 
-    def forward(self, x, h, batch, accumulate=True):
+    def forward(self, x, h, batch, accumulate=True, add_bias=True):
         a = torch.empty((x.shape[0], self.f), dtype=x.dtype, device=x.device)
-        self.k.linear(x, self.w_up, a, activation=self.activation)
+        more = {}
+        if self.up_bias is not None:
+            more["bias"] = self.up_bias
+        if self.act_params is not None:
+            more["act_params"] = self.act_params
+        self.k.linear(x, self.w_up, a, activation=self.activation, **more)
+        if add_bias and self.output_bias is not None:
+            self.k.fill_rows(h, self.output_bias, accumulate=accumulate)
+            accumulate = True
         self.k.linear(a, self.w_down, h, accumulate=accumulate)
 
 

@@ -129,3 +129,17 @@ def open_checkpoint(folder) -> list[SafetensorsFile]:
     if not single.is_file():
         raise SafetensorsError(f"{folder}: neither model.safetensors nor model.safetensors.index.json found")
     return [SafetensorsFile(single)]
+
+
+def checkpoint_shapes(folder) -> dict:
+    """{tensor name: shape} of what the folder's files hold (empty where there is no readable file yet); headers alone are read."""
+    try:
+        files = open_checkpoint(folder)
+    except SafetensorsError:
+        return {}
+    shapes = {}
+    for f in files:
+        with f:
+            for name in f.names():
+                shapes[name] = tuple(f.entries[name][1])
+    return shapes

@@ -24,11 +24,11 @@ class TorchReferenceKernels(KernelSet):
         self.acc = acc
 
     # ---- elementwise
-    def embed(self, table, token_ids, out_h, *, scale=1.0, position_table=None, positions=None):
+    def embed(self, table, token_ids, out_h, *, scale=1.0, position_table=None, positions=None, copies=1):
         x = table[token_ids.long()].to(self.acc) * scale
         if position_table is not None:
             x = x + position_table[positions.long()].to(self.acc)
-        out_h.copy_(x.to(out_h.dtype))
+        out_h.copy_(x.to(out_h.dtype) if copies == 1 else x.to(out_h.dtype)[:, None].expand_as(out_h))
 
     def pack_pair(self, a, b, out, *, refill=None):
         out.copy_(torch.cat([a, b], -1).to(out.dtype))
@@ -62,7 +62,7 @@ class TorchReferenceKernels(KernelSet):
     def cast_rows(self, h, out):
         out.copy_(h.to(out.dtype))
 
-    def short_conv(self, x, w, out, batch, state, *, channels, activation=None, state_offset=0):
+    def short_conv(self, x, w, out, batch, state, *, channels, activation=None, state_offset=0, bias=None):
         taps = w.shape[1]
         cu = batch.cu_seqlens.tolist()
         slots = batch.slots.tolist()
@@ -82,6 +82,8 @@ class TorchReferenceKernels(KernelSet):
                 y = torch.zeros(channels, dtype=self.acc)
                 for j in range(taps):
                     y = y + wv[:, j] * hist[i + j]
+                if bias is not None:
+                    y = y + bias.to(self.acc)
                 if activation == "silu":
                     y = y * torch.sigmoid(y)
                 out[cu[s] + i, :channels] = y.to(out.dtype)
@@ -124,7 +126,8 @@ class TorchReferenceKernels(KernelSet):
         else:
             out.copy_(vec[None, :].to(out.dtype).expand_as(out))
 
-    def head_norm_gate(self, x, out, *, heads, size, gates=None, gate_column=0, gain=None, eps=None, gate_activation="sigmoid"):
+    def head_norm_gate(self, x, out, *, heads, size, gates=None, gate_column=0, gain=None, eps=None, gate_activation="sigmoid",
+                       out_column=None):
         M = x.shape[0]
         v = x.to(self.acc).reshape(M, heads, size)
         if eps is not None:
@@ -135,7 +138,109 @@ class TorchReferenceKernels(KernelSet):
         if gates is not None:
             z = gates[:, gate_column:gate_column + heads * size].to(self.acc)
             v = v * (torch.sigmoid(z) * z if gate_activation == "silu" else torch.sigmoid(z))
-        out.copy_(v.to(out.dtype))
+        c = out_column or 0
+        out[:, c:c + heads * size] = v.to(out.dtype)
+
+    def turn_heads(self, x, out, batch, *, heads, size, rotation=None, scale=1.0, out_column=0):
+        M = x.shape[0]
+        v = x.to(self.acc).reshape(M, heads, -1)[:, :, :size].clone()
+        if rotation is not None:
+            v = self._turn(v, batch.positions, rotation, -1.0)
+        out[:, out_column:out_column + heads * size] = (v * scale).reshape(M, heads * size).to(out.dtype)
+
+    def _turn(self, v, positions, rotation, sign):
+        """v [M, heads, size]: the leading pairs turn by sign * position * frequency."""
+        n = rotation.inv_freq.numel()
+        a = sign * positions.to(self.acc)[:, None] * rotation.inv_freq.to(self.acc)[None, :]
+        c, s = torch.cos(a)[:, None, :], torch.sin(a)[:, None, :]
+        i0, i1 = (slice(0, n), slice(n, 2 * n)) if rotation.pairing == "halves" else (slice(0, 2 * n, 2), slice(1, 2 * n, 2))
+        out = v.clone()
+        out[..., i0] = v[..., i0] * c - v[..., i1] * s
+        out[..., i1] = v[..., i1] * c + v[..., i0] * s
+        return out
+
+    def gate_group_norm(self, x, z, gain, out, *, groups, eps, z_column=0):
+        M, n = x.shape
+        g = z[:, z_column:z_column + n].to(self.acc)
+        v = (x.to(self.acc) * g * torch.sigmoid(g)).reshape(M, groups, n // groups)
+        v = v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps)
+        out.copy_((v.reshape(M, n) * gain.to(self.acc)).to(out.dtype))
+
+    def token_shift(self, x, mu, out, batch, state, *, state_offset=0, offsets_out=None):
+        M, d = x.shape
+        cu, slots = batch.cu_seqlens.tolist(), batch.slots.tolist()
+        xv = x.to(self.acc)
+        before = torch.zeros_like(xv)
+        for s in range(len(cu) - 1):
+            copy = s > 0 and slots[s] == slots[0]               # a padding copy of the first row leaves the slot alone
+            st = state[slots[s]].reshape(-1)[state_offset:state_offset + d]
+            if not copy:
+                before[cu[s]] = st.to(self.acc)
+            before[cu[s] + 1:cu[s + 1]] = xv[cu[s]:cu[s + 1] - 1]
+            if not copy:
+                st.copy_(x[cu[s + 1] - 1].to(st.dtype))
+        for g in range(mu.shape[0]):
+            out[g] = (xv + (before - xv) * mu[g].to(self.acc)).to(out.dtype)
+        if offsets_out is not None:
+            offsets_out.copy_(torch.arange(mu.shape[0] + 1, dtype=torch.int32) * M)
+
+    def streams(self, x, *, y=None, bias=None, scale=None, mix=None, w_out=None, w_in=None, gain=None, eps=None, next_out=None,
+                rows=None, write_back=True):
+        new = x.to(self.acc)
+        if y is not None:
+            v = y.to(self.acc)
+            if bias is not None:
+                v = v + bias.to(self.acc)
+            if scale is not None:
+                v = v * scale.to(self.acc)
+            new = torch.einsum("st,msd->mtd", mix.to(self.acc), new) + w_out.to(self.acc)[None, :, None] * v[:, None, :]
+            if write_back:
+                x.copy_(new.to(x.dtype))
+        if next_out is not None:
+            u = torch.einsum("s,msd->md", w_in.to(self.acc), new if rows is None else new[rows.long()])
+            if gain is not None:
+                u = u / torch.sqrt(u.pow(2).mean(-1, keepdim=True) + eps) * gain.to(self.acc)
+            next_out.copy_(u.to(next_out.dtype))
+
+    def _scan_segments(self, batch, state, state_offset, heads, dim, vdim, out, token):
+        """Walk every segment; `token(h, t, S)` returns (read-out, new S)."""
+        dim4 = -(-dim // 4) * 4
+        cu, slots = batch.cu_seqlens.tolist(), batch.slots.tolist()
+        for s in range(len(cu) - 1):
+            if s > 0 and slots[s] == slots[0]:                  # a padding copy of the first row
+                out[cu[s]:cu[s + 1]] = 0
+                continue
+            flat = state[slots[s]].reshape(-1)
+            for h in range(heads):
+                st = flat[state_offset + h * vdim * dim4:state_offset + (h + 1) * vdim * dim4].view(vdim, dim4)
+                S = st[:, :dim].T.to(self.acc).clone()
+                for t in range(cu[s], cu[s + 1]):
+                    o, S = token(h, t, S)
+                    out[t, h * vdim:(h + 1) * vdim] = o.to(out.dtype)
+                st[:, :dim] = S.T.to(st.dtype)
+
+    def state_space_scan(self, q, k, v, step, out, batch, state, *, heads, kv_heads, dim, vdim, a_log, dt_bias, skip,
+                         state_offset=0):
+        def token(h, t, S):
+            g = h // (heads // kv_heads)
+            qt = q[0][t, q[1] + g * dim:q[1] + (g + 1) * dim].to(self.acc)
+            kt = k[0][t, k[1] + g * dim:k[1] + (g + 1) * dim].to(self.acc)
+            vt = v[0][t, v[1] + h * vdim:v[1] + (h + 1) * vdim].to(self.acc)
+            dt = torch.nn.functional.softplus(step[0][t, step[1] + h].to(self.acc) + dt_bias[h].to(self.acc), threshold=1e9)
+            S = torch.exp(-torch.exp(a_log[h].to(self.acc)) * dt) * S + dt * torch.outer(kt, vt)
+            return S.T @ qt + skip[h].to(self.acc) * vt, S
+        self._scan_segments(batch, state, state_offset, heads, dim, vdim, out, token)
+
+    def decay_scan(self, r, k, v, w, out, batch, state, *, heads, dim, vdim, w0, u, state_offset=0):
+        w.copy_(torch.exp(-torch.exp(w.to(self.acc) + w0.to(self.acc))).to(w.dtype))
+        uv = u.to(self.acc).reshape(heads, dim)
+
+        def token(h, t, S):
+            rt, kt = (x[0][t, x[1] + h * dim:x[1] + (h + 1) * dim].to(self.acc) for x in (r, k))
+            vt = v[0][t, v[1] + h * vdim:v[1] + (h + 1) * vdim].to(self.acc)
+            o = S.T @ rt + (rt * uv[h] * kt).sum() * vt
+            return o, w[t, h * dim:(h + 1) * dim].to(self.acc)[:, None] * S + torch.outer(kt, vt)
+        self._scan_segments(batch, state, state_offset, heads, dim, vdim, out, token)
 
     # ---- recurrent mixers
     def mlstm_scan(self, proj, out, batch, state, *, heads, dim, vdim, gate_cap, q_scale, columns, i_bias, f_bias, chunked=None):
@@ -176,14 +281,28 @@ class TorchReferenceKernels(KernelSet):
     def _mm(self, x, w):
         return x.to(self.acc) @ w.to(self.acc).T
 
-    def linear(self, x, w, out, *, accumulate=False, row_scale=None, activation=None):
+    def batched_linear(self, x, w, offsets, out):
+        assert offsets.tolist() == [g * x.shape[1] for g in range(x.shape[0] + 1)]
+        for g in range(x.shape[0]):
+            out[g] = self._mm(x[g], w[g]).to(out.dtype)
+
+    def linear(self, x, w, out, *, accumulate=False, row_scale=None, activation=None, bias=None, act_params=None):
         y = self._mm(x, w)
         if row_scale is not None:
             y = y * row_scale.to(self.acc)[:, None]
+        if bias is not None:
+            assert not accumulate
+            y = y + bias.to(self.acc)
         if activation is not None:
-            assert activation in ("relu2", "gelu_tanh") and not accumulate
+            assert activation in ("relu2", "gelu_tanh", "xielu", "tanh") and not accumulate
             if activation == "relu2":
                 y = torch.relu(y) ** 2
+            elif activation == "tanh":
+                y = torch.tanh(y)
+            elif activation == "xielu":
+                a, b = act_params
+                n = torch.clamp(y, max=0)
+                y = torch.where(y > 0, a * y * y, b * (torch.expm1(n) - n)) + 0.5 * y
             else:
                 y = 0.5 * y * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (y + 0.044715 * y ** 3)))
         if accumulate:
@@ -256,7 +375,7 @@ class TorchReferenceKernels(KernelSet):
 
     # ---- attention
     def qk_prepare(self, qkv, q_out, batch, cache, *, num_heads, rotation, qk_norm, temperature,
-                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None):
+                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None, value_rotation=None):
         kv = cache.kv
         nkv, P, hd = kv.shape[2], kv.shape[3], kv.shape[4]
         nq = num_heads
@@ -279,6 +398,9 @@ class TorchReferenceKernels(KernelSet):
             for g in range(nkv):
                 o = other[:, col + g * stride: col + g * stride + vd].to(self.acc)
                 v[:, g, :vd] = (1.0 - lam) * v[:, g, :vd] + lam * o
+
+        if value_rotation is not None:
+            v = self._turn(v, batch.positions, value_rotation, 1.0)
 
         def norm(t, gain):
             t = t * (1.0 / torch.sqrt(t.pow(2).sum(-1, keepdim=True) / (norm_dim or hd) + qk_norm.eps))

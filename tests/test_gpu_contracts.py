@@ -150,7 +150,7 @@ def test_elementwise_entry_points(libs):
                  (1, ptr(table), ptr(toks), None, 4, 16, 10, C.c_float(1.0)), (1, ptr(table), ptr(toks), ptr(h), -1, 16, 10, C.c_float(1.0)),
                  (1, ptr(table), ptr(toks), ptr(h), 4, 0, 10, C.c_float(1.0)), (1, ptr(table), ptr(toks), ptr(h), 4, 16, 0, C.c_float(1.0)),
                  (7, ptr(table), ptr(toks), ptr(h), 4, 16, 10, C.c_float(1.0))):
-        assert lib.spite_embed(*args, None) == BAD_ARG, args
+        assert lib.spite_embed(*args, 1, None) == BAD_ARG, args
     assert untouched(h)
     x = torch.ones((4, 16), dtype=torch.float32, device=DEV)
     gain = torch.ones(16, dtype=torch.float32, device=DEV)
