@@ -14,6 +14,7 @@ Two further workloads print a line of the same kind (they are extra modes; the d
                                          # 8,192, then 256 decode steps at batch 1 and at batch 4
     python bench.py --config mibezen     # the Mibezen design beside Llama 4 at equal layer sizes, measured the same way
     python bench.py --config paposun     # the Paposun design beside a dense Llama 4 at equal layer sizes, measured the same way
+    python bench.py --config zuzadra     # the Zuzadra design beside Paposun at equal layer sizes, measured the same way
     python bench.py --config gapevik     # the Gapevik design beside Llama 4 at equal layer sizes, measured the same way
     python bench.py --config sezazen     # the Sezazen design beside Llama 4 at equal layer sizes (three sizes): prefill
                                          # of 2,048 tokens and decode at batch 1 and 8, each with its roofline fraction
@@ -391,6 +392,32 @@ def gapevik_configs(size, runs=8):
     return gap, llama
 
 
+def zuzadra_configs(size, runs=8):
+    """A Zuzadra model of eight layer runs (two state-space layers, the parallel layer of attention and decaying memory, one
+    more state-space layer, all run twice on one set of weights) with four residual streams, and a Paposun model of eight
+    layers (a matrix memory where Zuzadra has a state space, attention where it has the parallel layer) with the same
+    width, attention heads, feed-forward width and vocabulary, a feed-forward in every layer of both.  A state space has
+    width / 32 heads of 64 with 128 state rows, a decaying memory width / 64 heads of 64, a matrix memory 8 heads of width /
+    16 key rows and width / 8 value columns; the window is longer than the measured contexts."""
+    name, d, nq, nkv, kd, vd, E, top, f, fs, fd, V = size
+    ff = {"kind": "dense", "ff": fd}
+    L = lambda t, m: {"type": t, "mixer": m, "mlp": ff}
+    ssm = {"heads": d // 32, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
+    par = {"left": {"heads": nq, "kv_heads": nkv, "dim": kd, "vdim": vd, "scale": kd ** -0.5, "mask": {"size": 8192},
+                    "rot": {"base": 500000.0, "dims": kd // 2}},
+           "right": {"heads": d // 64, "dim": 64, "rank": 64}, "left_scale": 0.75, "right_scale": 0.6}
+    zuz = {"architecture": "Zuzadra", "vocab": V, "width": d, "max_positions": 8192, "norm": {"eps": 1e-6}, "streams": 4,
+           "loop": {"start": 0, "stop": 4, "times": 2},
+           "layers": [L("mamba2", ssm), L("mamba2", ssm), L("parallel", par), L("mamba2", ssm)]}
+    mem = {"heads": 8, "dim": d // 16, "vdim": d // 8, "gate_cap": 10.0}
+    att = {"heads": nq, "kv_heads": nkv, "dim": kd, "vdim": vd, "scale": kd ** -0.5, "mask": {"size": 8192},
+           "rot": {"base": 500000.0, "dims": kd // 2}}
+    pap = {"architecture": "Paposun", "vocab": V, "width": d, "max_positions": 8192, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+           "logit_scale": 0.5,
+           "layers": [L("mlstm", mem), L("mlstm", mem), L("attention", att), L("mlstm", mem)] * 2}
+    return zuz, pap
+
+
 def design_work(model, T, contexts):
     """(flops of a prompt of T tokens, bytes a decode step over `contexts` must read), from the parts' own sizes
     as the design states them (no padding): every layer run reads its weights once; experts by the tokens' draw."""
@@ -399,6 +426,8 @@ def design_work(model, T, contexts):
     from spite_b200.parts.latent import LatentAttention
     from spite_b200.parts.mlstm import MatrixLstm
     from spite_b200.parts.delta import GatedDelta
+    from spite_b200.parts.parallel import ParallelMixers
+    from spite_b200.parts.statespace import StateSpace
     es, p = 2, model.plan
     flops, nbytes = 2 * p.hidden_size * p.vocab_size, p.vocab_size * p.hidden_size * es
     for j in model.junctions:
@@ -427,6 +456,16 @@ def design_work(model, T, contexts):
             w = d * (2 * m.G * m.kd + 2 * m.H * m.vd + 2 * m.H) + m.H * m.vd * d
             flops += 2 * T * w + 4 * T * m.H * m.kd * m.vd
             nbytes += w * es + len(contexts) * 2 * m.H * m.kd * m.vd * 4
+        elif isinstance(m, StateSpace):
+            # both projections; per token and head the matrix's update and its read-out, two multiply-adds an element
+            w = d * (2 * m.inner + 2 * m.G * m.N + m.H) + m.inner * d
+            flops += 2 * T * w + 4 * T * m.inner * m.N
+            nbytes += w * es + len(contexts) * 2 * m.inner * m.N * 4
+        elif isinstance(m, ParallelMixers):
+            a, b = m.sides["left"], m.sides["right"]
+            w = d * (a.nq * a.kd + a.nkv * (a.kd + a.vd)) + a.nq * a.vd * d + d * (4 * b.n + b.rank) + b.n * b.rank + b.n * d
+            flops += 2 * T * w + 2 * a.nq * (a.kd + a.vd) * T * (T + 1) // 2 + 4 * T * b.n * b.dim
+            nbytes += w * es + sum(c * a.nkv * (a.kd + a.vd) * es for c in contexts) + len(contexts) * 2 * b.n * b.dim * 4
         else:
             shared = getattr(m, "kv_shared", False)
             w = d * (m.nq * m.kd + (0 if shared else m.nkv * (m.kd + m.vd))) + m.nq * m.vd * d + \
@@ -470,7 +509,8 @@ def run_sezazen(args):
     the first size."""
     design = args.config
     configs_of = {"sezazen": design_configs, "mibezen": mibezen_configs, "paposun": paposun_configs,
-                  "gapevik": gapevik_configs}[design]
+                  "gapevik": gapevik_configs, "zuzadra": zuzadra_configs}[design]
+    other = "paposun" if design == "zuzadra" else "llama4"
     import torch
     from spite_b200.config import config_from_dict
     from spite_b200.engine import Engine, Model, StepEntry
@@ -542,13 +582,13 @@ def run_sezazen(args):
     with clocks:
         for size in sizes:
             sez, llama = configs_of(size)
-            out[size[0]] = {name: measure(cfgd) for name, cfgd in ((design, sez), ("llama4", llama))
+            out[size[0]] = {name: measure(cfgd) for name, cfgd in ((design, sez), (other, llama))
                             if args.design in ("both", name)}
     first = next(iter(out[sizes[0][0]].values()))
     key = f"decode_b{args.batch if args.only_decode else 8}"
     line = base_line(f"decode tok/s at batch 8, context 2,048 ({design.capitalize()} design, first size)", first.get(key + "_tok_s", 0.0), "tok/s",
                      steps, warmup, first.get(key + "_ms", 0.0),
-                     {"model": f"{design} beside llama4 at equal layer sizes", "layer_runs": 8, "prefill_tokens": T, "context": C,
+                     {"model": f"{design} beside {other} at equal layer sizes", "layer_runs": 8, "prefill_tokens": T, "context": C,
                       "sizes": {s[0]: dict(zip(("width", "q_heads", "kv_heads", "key_dim", "value_dim", "experts", "top", "expert_ff",
                                                 "shared_ff", "dense_ff", "vocab"), s[1:])) for s in DESIGN_SIZES},
                       "global_batch": 8, "seq_len": C, "page_size": 64, "parallelism": "single-gpu",
@@ -751,8 +791,8 @@ def main(argv=None):
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", choices=["ours", "reference"], default="ours")
-    ap.add_argument("--config", choices=["scout", "maverick", "long", "sezazen", "mibezen", "paposun", "gapevik"], default="scout",
-                    help="scout: the benchmark line; maverick, long, sezazen, mibezen, paposun, gapevik: further workloads, one line each")
+    ap.add_argument("--config", choices=["scout", "maverick", "long", "sezazen", "mibezen", "paposun", "gapevik", "zuzadra"], default="scout",
+                    help="scout: the benchmark line; maverick, long, sezazen, mibezen, paposun, gapevik, zuzadra: further workloads, one line each")
     ap.add_argument("--layers", type=int, default=FULL_LAYERS)
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=8192)
@@ -762,8 +802,8 @@ def main(argv=None):
     ap.add_argument("--only-prefill", action="store_true", help="measure the prefill step only (for profiling)")
     ap.add_argument("--verbose", action="store_true", help="print the single prefill timings to standard error")
     ap.add_argument("--size", default=None, help="--config sezazen: only this set of layer sizes (small, medium, ...)")
-    ap.add_argument("--design", choices=["both", "sezazen", "mibezen", "paposun", "gapevik", "llama4"], default="both",
-                    help="--config sezazen / mibezen / paposun / gapevik: only this design")
+    ap.add_argument("--design", choices=["both", "sezazen", "mibezen", "paposun", "gapevik", "zuzadra", "llama4"], default="both",
+                    help="--config sezazen / mibezen / paposun / gapevik / zuzadra: only this design")
     args = ap.parse_args(argv)
     if args.impl == "reference":
         return run_reference(args)
@@ -776,7 +816,7 @@ def main(argv=None):
     if args.config == "long":
         run_long(args)
         return 0
-    if args.config in ("sezazen", "mibezen", "paposun", "gapevik"):
+    if args.config in ("sezazen", "mibezen", "paposun", "gapevik", "zuzadra"):
         run_sezazen(args)
         return 0
     if args.warmup < 3:

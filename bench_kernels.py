@@ -13,6 +13,7 @@ peak.  Also the small driver that `ncu` captures for the summaries under `profil
     python bench_kernels.py --only gated_less    # experts without a gate (squared ReLU), the junction of a loop,
                                                  # the embedding with learned positions
     python bench_kernels.py --only recurrent     # the matrix memory's scan in prompts and decode steps, the heads' norm
+    python bench_kernels.py --only scan          # the scans of the state space and the decaying memory, streams, token shift, gated norm
     python bench_kernels.py --only delta         # the gated delta rule's scan in prompts and decode steps, the short convolution
                                                  # and gate, the norm behind a sublayer
 
@@ -397,6 +398,82 @@ def main(argv=None):
                 return lambda: ks.cast_rows(h, x)
             nbytes = M * dm * 6
             report("delta", f"cast_rows M={M} d={dm}", timed_rotating(make_cast, max(nbytes, 64 << 20) if M == 8 else nbytes), nbytes=nbytes)
+
+    # ---- the scans of the state space and of the decaying memory, and what stands around them
+    if want("scan"):
+        dm = 2048 if args.small else 4096
+        fma_peak = 148 * 128 * 2 * pk.get("sm_max_mhz", 1965.0) * 1e6
+        for n_seg, n_tok in ((1, 2048), (8, 2048), (1, 1), (8, 1), (64, 1)):
+            M = n_seg * n_tok
+            segs = [Segment(i, i, 0, n_tok, i * n_tok, True) for i in range(n_seg)]
+            batch = build_step_batch(segs, [[0] * n_tok] * n_seg, [[]] * n_seg, [[[0]] * n_seg], dev)
+            for kind, H, kd, vd in (("state_space", dm // 32, 128, 64), ("decay", dm // 64, 64, 64)):
+                G = 1 if kind == "state_space" else H
+                size = H * ks.scan_state_size(kd, vd)
+                def make_scan(M=M, batch=batch, n_seg=n_seg, kind=kind, H=H, kd=kd, vd=vd, G=G, size=size):
+                    out, state = torch.empty((M, H * vd), device=dev), torch.zeros((n_seg, size), device=dev)
+                    hv = torch.zeros(H, device=dev)
+                    if kind == "state_space":
+                        x, step = torch.randn((M, 2 * kd + H * vd), device=dev), torch.randn((M, H), device=dev)
+                        return lambda: ks.state_space_scan((x, kd), (x, 0), (x, 2 * kd), (step, 0), out, batch, state, heads=H, kv_heads=1,
+                                                           dim=kd, vdim=vd, a_log=hv, dt_bias=hv, skip=hv)
+                    r, k, v, w = (torch.randn((M, H * kd), device=dev) for _ in range(4))
+                    u = torch.zeros(H * kd, device=dev)
+                    return lambda: ks.decay_scan((r, 0), (k, 0), (v, 0), w, out, batch, state, heads=H, dim=kd,
+                                                 vdim=vd, w0=u, u=u)
+                nbytes = n_seg * size * 8 + M * ((2 * G * kd + 2 * H * vd + H) * 4 + (0 if kind == "state_space" else H * kd * 4))
+                flops = 4 * M * H * kd * vd
+                name = f"{kind}_scan {n_seg} x {n_tok} tokens, {H} heads of {kd} x {vd}"
+                if args.case and args.case not in name:
+                    continue
+                if n_tok > 1:
+                    ms = timed(make_scan())()
+                    print(json.dumps({"family": "scan", "case": name, "us": round(ms * 1e3, 2), "TFLOPs_fp32": round(flops / ms / 1e9, 2),
+                                      "fp32_fma_frac": round(flops / (ms * 1e-3) / fma_peak, 3), "GBps": round(nbytes / ms / 1e6, 1),
+                                      "peaks": src}), flush=True)
+                else:
+                    report("scan", name, timed_rotating(make_scan, nbytes), nbytes=nbytes)
+            inner = 2 * dm
+            ch, width = inner + 256, 2 * inner + 256 + dm // 32
+            def make_conv(M=M, batch=batch, n_seg=n_seg):
+                x, w, b = torch.randn((M, width), device=dev), torch.randn((ch, 4), device=dev), torch.randn(ch, device=dev)
+                out, state = torch.empty((M, ch), device=dev), torch.zeros((n_seg, 3 * ch), device=dev)
+                return lambda: ks.short_conv(x, w, out, batch, state, channels=ch, activation="silu", bias=b)
+            nbytes = M * ch * 8 + n_seg * 3 * ch * 8
+            report("scan", f"short_conv with a bias {n_seg} x {n_tok} tokens, {ch} channels of 4 taps", timed_rotating(make_conv, max(nbytes, 64 << 20) if n_tok == 1 else nbytes), nbytes=nbytes)
+            def make_shift(M=M, batch=batch, n_seg=n_seg):
+                x, mu = rnd(M, dm), torch.rand((5, dm), device=dev)
+                out, state = torch.empty((5, M, dm), dtype=bf, device=dev), torch.zeros((n_seg, dm), device=dev)
+                return lambda: ks.token_shift(x, mu, out, batch, state)
+            nbytes = M * dm * 12 + n_seg * dm * 8
+            report("scan", f"token_shift {n_seg} x {n_tok} tokens, 5 mixes of {dm}", timed_rotating(make_shift, max(nbytes, 64 << 20) if n_tok == 1 else nbytes), nbytes=nbytes)
+        for M in (8, 2048):
+            inner = 2 * dm
+            def make_norm(M=M):
+                y, z, g = torch.randn((M, inner), device=dev), torch.randn((M, inner), device=dev), torch.ones(inner, device=dev)
+                a = torch.empty((M, inner), dtype=bf, device=dev)
+                return lambda: ks.gate_group_norm(y, z, g, a, groups=1, eps=1e-6)
+            nbytes = M * inner * 10
+            report("scan", f"gate_group_norm M={M}, one part of {inner}", timed_rotating(make_norm, max(nbytes, 64 << 20) if M == 8 else nbytes), nbytes=nbytes)
+            def make_streams(M=M):
+                S = 4
+                x, y = torch.randn((M, S, dm), device=dev), torch.randn((M, dm), device=dev)
+                mix, wo, wi = torch.eye(S, device=dev).contiguous(), torch.zeros(S, device=dev), torch.ones(S, device=dev)
+                sc, b, g = torch.ones(dm, device=dev), torch.zeros(dm, device=dev), torch.ones(dm, device=dev)
+                a = torch.empty((M, dm), dtype=bf, device=dev)
+                return lambda: ks.streams(x, y=y, bias=b, scale=sc, mix=mix, w_out=wo, w_in=wi, gain=g, eps=1e-6, next_out=a)
+            nbytes = M * dm * (4 * 8 + 4 + 2)
+            report("scan", f"streams M={M}, four of {dm}, output laid in and next norm", timed_rotating(make_streams, max(nbytes, 64 << 20) if M == 8 else nbytes), nbytes=nbytes)
+            segs = [Segment(0, 0, 0, M, 0, True)]
+            batch = build_step_batch(segs, [[0] * M], [[]], [[[0]]], dev)
+            from spite_b200.parts import Rotation
+            vrot = Rotation(torch.tensor([500000.0 ** (-2.0 * i / 128) for i in range(64)], dtype=torch.float32, device=dev), "halves", 128)
+            def make_turn(M=M, batch=batch):
+                h = dm // 128
+                x, o = rnd(M, dm), torch.empty((M, 2 * dm), dtype=bf, device=dev)
+                return lambda: ks.turn_heads(x, o, batch, heads=h, size=128, rotation=vrot, scale=0.5)
+            nbytes = M * dm * 4
+            report("scan", f"turn_heads M={M}, {dm // 128} heads of 128", timed_rotating(make_turn, max(nbytes, 64 << 20) if M == 8 else nbytes), nbytes=nbytes)
 
     # ---- the small kernels of a decode step
     if want("small"):

@@ -277,8 +277,8 @@ class ZuzadraConfig:
                     "value_dim": a.vdim, "softmax_scale": a.scale,
                     "window": ("sliding", a.window) if a.window is not None else ("full", 0),
                     "qk_norm_eps": c.norm_eps, "qk_norm_gain": True, "qk_norm_before_rotation": True,
-                    "position": PartSpec("rotary_halves", {"rotary_dim": a.rot_dims, "theta": a.rot_base}),
-                    "value_rotation": PartSpec("rotary_halves", {"rotary_dim": a.vdim, "theta": a.rot_base})})
+                    "position": PartSpec("rotary_halves", {"rotary_dim": a.rot_dims, "theta": a.rot_base, "exact_angles": True}),
+                    "value_rotation": PartSpec("rotary_halves", {"rotary_dim": a.vdim, "theta": a.rot_base, "exact_angles": True})})
                 right = PartSpec("decay_memory", {"hidden_size": c.width, "num_heads": b.heads, "head_dim": b.dim,
                                                   "decay_rank": b.decay_rank, "norm_eps": c.norm_eps})
                 mixer = PartSpec("parallel_mixers", {"hidden_size": c.width, "left": left, "right": right,

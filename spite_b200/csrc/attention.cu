@@ -67,9 +67,9 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkPrepareParams p
     // sincosf of an angle of thousands of radians is the most expensive thing here) and its warps read them
     __shared__ float cs_s[128], sn_s[128], vc_s[128], vs_s[128];
     const int vrot = p.v_inv_freq ? p.v_rotary_dim : 0;
-    for (int i = threadIdx.x; 2 * i < vrot; i += blockDim.x) sincosf((float)pos * p.v_inv_freq[i], &vs_s[i], &vc_s[i]);
+    for (int i = threadIdx.x; 2 * i < vrot; i += blockDim.x) turn_of((float)pos, p.v_inv_freq, p.v_inv_freq_low, i, vc_s[i], vs_s[i]);
     for (int i = threadIdx.x; 2 * i < rot; i += blockDim.x) {
-        sincosf((float)pos * p.inv_freq[i], &sn_s[i], &cs_s[i]);
+        turn_of((float)pos, p.inv_freq, p.inv_freq_low, i, cs_s[i], sn_s[i]);
         sn_s[i] *= p.rot_amplitude; cs_s[i] *= p.rot_amplitude;
     }
     __syncthreads();
@@ -189,14 +189,14 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkPrepareParams p
 template <typename T>
 __global__ void __launch_bounds__(128) turn_heads_kernel(const T* __restrict__ x, T* __restrict__ out, long long out_stride,
                                                          const int* __restrict__ positions, const float* __restrict__ inv_freq,
-                                                         int rot, int pairing, int heads, int head_dim, int size, float scale,
+                                                         const float* __restrict__ inv_freq_low, int rot, int pairing, int heads, int head_dim, int size, float scale,
                                                          int heads_per_block) {
     pdl_wait();
     pdl_launch_dependents();
     __shared__ float cs_s[128], sn_s[128];
     const int t = blockIdx.x;
     for (int i = threadIdx.x; 2 * i < rot; i += blockDim.x) {
-        sincosf((float)positions[t] * inv_freq[i], &sn_s[i], &cs_s[i]);
+        turn_of((float)positions[t], inv_freq, inv_freq_low, i, cs_s[i], sn_s[i]);
     }
     __syncthreads();
     const int h0 = blockIdx.y * heads_per_block, h1 = min(heads, h0 + heads_per_block);
@@ -349,7 +349,7 @@ SPITE_API int spite_qk_prepare(int dtype, const QkPrepareParams* given, const St
 }
 
 SPITE_API int spite_turn_heads(int dtype, const void* x, void* out, long long out_stride, const int* positions,
-                               const float* inv_freq, int rotary_dim, int pairing, int n_tokens, int heads, int head_dim,
+                               const float* inv_freq, const float* inv_freq_low, int rotary_dim, int pairing, int n_tokens, int heads, int head_dim,
                                int size, float scale, void* stream) {
     if (!x || !out || n_tokens < 0 || heads < 1 || size < 1 || head_dim < size || !(scale == scale)) return SPITE_BAD_ARG;
     if (out_stride < (long long)heads * size) return SPITE_BAD_ARG;
@@ -364,11 +364,11 @@ SPITE_API int spite_turn_heads(int dtype, const void* x, void* out, long long ou
     const int rot = inv_freq ? rotary_dim : 0;
     cudaStream_t st = (cudaStream_t)stream;
     if (dtype == SPITE_DT_F32)
-        SPITE_LAUNCH(turn_heads_kernel<float>, grid, 128, 0, st, (const float*)x, (float*)out, out_stride, positions, inv_freq, rot,
+        SPITE_LAUNCH(turn_heads_kernel<float>, grid, 128, 0, st, (const float*)x, (float*)out, out_stride, positions, inv_freq, inv_freq_low, rot,
                      pairing, heads, head_dim, size, scale, hpb);
     else
         SPITE_LAUNCH(turn_heads_kernel<__nv_bfloat16>, grid, 128, 0, st, (const __nv_bfloat16*)x, (__nv_bfloat16*)out, out_stride,
-                     positions, inv_freq, rot, pairing, heads, head_dim, size, scale, hpb);
+                     positions, inv_freq, inv_freq_low, rot, pairing, heads, head_dim, size, scale, hpb);
     return spite_launch_status();
 }
 

@@ -68,7 +68,23 @@ struct QkPrepareParams {
     const float* v_inv_freq;
     int v_rotary_dim;
     int v_pairing;
+    // what inv_freq and v_inv_freq lost when they were rounded to float32 (null: the angle is the rounded product)
+    const float* inv_freq_low;
+    const float* v_inv_freq_low;
 };
+
+// cos and sin of pos * (freq + low).  With `low` the product's own rounding error and the frequency's are put back to first
+// order, so that the angle of a far position is as exact as that of a near one; without it the float32 product counts.
+__device__ __forceinline__ void turn_of(float pos, const float* freq, const float* low, int i, float& c, float& s) {
+    const float f = freq[i], a = pos * f;
+    sincosf(a, &s, &c);
+    if (low) {
+        const float e = fmaf(pos, f, -a) + pos * low[i];
+        const float c0 = c;
+        c = fmaf(-e, s, c);
+        s = fmaf(e, c0, s);
+    }
+}
 
 struct AttentionParams {
     const void* q;              // [tokens, nq * head_dim]

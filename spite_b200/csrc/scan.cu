@@ -9,12 +9,13 @@
 // S is [dim keys, vdim values], zeros at the start of a sequence.  Everything is float32.
 //
 // Unlike a delta rule, what a token writes does not depend on the state, so the walk is bound by what its warps can issue,
-// not by one token's chain.  A warp is LR lanes along the keys times 32 / LR lanes along the values; a lane holds RP = 4 RPV
-// key rows (as packed pairs, for the two-at-a-time multiply-adds of sm_100) of CC value columns.  TB = LR / CC tokens form a
-// batch: their inputs arrive in one stage of a shared-memory ring by asynchronous copies two batches ahead, one barrier a
-// batch, and their partial read-outs (TB * CC a lane) are summed over the LR lanes by a halving exchange that leaves every
-// lane one finished number.  The order of the sums depends on the head's sizes alone, so the result does not depend on
-// how a sequence was cut into steps.
+// not by one token's chain.  A warp is LR lanes along the keys times 32 / LR lanes along the values; a lane holds 4 RPV
+// key rows (as packed pairs, for the two-at-a-time multiply-adds of sm_100) of CC value columns.  TB tokens form a batch:
+// one more warp of the block brings their inputs into one stage of a shared-memory ring by asynchronous copies two batches
+// ahead (so that the walking warps spend nothing on it), one barrier stands between two batches, and the batch's TB * CC
+// partial read-outs a lane are summed over the LR lanes by a halving exchange that leaves every lane TB * CC / LR finished
+// numbers.  The order of the sums depends on the head's sizes alone, so the result does not depend on how a sequence was
+// cut into steps.
 //
 // The slot holds S transposed: value column j's keys are contiguous, [vdim, dim4] with dim4 = dim rounded up to a multiple
 // of four (the padding stays zero), so that a lane's rows are whole 16-byte groups and a warp's loads whole lines.
@@ -66,33 +67,64 @@ template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.as
 
 constexpr int RING = 3;
 
-template <int LR, int RPV, int CC, bool CH>
+constexpr int MAX_WARPS = 4;                              // walking warps a block
+
+template <int LR, int RPV, int CC, int TB, bool CH>
 struct Shape {
-    static constexpr int TB = LR / CC;                    // tokens a batch
     static constexpr int DP = LR * RPV * 4;               // key rows a warp covers
     static constexpr int WC = 32 / LR * CC;               // value columns a warp covers
     static constexpr int ROWS = CH ? 3 : 2;               // q, k (and w) of a token
-    static __host__ __device__ constexpr int token_floats(int warps) { return ROWS * DP + ((WC * warps + 3) & ~3) + 4; }
+    static constexpr int TOKEN = ROWS * DP + WC * MAX_WARPS + 4;      // floats of a token's stage
+    static constexpr int KEEP = TB * CC / LR;             // finished numbers a lane
+    static_assert(KEEP >= 1 && KEEP * LR == TB * CC && TOKEN % 4 == 0, "a batch's read-outs must fill the lanes");
 };
 
-// grid (ceil(vdim / (WC * warps)), heads, segments)
-template <int LR, int RPV, int CC, bool CH>
-__global__ void __launch_bounds__(128) scan_kernel(const ScanParams p, const int wide) {
-    using SH = Shape<LR, RPV, CC, CH>;
-    constexpr int TB = SH::TB, DP = SH::DP, WC = SH::WC, NP = RPV * 2;
+// All threads of the block (the number is a multiple of 32).
+__device__ __forceinline__ void block_barrier(int threads) { asm volatile("bar.sync 1, %0;" ::"r"(threads) : "memory"); }
+
+// The copies of one batch (tokens tb .. tb + n - 1) into its stage, by one warp.
+template <typename SH>
+__device__ __forceinline__ void bring_batch(const ScanParams& p, const float* qp, const float* kp, const float* wp, const float* vp,
+                                            const float* sp, int n_cols, int tb, int n, float* stage, int lane, int wide) {
+    constexpr bool CH = SH::ROWS == 3;
+    constexpr int V = SH::ROWS * SH::DP, TOKEN = SH::TOKEN;
+    const int u = wide ? 4 : 1, du = p.dim / u, vu = n_cols / u;         // copies of 16 or of 4 bytes
+    const int rows = SH::ROWS * du, per = rows + vu + 2;
+    for (int e = lane; e < per; e += 32) {
+        const float* src;
+        long long stride;
+        int dst;
+        if (e < du) { src = qp + u * e; stride = p.q_stride; dst = u * e; }
+        else if (e < 2 * du) { src = kp + u * (e - du); stride = p.k_stride; dst = SH::DP + u * (e - du); }
+        else if (CH && e < 3 * du) { src = wp + u * (e - 2 * du); stride = p.w_stride; dst = 2 * SH::DP + u * (e - 2 * du); }
+        else if (e < rows + vu) { src = vp + u * (e - rows); stride = p.v_stride; dst = V + u * (e - rows); }
+        else { src = sp + (e - rows - vu); stride = 2 * p.heads; dst = TOKEN - 4 + (e - rows - vu); }
+        src += (long long)tb * stride;
+        float* d = stage + dst;
+        if (wide && e < rows + vu) {
+            for (int tt = 0; tt < n; ++tt, src += stride, d += TOKEN) cp_async16(d, src);
+        } else {
+            for (int tt = 0; tt < n; ++tt, src += stride, d += TOKEN) cp_async4(d, src);
+        }
+    }
+}
+
+// grid (ceil(vdim / (WC * warps)), heads, segments), block 32 * (warps + 1)
+template <int LR, int RPV, int CC, int TB, bool CH>
+__global__ void __launch_bounds__(32 * (MAX_WARPS + 1)) scan_kernel(const ScanParams p, const int wide) {
+    using SH = Shape<LR, RPV, CC, TB, CH>;
+    constexpr int DP = SH::DP, WC = SH::WC, NP = RPV * 2, TOKEN = SH::TOKEN, V = SH::ROWS * DP;
     extern __shared__ __align__(16) float ring[];
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-    const int r = lane % LR, cl = lane / LR;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = (blockDim.x >> 5) - 1;
     const int seg = blockIdx.z, head = blockIdx.y;
     const int dim = p.dim, vdim = p.vdim, dim4 = (dim + 3) & ~3;
     const int BC = WC * warps, c0 = blockIdx.x * BC;
-    const int tok_floats = SH::token_floats(warps);
-    // rows beyond dim stay zero in every stage (q and k; a decay there multiplies zeros)
+    // rows beyond dim stay zero in every stage (a decay there multiplies zeros)
     if (DP > dim) {
         const int gap = DP - dim;
         for (int e = threadIdx.x; e < RING * TB * SH::ROWS * gap; e += blockDim.x) {
-            const int slot = e / (SH::ROWS * gap), i = e % (SH::ROWS * gap);
-            ring[(size_t)slot * tok_floats + (i / gap) * DP + dim + i % gap] = 0.f;
+            const int t = e / (SH::ROWS * gap), i = e % (SH::ROWS * gap);
+            ring[t * TOKEN + (i / gap) * DP + dim + i % gap] = 0.f;
         }
     }
     pdl_wait();
@@ -104,61 +136,35 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p, const int
             if (c0 + e % BC < vdim) p.out[(size_t)(t0 + e / BC) * p.out_stride + (size_t)head * vdim + c0 + e % BC] = 0.f;
         return;
     }
-    const int kvh = head / (p.heads / p.kv_heads);
-    const float* qp = p.q + (size_t)kvh * dim;
-    const float* kp = p.k + (size_t)kvh * dim;
-    const float* vp = p.v + (size_t)head * vdim + c0;
-    const float* wp = CH ? p.w + (size_t)head * dim : nullptr;
-    const float* sp = p.scalars + 2 * head;
-
     const int n_cols = min(BC, vdim - c0);
     const int n_batches = (t1 - t0 + TB - 1) / TB;
-    auto issue = [&](int b) {
-        const int tb = t0 + b * TB, n = min(TB, t1 - tb);
-        float* stage = ring + (size_t)(b % RING) * TB * tok_floats;
-        if (b < n_batches) {
-            if (wide) {                                   // whole 16-byte groups everywhere
-                const int d4 = dim >> 2, v4 = n_cols >> 2, per = SH::ROWS * d4 + v4 + 1;
-                for (int e = threadIdx.x; e < per; e += blockDim.x) {
-                    const float* src;
-                    long long stride;
-                    int dst;
-                    if (e < d4) { src = qp + 4 * e; stride = p.q_stride; dst = 4 * e; }
-                    else if (e < 2 * d4) { src = kp + 4 * (e - d4); stride = p.k_stride; dst = DP + 4 * (e - d4); }
-                    else if (CH && e < 3 * d4) { src = wp + 4 * (e - 2 * d4); stride = p.w_stride; dst = 2 * DP + 4 * (e - 2 * d4); }
-                    else if (e < SH::ROWS * d4 + v4) { src = vp + 4 * (e - SH::ROWS * d4); stride = p.v_stride; dst = SH::ROWS * DP + 4 * (e - SH::ROWS * d4); }
-                    else { src = sp; stride = 2 * p.heads; dst = tok_floats - 4; }
-                    src += (size_t)tb * stride;
-                    float* d = stage + dst;
-                    if (e == per - 1) {
-                        for (int tt = 0; tt < n; ++tt, src += stride, d += tok_floats) { cp_async4(d, src); cp_async4(d + 1, src + 1); }
-                    } else {
-                        for (int tt = 0; tt < n; ++tt, src += stride, d += tok_floats) cp_async16(d, src);
-                    }
-                }
-            } else {
-                const int per = SH::ROWS * dim + n_cols + 2;
-                for (int e = threadIdx.x; e < per; e += blockDim.x) {
-                    const float* src;
-                    long long stride;
-                    int dst;
-                    if (e < dim) { src = qp + e; stride = p.q_stride; dst = e; }
-                    else if (e < 2 * dim) { src = kp + e - dim; stride = p.k_stride; dst = DP + e - dim; }
-                    else if (CH && e < 3 * dim) { src = wp + e - 2 * dim; stride = p.w_stride; dst = 2 * DP + e - 2 * dim; }
-                    else if (e < SH::ROWS * dim + n_cols) { src = vp + e - SH::ROWS * dim; stride = p.v_stride; dst = SH::ROWS * DP + e - SH::ROWS * dim; }
-                    else { const int i = e - SH::ROWS * dim - n_cols; src = sp + i; stride = 2 * p.heads; dst = tok_floats - 4 + i; }
-                    src += (size_t)tb * stride;
-                    float* d = stage + dst;
-                    for (int tt = 0; tt < n; ++tt, src += stride, d += tok_floats) cp_async4(d, src);
-                }
-            }
-        }
-        cp_commit();
-    };
+
+    if (warp == warps) {                                  // the warp that brings the inputs
+        const int kvh = head / (p.heads / p.kv_heads);
+        const float* qp = p.q + (size_t)kvh * dim;
+        const float* kp = p.k + (size_t)kvh * dim;
+        const float* vp = p.v + (size_t)head * vdim + c0;
+        const float* wp = CH ? p.w + (size_t)head * dim : nullptr;
+        const float* sp = p.scalars + 2 * head;
+        auto bring = [&](int b) {
+            if (b < n_batches)
+                bring_batch<SH>(p, qp, kp, wp, vp, sp, n_cols, t0 + b * TB, min(TB, t1 - t0 - b * TB), ring + (b % RING) * TB * TOKEN, lane, wide);
+            cp_commit();
+        };
 #pragma unroll 1
-    for (int b = 0; b < RING - 1; ++b) issue(b);
+        for (int b = 0; b < RING - 1; ++b) bring(b);
+#pragma unroll 1
+        for (int b = 0; b < n_batches; ++b) {
+            cp_wait<RING - 2>();
+            block_barrier(blockDim.x);                    // batch b has landed, and every warp is done with batch b - 1
+            bring(b + RING - 1);                          // (into the stage that batch b - 1 had)
+        }
+        cp_wait<0>();
+        return;
+    }
 
     // the state: value column j = c0 + warp * WC + cl * CC + c, key rows 4 (r + LR i) .. + 3
+    const int r = lane % LR, cl = lane / LR;
     float* st = p.state + (size_t)slot * p.slot_stride + (size_t)head * vdim * dim4;
     const int j0 = warp * WC + cl * CC;                   // within the block's columns
     f2 S[NP][CC];
@@ -173,7 +179,7 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p, const int
         }
 
     const float skip = p.skip ? p.skip[head] : 0.f;
-    auto token = [&](const float* in, float* o) {
+    auto token = [&](const float* in, float* o) {         // in: the token's stage
         f2 q[NP], k[NP], w[CH ? NP : 1];
 #pragma unroll
         for (int i = 0; i < RPV; ++i) {
@@ -186,12 +192,18 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p, const int
             }
         }
         f2 decay = 0;
-        float dt = 1.f;
-        if constexpr (!CH) { const float2 s = *(const float2*)(in + tok_floats - 4); decay = pack2(s.x, s.x); dt = s.y; }
+        float v[CC];
+        if constexpr (CC == 4) { const float4 f = *(const float4*)(in + V + j0); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+        else { const float2 f = *(const float2*)(in + V + j0); v[0] = f.x; v[1] = f.y; }
+        if constexpr (!CH) {
+            const float2 s = *(const float2*)(in + TOKEN - 4);
+            decay = pack2(s.x, s.x);
+#pragma unroll
+            for (int c = 0; c < CC; ++c) v[c] *= s.y;
+        }
 #pragma unroll
         for (int c = 0; c < CC; ++c) {
-            const float v = CH ? in[SH::ROWS * DP + j0 + c] : dt * in[SH::ROWS * DP + j0 + c];
-            const f2 v2 = pack2(v, v);
+            const f2 v2 = pack2(v[c], v[c]);
             f2 acc = 0;
 #pragma unroll
             for (int i = 0; i < NP; ++i) {
@@ -209,44 +221,46 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p, const int
         }
     };
 
+    float* out = p.out + (size_t)t0 * p.out_stride + (size_t)head * vdim + c0 + j0;
+    int stage = 0;
 #pragma unroll 1
-    for (int b = 0; b < n_batches; ++b) {
-        cp_wait<RING - 2>();
-        __syncthreads();                                  // batch b has landed, and every thread is done with batch b - 1
-        issue(b + RING - 1);                              // (into the stage that batch b - 1 had)
-        const float* in = ring + (size_t)(b % RING) * TB * tok_floats;
-        const int tb = t0 + b * TB, n = min(TB, t1 - tb);
+    for (int left = t1 - t0; left > 0; left -= TB) {
+        block_barrier(blockDim.x);
+        const float* in = ring + stage * (TB * TOKEN);
+        stage = stage + 1 == RING ? 0 : stage + 1;
         float o[TB * CC];
-        if (n == TB) {
+        if (left >= TB) {
 #pragma unroll
-            for (int tt = 0; tt < TB; ++tt) token(in + (size_t)tt * tok_floats, o + tt * CC);
+            for (int tt = 0; tt < TB; ++tt) token(in + tt * TOKEN, o + tt * CC);
         } else {
 #pragma unroll
             for (int tt = 0; tt < TB; ++tt) {
-                if (tt < n) token(in + (size_t)tt * tok_floats, o + tt * CC);
+                if (tt < left) token(in + tt * TOKEN, o + tt * CC);
                 else
 #pragma unroll
                     for (int c = 0; c < CC; ++c) o[tt * CC + c] = 0.f;
             }
         }
-        // sums over the LR lanes of the keys; lane r keeps number r = (token r / CC, column r % CC)
+        // sums over the LR lanes of the keys; lane r keeps the numbers r * KEEP .. (number n: token n / CC, column n % CC)
 #pragma unroll
         for (int h = LR / 2; h >= 1; h >>= 1) {
             const bool up = (r & h) != 0;
 #pragma unroll
-            for (int i = 0; i < h; ++i) {
-                const float give = up ? o[i] : o[i + h], keep = up ? o[i + h] : o[i];
+            for (int i = 0; i < h * SH::KEEP; ++i) {
+                const float give = up ? o[i] : o[i + h * SH::KEEP], keep = up ? o[i + h * SH::KEEP] : o[i];
                 o[i] = keep + __shfl_xor_sync(0xffffffffu, give, h);
             }
         }
-        const int tt = r / CC, j = j0 + r % CC;
-        if (tt < n && j < n_cols) {
-            const float* tok = in + (size_t)tt * tok_floats;
-            const float v = tok[SH::ROWS * DP + j];
-            p.out[(size_t)(tb + tt) * p.out_stride + (size_t)head * vdim + c0 + j] = fmaf(CH ? tok[tok_floats - 4] : skip, v, o[0]);
+#pragma unroll
+        for (int i = 0; i < SH::KEEP; ++i) {
+            const int num = r * SH::KEEP + i, tt = num / CC, c = num % CC;
+            if (tt < left && j0 + c < n_cols) {
+                const float* tok = in + tt * TOKEN;
+                out[(long long)tt * p.out_stride + c] = fmaf(CH ? tok[TOKEN - 4] : skip, tok[V + j0 + c], o[i]);
+            }
         }
+        out += TB * p.out_stride;
     }
-    cp_wait<0>();
 #pragma unroll
     for (int c = 0; c < CC; ++c)
 #pragma unroll
@@ -302,22 +316,22 @@ __global__ void __launch_bounds__(128) memory_gates_kernel(float* __restrict__ w
     if (lane == 0) *(float2*)(scalars + 2 * row) = make_float2(s, 0.f);
 }
 
-template <int LR, int RPV, int CC, bool CH>
+template <int LR, int RPV, int CC, int TB, bool CH>
 int launch_scan(const ScanParams& p, int wide, cudaStream_t st) {
-    using SH = Shape<LR, RPV, CC, CH>;
-    // four warps a block, fewer where a step has so few (segment, head) pairs that more and smaller blocks spread better
-    int warps = 4;
+    using SH = Shape<LR, RPV, CC, TB, CH>;
+    // four walking warps a block, fewer where a step has so few (segment, head) pairs that more and smaller blocks spread better
+    int warps = MAX_WARPS;
     while (warps > 1 && ((long long)((p.vdim + SH::WC * warps - 1) / (SH::WC * warps)) * p.heads * p.n_segments < 148 ||
                          SH::WC * (warps / 2) >= p.vdim)) warps /= 2;
-    const size_t bytes = (size_t)RING * SH::TB * SH::token_floats(warps) * sizeof(float);
-    auto kernel = scan_kernel<LR, RPV, CC, CH>;
+    const size_t bytes = (size_t)RING * TB * SH::TOKEN * sizeof(float);
+    auto kernel = scan_kernel<LR, RPV, CC, TB, CH>;
     if (bytes > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess)
         return SPITE_LAUNCH_FAILED;
     dim3 grid((p.vdim + SH::WC * warps - 1) / (SH::WC * warps), p.heads, p.n_segments);
     // A step of single tokens is launched as a programmatic dependent; a longer walk in the ordinary way: started early, its
     // blocks would take the multiprocessors that the kernel before frees first, several to one, for the whole walk.
-    if (p.n_tokens == p.n_segments) SPITE_LAUNCH(kernel, grid, 32 * warps, bytes, st, p, wide);
-    else kernel<<<grid, 32 * warps, bytes, st>>>(p, wide);
+    if (p.n_tokens == p.n_segments) SPITE_LAUNCH(kernel, grid, 32 * (warps + 1), bytes, st, p, wide);
+    else kernel<<<grid, 32 * (warps + 1), bytes, st>>>(p, wide);
     return spite_launch_status();
 }
 
@@ -326,11 +340,11 @@ int choose_scan(const ScanParams& p, cudaStream_t st) {
     const auto al = [](const void* x) { return ((uintptr_t)x & 15) == 0; };
     const int wide = p.dim % 4 == 0 && p.vdim % 4 == 0 && p.q_stride % 4 == 0 && p.k_stride % 4 == 0 && p.v_stride % 4 == 0 &&
                      al(p.q) && al(p.k) && al(p.v) && (!CH || (p.w_stride % 4 == 0 && al(p.w)));
-    if (p.dim <= 32) return launch_scan<8, 1, 2, CH>(p, wide, st);
-    if (p.dim <= 64) return launch_scan<8, 2, 2, CH>(p, wide, st);
-    if (p.dim <= 128) return launch_scan<16, 2, 2, CH>(p, wide, st);
-    if (p.dim <= 256) return launch_scan<16, 4, 2, CH>(p, wide, st);
-    return launch_scan<32, 4, 4, CH>(p, wide, st);
+    if (p.dim <= 32) return launch_scan<8, 1, 2, 8, CH>(p, wide, st);
+    if (p.dim <= 64) return launch_scan<8, 2, 2, 8, CH>(p, wide, st);
+    if (p.dim <= 128) return launch_scan<8, 4, 2, 8, CH>(p, wide, st);
+    if (p.dim <= 256) return launch_scan<16, 4, 2, 8, CH>(p, wide, st);
+    return launch_scan<32, 4, 4, 8, CH>(p, wide, st);
 }
 
 int check_scan(const ScanParams* p) {

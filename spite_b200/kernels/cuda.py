@@ -53,7 +53,8 @@ class QkPrepareParams(C.Structure):
                 ("v_other", C.c_void_p), ("v_other_stride", C.c_longlong), ("v_other_head", C.c_int),
                 ("v_mix_dim", C.c_int), ("v_mix", C.c_float), ("gates_out", C.c_void_p),
                 ("bias", C.c_void_p), ("q_only", C.c_int), ("norm_dim", C.c_int),
-                ("v_inv_freq", C.c_void_p), ("v_rotary_dim", C.c_int), ("v_pairing", C.c_int)]
+                ("v_inv_freq", C.c_void_p), ("v_rotary_dim", C.c_int), ("v_pairing", C.c_int),
+                ("inv_freq_low", C.c_void_p), ("v_inv_freq_low", C.c_void_p)]
 
 
 class AttentionParams(C.Structure):
@@ -873,10 +874,12 @@ class CudaKernels(KernelSet):
             rotary_dim = int(rotation.rotary_dim or head_dim)
             if inv_freq.numel() != rotary_dim // 2:
                 raise KernelError(f"qk_prepare: {inv_freq.numel()} frequencies for {rotary_dim} rotating elements")
-        v_freq, v_dims, v_pairing = None, 0, 0
+        v_freq, v_dims, v_pairing, v_low = None, 0, 0, None
+        low = self._freq_low(rotation)
         if value_rotation is not None:
             f = self._t(value_rotation.inv_freq, torch.float32, "inv_freq")
             v_freq, v_dims, v_pairing = f.data_ptr(), 2 * f.numel(), self._PAIRING[value_rotation.pairing]
+            v_low = self._freq_low(value_rotation)
             if value_rotation.amplitude != 1.0 or (value_rotation.rotary_dim or v_dims) != v_dims:
                 raise KernelError("qk_prepare: values turn by a pure rotation")
         eps, before, q_gain, k_gain = 0.0, 0, None, None
@@ -894,13 +897,21 @@ class CudaKernels(KernelSet):
                             write_cache=int(cache.write), qkv_stride=qkv.shape[1], rot_amplitude=amplitude,
                             v_other=v_other, v_other_stride=v_stride, v_other_head=int(v_head), v_mix_dim=int(v_dim),
                             v_mix=float(v_lam), gates_out=_ptr(gates_out), bias=_ptr(bias), q_only=int(bool(q_only)),
-                            norm_dim=int(norm_dim or 0), v_inv_freq=v_freq, v_rotary_dim=v_dims, v_pairing=v_pairing)
+                            norm_dim=int(norm_dim or 0), v_inv_freq=v_freq, v_rotary_dim=v_dims, v_pairing=v_pairing,
+                            inv_freq_low=low, v_inv_freq_low=v_low)
         b, c = self._step_tokens(batch, cache.group), self._paged(cache)
         st = self._lib("attention").spite_qk_prepare(self._dt, C.byref(p), C.byref(b), C.byref(c), self._stream())
         self._count("attention", 1)
         _check(st, "qk_prepare")
 
     _PAIRING = {"neighbours": 0, "halves": 1}
+
+    def _freq_low(self, rotation):
+        if rotation is None or rotation.inv_freq_low is None:
+            return None
+        if self._t(rotation.inv_freq_low, torch.float32, "inv_freq_low").numel() != rotation.inv_freq.numel():
+            raise KernelError("a rotation's inv_freq_low must have one element per frequency")
+        return rotation.inv_freq_low.data_ptr()
 
     def turn_heads(self, x, out, batch, *, heads, size, rotation=None, scale=1.0, out_column=0):
         self._t(x, self.dtype, "x"); self._t(out, self.dtype, "out")
@@ -916,7 +927,7 @@ class CudaKernels(KernelSet):
                 raise KernelError("turn_heads: heads turn back by a pure rotation")
         st = self._lib("attention").spite_turn_heads(
             self._dt, C.c_void_p(x.data_ptr()), C.c_void_p(o_ptr), C.c_longlong(out.shape[1]),
-            C.c_void_p(batch.positions.data_ptr()), C.c_void_p(_ptr(freq)), int(dims), pairing, M, int(heads),
+            C.c_void_p(batch.positions.data_ptr()), C.c_void_p(_ptr(freq)), C.c_void_p(self._freq_low(rotation)), int(dims), pairing, M, int(heads),
             x.shape[1] // heads, int(size), C.c_float(scale), self._stream())
         self._count("attention", 1)
         _check(st, "turn_heads")

@@ -153,6 +153,7 @@ class Rotation:
     pairing: str = "neighbours"
     rotary_dim: Optional[int] = None
     amplitude: float = 1.0
+    inv_freq_low: Optional[torch.Tensor] = None     # what inv_freq lost to float32: angles of far positions stay exact
 
     def __post_init__(self):
         if self.pairing not in ("neighbours", "halves"):

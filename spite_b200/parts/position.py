@@ -113,10 +113,12 @@ class RotaryYarn(PositionEncoding):
 class RotaryHalves(PositionEncoding):
     """Rotation of the first `rotary_dim` elements of every head of q and k, element i paired with element
     i + rotary_dim / 2; the other elements pass unchanged.  f_i = theta^(-2i / rotary_dim), optionally rescaled by
-    wavelength as `rotary_frequencies` describes, with `scaling` = {factor, low, high, original}."""
+    wavelength as `rotary_frequencies` describes, with `scaling` = {factor, low, high, original}.  `exact_angles`: the
+    frequencies keep what float32 takes from them, and the kernels put it and the product's rounding back (the angle of
+    position 100,000 is then as exact as that of position 1)."""
     graph_safe = True
 
-    def __init__(self, ctx, rotary_dim: int, theta: float, scaling: dict | None = None):
+    def __init__(self, ctx, rotary_dim: int, theta: float, scaling: dict | None = None, exact_angles: bool = False):
         super().__init__(ctx)
         if rotary_dim % 2 or rotary_dim < 2:
             raise ConfigError("a rotation needs an even number of elements")
@@ -127,8 +129,9 @@ class RotaryHalves(PositionEncoding):
             scaling = {"factor": scaling["factor"], "low_freq_factor": scaling["low"], "high_freq_factor": scaling["high"],
                        "original_max_position_embeddings": scaling["original"]}
         f = rotary_frequencies(int(rotary_dim), float(theta), scaling)
-        self._rotation = Rotation(torch.tensor(f, dtype=torch.float64).to(torch.float32).to(ctx.device), "halves",
-                                  int(rotary_dim))
+        exact = torch.tensor(f, dtype=torch.float64)
+        low = (exact - exact.to(torch.float32).double()).to(torch.float32).to(ctx.device) if exact_angles else None
+        self._rotation = Rotation(exact.to(torch.float32).to(ctx.device), "halves", int(rotary_dim), inv_freq_low=low)
 
     def rotation(self):
         return self._rotation
