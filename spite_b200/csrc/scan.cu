@@ -11,8 +11,8 @@
 // Unlike a delta rule, what a token writes does not depend on the state, so the walk is bound by what its warps can issue,
 // not by one token's chain.  A warp is LR lanes along the keys times 32 / LR lanes along the values; a lane holds 4 RPV
 // key rows (as packed pairs, for the two-at-a-time multiply-adds of sm_100) of CC value columns.  TB tokens form a batch:
-// one more warp of the block brings their inputs into one stage of a shared-memory ring by asynchronous copies two batches
-// ahead (so that the walking warps spend nothing on it), one barrier stands between two batches, and the batch's TB * CC
+// one more warp of the block brings their inputs into one stage of a shared-memory ring by asynchronous copies three batches
+// ahead (so that the walking warps spend nothing on it; its lanes keep the addresses of what they copy in registers), one barrier stands between two batches, and the batch's TB * CC
 // partial read-outs a lane are summed over the LR lanes by a halving exchange that leaves every lane TB * CC / LR finished
 // numbers.  The order of the sums depends on the head's sizes alone, so the result does not depend on how a sequence was
 // cut into steps.
@@ -25,7 +25,7 @@ struct ScanParams {
     const float* q; const float* k; const float* v;       // first element of token 0's q, k [kv_heads * dim], v [heads * vdim]
     long long q_stride, k_stride, v_stride;               // floats between two tokens' rows
     const float* w; long long w_stride;                   // decay per key channel [tokens, heads * dim], or null: per head
-    const float* scalars;                                 // [tokens, heads, 2]: (decay, dt) without w; (bonus, unused) with w
+    const float* scalars;                                 // [tokens, heads, 4]: (decay, dt, -, -) without w; (bonus, -, -, -) with w
     const float* skip;                                    // [heads] the factor D on v in the read-out, or null
     float* out; long long out_stride;                     // [tokens, heads * vdim]
     float* state; long long slot_stride;                  // state + slot * slot_stride + head * vdim * dim4
@@ -65,7 +65,7 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
 
-constexpr int RING = 3;
+constexpr int RING = 4;
 
 constexpr int MAX_WARPS = 4;                              // walking warps a block
 
@@ -82,30 +82,64 @@ struct Shape {
 // All threads of the block (the number is a multiple of 32).
 __device__ __forceinline__ void block_barrier(int threads) { asm volatile("bar.sync 1, %0;" ::"r"(threads) : "memory"); }
 
-// The copies of one batch (tokens tb .. tb + n - 1) into its stage, by one warp.
-template <typename SH>
-__device__ __forceinline__ void bring_batch(const ScanParams& p, const float* qp, const float* kp, const float* wp, const float* vp,
-                                            const float* sp, int n_cols, int tb, int n, float* stage, int lane, int wide) {
-    constexpr bool CH = SH::ROWS == 3;
-    constexpr int V = SH::ROWS * SH::DP, TOKEN = SH::TOKEN;
-    const int u = wide ? 4 : 1, du = p.dim / u, vu = n_cols / u;         // copies of 16 or of 4 bytes
-    const int rows = SH::ROWS * du, per = rows + vu + 2;
-    for (int e = lane; e < per; e += 32) {
-        const float* src;
-        long long stride;
-        int dst;
-        if (e < du) { src = qp + u * e; stride = p.q_stride; dst = u * e; }
-        else if (e < 2 * du) { src = kp + u * (e - du); stride = p.k_stride; dst = SH::DP + u * (e - du); }
-        else if (CH && e < 3 * du) { src = wp + u * (e - 2 * du); stride = p.w_stride; dst = 2 * SH::DP + u * (e - 2 * du); }
-        else if (e < rows + vu) { src = vp + u * (e - rows); stride = p.v_stride; dst = V + u * (e - rows); }
-        else { src = sp + (e - rows - vu); stride = 2 * p.heads; dst = TOKEN - 4 + (e - rows - vu); }
-        src += (long long)tb * stride;
-        float* d = stage + dst;
-        if (wide && e < rows + vu) {
-            for (int tt = 0; tt < n; ++tt, src += stride, d += TOKEN) cp_async16(d, src);
-        } else {
-            for (int tt = 0; tt < n; ++tt, src += stride, d += TOKEN) cp_async4(d, src);
+// What one lane of the bringing warp copies of every token, in 16-byte groups (rows that are whole groups).
+template <typename SH, int TB>
+struct Bringer {
+    static constexpr bool CH = SH::ROWS == 3;
+    static constexpr int V = SH::ROWS * SH::DP;
+    static constexpr int SLOTS = (SH::ROWS * (SH::DP / 4) + SH::WC * MAX_WARPS / 4 + 1 + 31) / 32;
+    const float* src[SLOTS];
+    long long stride[SLOTS];
+    int dst[SLOTS];                                       // floats into a token's stage; < 0: nothing
+
+    __device__ __forceinline__ Bringer(const ScanParams& p, const float* qp, const float* kp, const float* wp, const float* vp,
+                                       const float* sp, int n_cols, long long t0, int lane) {
+        const int du = p.dim >> 2, vu = n_cols >> 2, rows = SH::ROWS * du;
+#pragma unroll
+        for (int s = 0; s < SLOTS; ++s) {
+            const int e = lane + 32 * s;
+            src[s] = nullptr; stride[s] = 0; dst[s] = -1;
+            if (e < du) { src[s] = qp + 4 * e; stride[s] = p.q_stride; dst[s] = 4 * e; }
+            else if (e < 2 * du) { src[s] = kp + 4 * (e - du); stride[s] = p.k_stride; dst[s] = SH::DP + 4 * (e - du); }
+            else if (CH && e < 3 * du) { src[s] = wp + 4 * (e - 2 * du); stride[s] = p.w_stride; dst[s] = 2 * SH::DP + 4 * (e - 2 * du); }
+            else if (e < rows + vu) { src[s] = vp + 4 * (e - rows); stride[s] = p.v_stride; dst[s] = V + 4 * (e - rows); }
+            else if (e == rows + vu) { src[s] = sp; stride[s] = 4 * p.heads; dst[s] = SH::TOKEN - 4; }
+            if (dst[s] >= 0) src[s] += t0 * stride[s];
         }
+    }
+    // the next n tokens into `stage`
+    __device__ __forceinline__ void bring(float* stage, int n) {
+#pragma unroll
+        for (int s = 0; s < SLOTS; ++s) {
+            if (dst[s] < 0) continue;
+            float* d = stage + dst[s];
+            if (n == TB) {
+#pragma unroll
+                for (int tt = 0; tt < TB; ++tt) { cp_async16(d + tt * SH::TOKEN, src[s]); src[s] += stride[s]; }
+            } else {
+                for (int tt = 0; tt < n; ++tt) { cp_async16(d + tt * SH::TOKEN, src[s]); src[s] += stride[s]; }
+            }
+        }
+    }
+};
+// The same element by element, for rows of other lengths.
+template <typename SH>
+__device__ __forceinline__ void bring_elements(const ScanParams& p, const float* qp, const float* kp, const float* wp, const float* vp,
+                                               const float* sp, int n_cols, long long tb, int n, float* stage, int lane) {
+    constexpr bool CH = SH::ROWS == 3;
+    constexpr int V = SH::ROWS * SH::DP;
+    const int dim = p.dim;
+#pragma unroll 1
+    for (int tt = 0; tt < n; ++tt) {
+        float* d = stage + tt * SH::TOKEN;
+        const long long t = tb + tt;
+        for (int e = lane; e < dim; e += 32) {
+            cp_async4(d + e, qp + t * p.q_stride + e);
+            cp_async4(d + SH::DP + e, kp + t * p.k_stride + e);
+            if constexpr (CH) cp_async4(d + 2 * SH::DP + e, wp + t * p.w_stride + e);
+        }
+        for (int e = lane; e < n_cols; e += 32) cp_async4(d + V + e, vp + t * p.v_stride + e);
+        if (lane < 2) cp_async4(d + SH::TOKEN - 4 + lane, sp + t * (4 * p.heads) + lane);
     }
 }
 
@@ -145,21 +179,29 @@ __global__ void __launch_bounds__(32 * (MAX_WARPS + 1)) scan_kernel(const ScanPa
         const float* kp = p.k + (size_t)kvh * dim;
         const float* vp = p.v + (size_t)head * vdim + c0;
         const float* wp = CH ? p.w + (size_t)head * dim : nullptr;
-        const float* sp = p.scalars + 2 * head;
-        auto bring = [&](int b) {
-            if (b < n_batches)
-                bring_batch<SH>(p, qp, kp, wp, vp, sp, n_cols, t0 + b * TB, min(TB, t1 - t0 - b * TB), ring + (b % RING) * TB * TOKEN, lane, wide);
-            cp_commit();
+        const float* sp = p.scalars + 4 * head;
+        const auto pump = [&](auto&& bring) {             // bring(batch): starts its copies
+#pragma unroll 1
+            for (int b = 0; b < RING - 1; ++b) { bring(b); cp_commit(); }
+#pragma unroll 1
+            for (int b = 0; b < n_batches; ++b) {
+                cp_wait<RING - 2>();
+                block_barrier(blockDim.x);                // batch b has landed, and every warp is done with batch b - 1
+                bring(b + RING - 1);                      // (into the stage that batch b - 1 had)
+                cp_commit();
+            }
+            cp_wait<0>();
         };
-#pragma unroll 1
-        for (int b = 0; b < RING - 1; ++b) bring(b);
-#pragma unroll 1
-        for (int b = 0; b < n_batches; ++b) {
-            cp_wait<RING - 2>();
-            block_barrier(blockDim.x);                    // batch b has landed, and every warp is done with batch b - 1
-            bring(b + RING - 1);                          // (into the stage that batch b - 1 had)
+        if (wide) {
+            Bringer<SH, TB> br(p, qp, kp, wp, vp, sp, n_cols, t0, lane);
+            pump([&](int b) { if (b < n_batches) br.bring(ring + (b % RING) * TB * TOKEN, min(TB, t1 - t0 - b * TB)); });
+        } else {
+            pump([&](int b) {
+                if (b < n_batches)
+                    bring_elements<SH>(p, qp, kp, wp, vp, sp, n_cols, t0 + (long long)b * TB, min(TB, t1 - t0 - b * TB),
+                                       ring + (b % RING) * TB * TOKEN, lane);
+            });
         }
-        cp_wait<0>();
         return;
     }
 
@@ -276,7 +318,7 @@ __global__ void __launch_bounds__(32 * (MAX_WARPS + 1)) scan_kernel(const ScanPa
 }
 
 // ---- what a token brings besides q, k and v
-// state space: scalars[t, h] = (exp(-exp(A_log[h]) dt), dt), dt = softplus(a[t, h] + dt_bias[h])
+// state space: scalars[t, h] = (exp(-exp(A_log[h]) dt), dt, -, -), dt = softplus(a[t, h] + dt_bias[h])
 __global__ void __launch_bounds__(128) state_space_gates_kernel(const float* __restrict__ a, long long stride,
                                                                 const float* __restrict__ a_log, const float* __restrict__ dt_bias,
                                                                 float* __restrict__ scalars, long long n, int heads) {
@@ -288,7 +330,7 @@ __global__ void __launch_bounds__(128) state_space_gates_kernel(const float* __r
     const int h = (int)(i % heads);
     const float z = a[t * stride + h] + dt_bias[h];
     const float dt = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
-    *(float2*)(scalars + 2 * i) = make_float2(expf(-expf(a_log[h]) * dt), dt);
+    *(float4*)(scalars + 4 * i) = make_float4(expf(-expf(a_log[h]) * dt), dt, 0.f, 0.f);
 }
 
 // decaying memory: w[t, h, i] = exp(-exp(z + w0)) in place, scalars[t, h, 0] = sum_i q_i u_i k_i.  One warp per (token, head).
@@ -313,7 +355,7 @@ __global__ void __launch_bounds__(128) memory_gates_kernel(float* __restrict__ w
         s = fmaf(qr[i] * u[h * dim + i], kr[i], s);
     }
     s = warp_sum(s);
-    if (lane == 0) *(float2*)(scalars + 2 * row) = make_float2(s, 0.f);
+    if (lane == 0) *(float4*)(scalars + 4 * row) = make_float4(s, 0.f, 0.f, 0.f);
 }
 
 template <int LR, int RPV, int CC, int TB, bool CH>
@@ -339,7 +381,7 @@ template <bool CH>
 int choose_scan(const ScanParams& p, cudaStream_t st) {
     const auto al = [](const void* x) { return ((uintptr_t)x & 15) == 0; };
     const int wide = p.dim % 4 == 0 && p.vdim % 4 == 0 && p.q_stride % 4 == 0 && p.k_stride % 4 == 0 && p.v_stride % 4 == 0 &&
-                     al(p.q) && al(p.k) && al(p.v) && (!CH || (p.w_stride % 4 == 0 && al(p.w)));
+                     al(p.q) && al(p.k) && al(p.v) && al(p.scalars) && (!CH || (p.w_stride % 4 == 0 && al(p.w)));
     if (p.dim <= 32) return launch_scan<8, 1, 2, 8, CH>(p, wide, st);
     if (p.dim <= 64) return launch_scan<8, 2, 2, 8, CH>(p, wide, st);
     if (p.dim <= 128) return launch_scan<8, 4, 2, 8, CH>(p, wide, st);

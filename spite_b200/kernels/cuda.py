@@ -1188,7 +1188,7 @@ class CudaKernels(KernelSet):
         for name, (t, column), width in (("q", q, kv_heads * dim), ("k", k, kv_heads * dim), ("v", v, heads * vdim)):
             self._t(t, torch.float32, name)
             at.append((self._columns(t, column, width, M, f"{what}: {name}"), t.shape[1]))
-        scalars = torch.empty((M, heads, 2), dtype=torch.float32, device=out.device)
+        scalars = torch.empty((M, heads, 4), dtype=torch.float32, device=out.device)
         p = ScanParams(q=at[0][0], k=at[1][0], v=at[2][0], q_stride=at[0][1], k_stride=at[1][1], v_stride=at[2][1],
                        w=None, w_stride=0, scalars=scalars.data_ptr(), skip=None, out=out.data_ptr(), out_stride=out.shape[1],
                        state=state.data_ptr() + 4 * int(state_offset), slot_stride=slot_stride,
