@@ -28,7 +28,7 @@ class TorchReferenceKernels(KernelSet):
         x = table[token_ids.long()].to(self.acc) * scale
         if position_table is not None:
             x = x + position_table[positions.long()].to(self.acc)
-        out_h.copy_(x.to(out_h.dtype) if copies == 1 else x.to(out_h.dtype)[:, None].expand_as(out_h))
+        out_h.copy_(x.to(out_h.dtype)[:, None].expand_as(out_h) if out_h.dim() == 3 else x.to(out_h.dtype))
 
     def pack_pair(self, a, b, out, *, refill=None):
         out.copy_(torch.cat([a, b], -1).to(out.dtype))
