@@ -298,9 +298,23 @@ class CudaKernels(KernelSet):
         # Scout shapes, one token 2.90 ms with (110 KiB, 2 per multiprocessor) against 3.01 with (74 KiB, 3), eight
         # tokens 7.10 against 7.02, sixty-four alike; one block per multiprocessor with 110 or 200 KiB: 3.2 and 3.1 ms
         self.stream_shape = [(110 * 1024, 2 * self.sm_count), (74 * 1024, 3 * self.sm_count)]
-        self._tickets, self._tickets_n = {}, 65536       # arrival counters of the k splits (zero between calls), per stream
+        # arrival counters of the splits (zero between calls), one set per stream, since calls that share a set must not
+        # overlap.  The sets are made ahead: one made while a CUDA graph is captured would lie in the graphs' memory
+        # pool, where a graph captured before keeps its temporaries.
+        self._tickets, self._tickets_n = {}, 65536
+        self._spare_tickets = [torch.zeros(self._tickets_n, dtype=torch.int32, device=self.device) for _ in range(4)]
 
     # ------------------------------------------------------------------ helpers
+    def _tickets_of(self, stream: int):
+        tickets = self._tickets.get(stream)
+        if tickets is None:
+            if not torch.cuda.is_current_stream_capturing():
+                self._spare_tickets.append(torch.zeros(self._tickets_n, dtype=torch.int32, device=self.device))
+            if not self._spare_tickets:
+                raise KernelError("a graph capture on yet another stream has no arrival counters left")
+            tickets = self._tickets[stream] = self._spare_tickets.pop(0)
+        return tickets
+
     def _count(self, library, n=1):
         self.launches += n
         self.launches_by_library[library] += n
@@ -570,24 +584,24 @@ class CudaKernels(KernelSet):
         _check(st, "clear_pages")
 
     # ------------------------------------------------------------------ matrix products
-    def _gemm(self, p: GemmParams, what, max_rows_per_group, gather_src=None):
+    def _gemm(self, p: GemmParams, what, max_rows_per_group, gather_src=None, even_groups=False):
         """Pick the kernel.  bfloat16: up to 16 rows (a decode step) go to the TMA weight-streaming
         kernel when K is a multiple of 64, else to the register-ring streaming kernel; more rows to
         the tcgen05 kernels (TMA-fed, accumulators in TMEM): one group of 256 rows and more, or groups
         of 512 rows on average, on pairs of multiprocessors, the rest on one block a tile; a very
         tall matrix (output head) goes there even with few rows.  float32, and shapes those refuse, go to the CUDA-core kernel.
         `gather_src` is the tensor whose rows `p.a_rows` gathers: the tcgen05 kernel wants contiguous
-        rows, so they are gathered first."""
+        rows, so they are gathered first.  `even_groups`: every group has `max_rows_per_group` rows."""
         if self.dtype == torch.bfloat16:
             grouped = bool(p.group_offsets)
             # measured on B200 at Scout shapes: the streaming kernel wins up to 16 rows except on very
             # tall matrices (output head), where the TMA pipeline of the tcgen05 kernel streams better
-            few = p.M <= self.skinny_max_rows and not (not grouped and p.N >= 65536 and p.M > self.skinny_tall_rows)
+            few = (max_rows_per_group if even_groups else p.M) <= self.skinny_max_rows and not (not grouped and p.N >= 65536 and p.M > self.skinny_tall_rows)
             tc_ok = self.use_tcgen05 and p.K % 8 == 0 and p.lda % 8 == 0
             # ... and a one-group product of up to 32 rows in place (the dense projections of a larger decode batch)
             more = (not grouped and not p.a_rows and 16 < p.M <= self.stream_max_rows and p.N < 65536)
             if (few or more) and self.use_stream and p.K % 64 == 0 and max_rows_per_group <= (32 if more else 16):
-                st = self._gemm_stream(p, int(max_rows_per_group), grouped)
+                st = self._gemm_stream(p, int(max_rows_per_group), grouped, int(max_rows_per_group) if even_groups else p.M)
                 if st != -2:
                     self._count("gemm_stream", 1)
                     _check(st, what + " (streaming)")
@@ -658,20 +672,20 @@ class CudaKernels(KernelSet):
             return p.n_groups >= self.tc_experts_down_min_groups and 32 <= avg <= self.tc_experts_max_group_rows
         return False
 
-    def _gemm_stream(self, p, max_rows_per_group, grouped):
+    def _gemm_stream(self, p, max_rows_per_group, grouped, rows):
         """The TMA weight-streaming kernel for decode steps: picks the tile height (k slices inside the block)
         and the k splits across blocks so that the work items are many enough to spread evenly, and lends the
         scratch for the partial sums of the splits."""
         swiglu = p.epilogue == EPI_SWIGLU
         groups = min(p.n_groups, p.M) if grouped else 1
-        smem, blocks = self.stream_shape[0 if p.M <= 3 or p.M > 16 else 1]      # (the tokens of many rows need the larger ring)
+        smem, blocks = self.stream_shape[0 if rows <= 3 or rows > 16 else 1]      # (the tokens of many rows need the larger ring)
         nt = 8 if max_rows_per_group <= 8 else 16 if max_rows_per_group <= 16 else 32
-        slices, splits = self.stream_force or self._stream_cut(p.M, p.N, p.K, groups, swiglu, blocks, smem, nt, grouped)
-        rows = 128 // slices
-        tiles = -(-p.N // (rows // 2 if swiglu else rows)) * groups
+        slices, splits = self.stream_force or self._stream_cut(rows, p.N, p.K, groups, swiglu, blocks, smem, nt, grouped)
+        tile_rows = 128 // slices
+        tiles = -(-p.N // (tile_rows // 2 if swiglu else tile_rows)) * groups
         lib = self._lib("gemm_stream")
         stream = torch.cuda.current_stream().cuda_stream
-        if slices == 1 and 2 <= splits <= self.stream_cluster_max_splits and p.M <= self.stream_cluster_max_rows:
+        if slices == 1 and 2 <= splits <= self.stream_cluster_max_splits and rows <= self.stream_cluster_max_rows:
             # the k splits of a tile as one thread-block cluster: their sums meet in shared memory
             st = lib.spite_gemm_stream(C.byref(p), max_rows_per_group, 1, 1, blocks, smem, splits, None, C.c_longlong(0),
                                        None, 0, C.c_void_p(stream))
@@ -681,12 +695,9 @@ class CudaKernels(KernelSet):
         if splits > 1:
             if tiles > self._tickets_n:
                 return -2
-            n_floats = tiles * splits * nt * rows
+            n_floats = tiles * splits * nt * tile_rows
             scratch = torch.empty(n_floats, dtype=torch.float32, device=self.device)
-        # the k splits' arrival counters: one set per stream, since calls that share a set must not overlap
-        tickets = self._tickets.get(stream)
-        if tickets is None and splits > 1:
-            tickets = self._tickets[stream] = torch.zeros(self._tickets_n, dtype=torch.int32, device=self.device)
+        tickets = self._tickets_of(stream) if splits > 1 else None
         return lib.spite_gemm_stream(
             C.byref(p), max_rows_per_group, slices, 0, blocks, smem, splits, C.c_void_p(_ptr(scratch)),
             C.c_longlong(n_floats), C.c_void_p(_ptr(tickets)), self._tickets_n, C.c_void_p(stream))
@@ -828,7 +839,7 @@ class CudaKernels(KernelSet):
         p = GemmParams(A=x.data_ptr(), W=w.data_ptr(), C=out.data_ptr(), a_rows=None, c_rows=None,
                        group_offsets=offsets.data_ptr(), row_scale=None, lda=K, ldc=N, w_group_stride=N * K,
                        n_groups=G, M=G * M, N=N, K=K, epilogue=EPI_STORE_F32, scale_by_a_row=0)
-        self._gemm(p, "batched_linear", M)
+        self._gemm(p, "batched_linear", M, even_groups=True)
 
     # ------------------------------------------------------------------ attention
     def _step_tokens(self, batch, group):
@@ -1056,10 +1067,7 @@ class CudaKernels(KernelSet):
                 raise KernelError(f"paged_attention: {base} (request block, kv head) pairs exceed the {self._tickets_n} tickets")
             partial = torch.empty((base * splits * 16 * (c.head_dim + 4),), dtype=torch.float32, device=self.device)
             self.attention_scratch_bytes = partial.numel() * 4
-            stream = torch.cuda.current_stream().cuda_stream
-            tickets = self._tickets.get(stream)
-            if tickets is None:
-                tickets = self._tickets[stream] = torch.zeros(self._tickets_n, dtype=torch.int32, device=self.device)
+            tickets = self._tickets_of(torch.cuda.current_stream().cuda_stream)
         x = AttnDecodeExtra(cu_seqlens=batch.cu_seqlens.data_ptr(), partial=_ptr(partial), tickets=_ptr(tickets),
                             n_segments=len(batch.segments), tokens_per_block=tpb, n_splits=splits,
                             seg_min_tokens=0, seg_max_tokens=seg_max, cache_settled=int(bool(cache_settled)))

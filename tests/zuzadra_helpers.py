@@ -121,7 +121,9 @@ _plain_cache: dict = {}
 
 def plain_logits(folder, tokens, sixteen=False):
     """(logits computed in float64, what a position may be off by through rounding alone, as a fraction of the largest
-    logit).  For float32 arithmetic: four times the distance of a float32 run.  With `sixteen`: the largest distance among
+    logit).  For float32 arithmetic: four times the distance of a float32 run, or eight times that of a run whose products'
+    inputs are disturbed by relative errors of up to 2^-23 (a head of a memory that puts out next to nothing before its norm is
+    ill-conditioned).  With `sixteen`: the largest distance among
     two runs whose products' and attention's inputs are disturbed by relative errors of up to 2^-7, or four times that of a
     run that rounds them to bfloat16."""
     key = (str(folder), tuple(tokens), sixteen)
@@ -135,7 +137,11 @@ def plain_logits(folder, tokens, sixteen=False):
             exact = plain.forward(cfg, tensors, list(tokens), torch.float64, round_inputs=lambda x: x.to(torch.bfloat16).to(x.dtype))
             moved = torch.stack([(ref - low).abs().amax(-1) for low in lows] + [4.0 * (ref - exact).abs().amax(-1)]).amax(0)
         else:
-            moved = 4.0 * (ref - plain.forward(cfg, tensors, list(tokens), torch.float32).double()).abs().amax(-1)
+            g = torch.Generator().manual_seed(len(tokens))
+            shake = lambda x: x * (1.0 + 2.0 ** -23 * (2.0 * torch.rand(x.shape, generator=g, dtype=x.dtype) - 1.0))
+            lows = [plain.forward(cfg, tensors, list(tokens), torch.float64, round_inputs=shake) for _ in range(3)]
+            moved = torch.stack([8.0 * (ref - low).abs().amax(-1) for low in lows] +
+                                [4.0 * (ref - plain.forward(cfg, tensors, list(tokens), torch.float32).double()).abs().amax(-1)]).amax(0)
         _plain_cache[key] = (ref, moved / float(ref.abs().max()))
     return _plain_cache[key]
 
