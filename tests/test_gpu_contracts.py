@@ -191,6 +191,66 @@ def test_router_entry_point(libs):
     assert untouched(ids, rows, wts, logits, offs)
 
 
+def test_scan_stream_and_shift_entry_points(libs):
+    from spite_b200.kernels.cuda import ScanParams, StreamsParams, TokenShiftParams
+    ew, scan, att = libs["elementwise"], libs["scan"], libs["attention"]
+    f32 = lambda *shape: torch.ones(shape, dtype=torch.float32, device=DEV)
+    i32 = lambda *v: torch.tensor(v, dtype=torch.int32, device=DEV)
+    M, H, N, P = 4, 2, 8, 8
+    q, k, v, w, a, one, cu, slots, seg = f32(M, H * N), f32(M, H * N), f32(M, H * P), f32(M, H * N), f32(M, H), f32(H * N), i32(0, 4), i32(0), i32(0, 0, 0, 0)
+    out, state, scalars = canary((M, H * P)), canary((1, H * P * N)), canary((M, H, 4))
+    good = dict(q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), q_stride=H * N, k_stride=H * N, v_stride=H * P, w=None, w_stride=0,
+                scalars=scalars.data_ptr(), skip=one.data_ptr(), out=out.data_ptr(), out_stride=H * P, state=state.data_ptr(),
+                slot_stride=H * P * N, cu_seqlens=cu.data_ptr(), slots=slots.data_ptr(), n_segments=1, n_tokens=M, heads=H, kv_heads=H,
+                dim=N, vdim=P)
+    ss = lambda **c: scan.spite_state_space_scan(C.byref(ScanParams(**dict(good, **c))), ptr(a), C.c_longlong(H), ptr(one), ptr(one), None)
+    dec = lambda **c: scan.spite_decay_scan(C.byref(ScanParams(**dict(good, skip=None, w=w.data_ptr(), w_stride=H * N, **c))), ptr(one), ptr(one), None)
+    for call in (ss, dec):
+        for c in (dict(q=None), dict(k=None), dict(v=None), dict(out=None), dict(state=None), dict(scalars=None), dict(cu_seqlens=None),
+                  dict(slots=None), dict(heads=0), dict(heads=3, kv_heads=2), dict(dim=0), dict(vdim=0), dict(slot_stride=7), dict(out_stride=3),
+                  dict(n_tokens=-1), dict(n_segments=-1), dict(q_stride=0)):
+            assert call(**c) == BAD_ARG, c
+        for c in (dict(dim=513, slot_stride=1 << 20), dict(slot_stride=H * P * N + 2), dict(state=state.data_ptr() + 4)):
+            assert call(**c) == UNSUPPORTED, c
+    assert ss(w=w.data_ptr(), w_stride=H * N) == BAD_ARG and dec(kv_heads=1) == BAD_ARG
+    assert scan.spite_state_space_scan(C.byref(ScanParams(**good)), None, C.c_longlong(H), ptr(one), ptr(one), None) == BAD_ARG
+    assert scan.spite_decay_scan(C.byref(ScanParams(**good)), ptr(one), ptr(one), None) == BAD_ARG
+    assert scan.spite_state_space_scan(None, ptr(a), C.c_longlong(H), ptr(one), ptr(one), None) == BAD_ARG
+    assert untouched(out, state, scalars)
+    # several residual streams
+    x, nxt = canary((M, 2, 16)), canary((M, 16))
+    good = dict(x=x.data_ptr(), y=f32(M, 16).data_ptr(), bias=None, scale=None, mix=one.data_ptr(), w_out=one.data_ptr(), w_in=one.data_ptr(),
+                gain=None, next_out=nxt.data_ptr(), rows=None, n_rows=M, d=16, streams=2, write_back=1, eps=1e-5)
+    st = lambda dt=0, **c: ew.spite_streams(dt, C.byref(StreamsParams(**dict(good, **c))), None)
+    for c in (dict(x=None), dict(y=None, next_out=None), dict(mix=None), dict(w_out=None), dict(w_in=None), dict(d=0), dict(streams=0),
+              dict(n_rows=-1), dict(gain=one.data_ptr(), eps=0.0), dict(rows=seg.data_ptr())):
+        assert st(**c) == BAD_ARG, c
+    assert st(dt=7) == BAD_ARG and st(streams=33) == UNSUPPORTED and st(d=60000) == UNSUPPORTED
+    assert ew.spite_streams(0, None, None) == BAD_ARG and untouched(x, nxt)
+    # token shift
+    mixes, slot = canary((2, M, 16)), canary((1, 16))
+    good = dict(x=f32(M, 16).data_ptr(), mu=f32(2, 16).data_ptr(), out=mixes.data_ptr(), state=slot.data_ptr(), slot_stride=16,
+                seg_of_token=seg.data_ptr(), cu_seqlens=cu.data_ptr(), slots=slots.data_ptr(), offsets_out=None, n_tokens=M, d=16, n_mixes=2)
+    sh = lambda dt=0, **c: ew.spite_token_shift(dt, C.byref(TokenShiftParams(**dict(good, **c))), None)
+    for c in (dict(x=None), dict(mu=None), dict(out=None), dict(state=None), dict(seg_of_token=None), dict(cu_seqlens=None), dict(slots=None),
+              dict(n_tokens=-1), dict(d=0), dict(n_mixes=0), dict(slot_stride=15)):
+        assert sh(**c) == BAD_ARG, c
+    assert sh(dt=3) == BAD_ARG and sh(n_mixes=9) == UNSUPPORTED and untouched(mixes, slot)
+    # gate and norm in parts, heads turned back
+    o = canary((M, 16))
+    gn = lambda x=q, z=k, zs=16, g=one, out=o, n=M, groups=2, size=8, eps=1e-5, dt=0: ew.spite_gate_group_norm(
+        dt, ptr(x), ptr(z), C.c_longlong(zs), ptr(g), ptr(out), n, groups, size, C.c_float(eps), None)
+    for c in (dict(x=None), dict(z=None), dict(g=None), dict(out=None), dict(n=-1), dict(groups=0), dict(size=0), dict(eps=0.0), dict(zs=15), dict(dt=5)):
+        assert gn(**c) == BAD_ARG, c
+    assert gn(size=60000, zs=120000) == UNSUPPORTED
+    th = lambda x=q, out=o, stride=16, pos=seg, f=one, rot=8, pair=1, n=M, heads=2, hd=8, size=8, dt=0: att.spite_turn_heads(
+        dt, ptr(x), ptr(out), C.c_longlong(stride), ptr(pos), ptr(f), None, rot, pair, n, heads, hd, size, C.c_float(1.0), None)
+    for c in (dict(x=None), dict(out=None), dict(stride=15), dict(pos=None), dict(rot=7), dict(rot=10), dict(pair=2), dict(n=-1), dict(heads=0),
+              dict(hd=7), dict(size=0), dict(dt=4)):
+        assert th(**c) == BAD_ARG, c
+    assert untouched(o)
+
+
 def test_convolution_cast_identity_and_delta_entry_points(libs):
     """The entry points of the short convolution, the cast, the identity experts and the delta rule refuse malformed calls
     and sizes outside their domain, and launch nothing then."""
