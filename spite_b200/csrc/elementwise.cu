@@ -787,7 +787,7 @@ SPITE_API int spite_token_shift(int dtype, const TokenShiftParams* p, void* stre
     const bool vec = p->d % 4 == 0 && ((((uintptr_t)p->x | (uintptr_t)p->mu | (uintptr_t)p->out) & 15) == 0);
     const int per = vec ? 4 : 1;
     const int threads = (p->d + per - 1) / per >= 256 ? 256 : 128;
-    dim3 grid(p->n_tokens, p->n_tokens < 64 ? (p->d + per * threads - 1) / (per * threads) : 1);
+    dim3 grid(p->n_tokens, p->n_tokens < 512 ? (p->d + per * threads - 1) / (per * threads) : 1);
     cudaStream_t st = (cudaStream_t)stream;
     if (dtype == SPITE_DT_F32) {
         if (vec) SPITE_LAUNCH((token_shift_kernel<float, true>), grid, threads, 0, st, *p);
