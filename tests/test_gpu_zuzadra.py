@@ -405,7 +405,7 @@ def test_bias_and_activation_in_every_product_kernel(dtype, M, N, K, library, ac
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("G,M,N,K", [(4, 1, 128, 192), (4, 3, 72, 40), (4, 8, 256, 128), (4, 33, 96, 72), (2, 300, 128, 64), (4, 600, 64, 128), (3, 5, 33, 50)])
+@pytest.mark.parametrize("G,M,N,K", [(4, 1, 136, 256), (4, 3, 72, 40), (4, 8, 256, 128), (4, 33, 96, 72), (2, 300, 128, 64), (4, 600, 64, 128), (3, 5, 33, 50)])
 def test_one_product_per_group(dtype, G, M, N, K):
     ks = kernels(dtype)
     g = gen(G * M)
