@@ -36,7 +36,7 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkPrepareParams p
     const int t = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
     const int nq = p.num_heads, nkv = c.num_kv_heads, hd = c.head_dim;
-    const int heads_total = p.q_only ? nq : nq + 2 * nkv;
+    const int heads_total = p.q_only ? nq : p.values_are_keys ? nq + nkv : nq + 2 * nkv;
     const int head_end = min(heads_total, (int)(blockIdx.y + 1) * heads_per_block);
     const int pos = b.positions[t];
     if (p.gates_out && blockIdx.y == 0)                      // the gate columns behind the heads
@@ -144,6 +144,14 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkPrepareParams p
                 if (bias) { x0[r] += bias[e0[r]]; x1[r] += bias[e1[r]]; }
             }
         }
+        if (p.values_are_keys && !is_q) {                        // the key as projected is the value
+#pragma unroll
+            for (int r = 0; r < MAXP; ++r) {
+                if (2 * (lane + 32 * r) >= hd) continue;
+                if (halves) { dst[c.v_offset + e0[r]] = from_f32<T>(x0[r]); dst[c.v_offset + e1[r]] = from_f32<T>(x1[r]); }
+                else store_pair(dst + c.v_offset + e0[r], x0[r], x1[r]);
+            }
+        }
         if (norm_first) {
             float ss = 0.f;
 #pragma unroll
@@ -247,6 +255,7 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const AttentionPar
     for (int r = 0; r < MAXD; ++r) acc[r] = 0.f;
     float m = -INFINITY, l = 0.f;
     const float slope = slope_of(p, h);
+    const float* dist = distance_row_of(p, h);
 
     for (int j0 = lo; j0 <= pos; j0 += 32) {
         const int j = j0 + lane;
@@ -259,6 +268,7 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const AttentionPar
             float dot = 0.f;
             for (int d = 0; d < hd; ++d) dot = fmaf(q_s[warp][d], to_f32(k[d]), dot);
             s = capped(p, dot * p.softmax_scale) - slope * (float)(pos - j);
+            if (dist) s += dist[min(pos - j, p.distance_len - 1)];
         }
         const float m_new = fmaxf(m, warp_max(s));
         const float corr = expf(m - m_new);                  // 0 on the first tile (m = -inf)
@@ -313,7 +323,7 @@ SPITE_API int spite_qk_prepare(int dtype, const QkPrepareParams* given, const St
     if (!c) return SPITE_BAD_ARG;
     QkPrepareParams filled = *given;                          // a caller that leaves the later fields at zero means: rows
     if (filled.qkv_stride == 0)                               // without anything behind the heads, a pure rotation
-        filled.qkv_stride = (long long)(filled.num_heads + (filled.q_only ? 0 : 2 * c->num_kv_heads)) * c->head_dim;
+        filled.qkv_stride = (long long)(filled.num_heads + (filled.q_only ? 0 : filled.values_are_keys ? 1 : 2) * (long long)(filled.q_only ? 0 : c->num_kv_heads)) * c->head_dim;
     if (filled.rot_amplitude == 0.f) filled.rot_amplitude = 1.f;
     const QkPrepareParams* p = &filled;
     const int chk = check_common(b, c, p->num_heads);
@@ -321,8 +331,9 @@ SPITE_API int spite_qk_prepare(int dtype, const QkPrepareParams* given, const St
     if (b->n_tokens == 0) return SPITE_OK;
     if (p->pairing != SPITE_PAIR_NEIGHBOURS && p->pairing != SPITE_PAIR_HALVES) return SPITE_BAD_ARG;
     if (p->inv_freq && (p->rotary_dim < 2 || p->rotary_dim % 2 || p->rotary_dim > c->head_dim)) return SPITE_BAD_ARG;
-    const int heads = p->num_heads + (p->q_only ? 0 : 2 * c->num_kv_heads);
-    if (p->q_only && (p->v_other || p->gates_out)) return SPITE_BAD_ARG;
+    const int heads = p->num_heads + (p->q_only ? 0 : (p->values_are_keys ? 1 : 2) * c->num_kv_heads);
+    if (p->q_only && (p->v_other || p->gates_out || p->values_are_keys)) return SPITE_BAD_ARG;
+    if (p->values_are_keys && (p->v_other || p->v_inv_freq || c->v_offset == 0)) return SPITE_BAD_ARG;
     if (p->qkv_stride < (long long)heads * c->head_dim || (p->qkv_stride & 1)) return SPITE_BAD_ARG;
     if (p->gates_out && p->qkv_stride < (long long)heads * c->head_dim + p->num_heads) return SPITE_BAD_ARG;
     if (p->v_inv_freq && (p->v_other || p->q_only || p->v_rotary_dim < 2 || p->v_rotary_dim % 2 || p->v_rotary_dim > c->head_dim ||
@@ -379,6 +390,7 @@ SPITE_API int spite_paged_attention(int dtype, const AttentionParams* p, const S
     if (chk != SPITE_OK) return chk;
     if (p->window_kind < 0 || p->window_kind > 2) return SPITE_BAD_ARG;
     if (p->window_kind != SPITE_WINDOW_FULL && p->window_size < 1) return SPITE_BAD_ARG;
+    if (!distance_bias_ok(p)) return SPITE_BAD_ARG;
     if (b->n_tokens == 0) return SPITE_OK;
     dim3 grid(b->n_tokens, (p->num_heads + 3) / 4);
     if (grid.y > 65535) return SPITE_UNSUPPORTED;

@@ -71,6 +71,9 @@ struct QkPrepareParams {
     // what inv_freq and v_inv_freq lost when they were rounded to float32 (null: the angle is the rounded product)
     const float* inv_freq_low;
     const float* v_inv_freq_low;
+    // the values are the projected keys (bias included), as they are before norm and rotation: a row of qkv holds q heads
+    // and k heads alone
+    int values_are_keys;
 };
 
 // cos and sin of pos * (freq + low).  With `low` the product's own rounding error and the frequency's are put back to second
@@ -101,7 +104,20 @@ struct AttentionParams {
     int out_by_head_tokens;     // 0: out is [tokens, num_heads, head_dim]; n > 0: out is [num_heads, n, head_dim], head by head
                                 // (n the tokens of the step), the order in which a product per head reads its rows
     float score_softcap;        // > 0: a scaled score s becomes cap * tanh(s / cap) before bias, mask and softmax
+    // A number per head and distance (or null): head h's score of a key n positions before the query gets
+    // distance_bias[h * (distance_len + 2 * SPITE_DISTANCE_PAD) + SPITE_DISTANCE_PAD + min(n, distance_len - 1)].  A row's ends
+    // are repeated SPITE_DISTANCE_PAD times on either side, so that a tile of keys around them reads without a test per key.
+    const float* distance_bias;
+    const int* distance_runs;   // [distance_len] the smallest distance from which up to this one every head's number stays the same
+    int distance_len;
 };
+
+#define SPITE_DISTANCE_PAD 64
+
+// The numbers of head `head` by distance (null without a table).
+__device__ __forceinline__ const float* distance_row_of(const AttentionParams& p, int head) {
+    return p.distance_bias ? p.distance_bias + (size_t)head * (p.distance_len + 2 * SPITE_DISTANCE_PAD) + SPITE_DISTANCE_PAD : nullptr;
+}
 
 // Where the output row of (token, head) starts, in rows of head_dim elements.
 __device__ __forceinline__ size_t out_row_of(const AttentionParams& p, int token, int head) {
@@ -116,14 +132,24 @@ __device__ __forceinline__ float sink_of(const AttentionParams& p, int head) {
 __device__ __forceinline__ float slope_of(const AttentionParams& p, int head) {
     return p.head_slopes ? p.head_slopes[head] : 0.f;
 }
-// A scaled score squashed into (-cap, cap), or itself without a cap.  The tensor-core kernels are compiled in both
-// forms (CAP): with the choice made per score at run time, the decode kernel took a tenth longer without any cap.
+// A scaled score squashed into (-cap, cap), or itself without a cap.
 __device__ __forceinline__ float capped(const AttentionParams& p, float s) {
     return p.score_softcap > 0.f ? p.score_softcap * tanhf(s / p.score_softcap) : s;
 }
-template <bool CAP> __device__ __forceinline__ float capped_if(const AttentionParams& p, float s) {
-    if constexpr (CAP) return p.score_softcap * tanhf(s / p.score_softcap);
-    else return s;
+// The tensor-core kernels are compiled in three forms: scores as they are, capped, and with a number per distance (capped
+// if there is a cap).  With the choice made per score at run time, the decode kernel took a tenth longer without any cap.
+enum ScoreForm { FORM_PLAIN = 0, FORM_CAP = 1, FORM_DISTANCE = 2 };
+static inline int score_form_of(const AttentionParams& p) {
+    return p.distance_bias ? FORM_DISTANCE : p.score_softcap > 0.f ? FORM_CAP : FORM_PLAIN;
+}
+static inline bool distance_bias_ok(const AttentionParams* p) {
+    return !p->distance_bias || (p->distance_runs && p->distance_len >= 1 && p->distance_len <= (1 << 24));
+}
+// The score of a visible key n positions before the query, from the scaled product `s`.
+template <int FORM> __device__ __forceinline__ float score_of(const AttentionParams& p, float s, float slope, const float* row, int n) {
+    if constexpr (FORM == FORM_CAP) return p.score_softcap * tanhf(s / p.score_softcap) - slope * (float)n;
+    else if constexpr (FORM == FORM_DISTANCE) return capped(p, s) - slope * (float)n + row[min(n, p.distance_len - 1)];
+    else return s - slope * (float)n;
 }
 // The factor on a finished output row.
 __device__ __forceinline__ float gate_of(const AttentionParams& p, int token, int head) {

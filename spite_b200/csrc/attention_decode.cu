@@ -69,7 +69,7 @@ __device__ __forceinline__ unsigned tile_addr(unsigned base, int r, int ch) {
 }
 
 // NKB = head_dim / 64.  grid (blocks over the served segments, kv heads, splits).
-template <int NKB, bool CAP>
+template <int NKB, int FORM>
 __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_constant__ CUtensorMap map_k,
                                                               const __grid_constant__ CUtensorMap map_v,
                                                               const AttentionParams p, const StepTokens b,
@@ -176,6 +176,7 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
         const int g = lane >> 2, cc = lane & 3;
         int row_pos[2], row_lo[2];
         float row_slope[2];                                  // what a key costs per position of distance (0: no bias)
+        const float* row_dist[2];                               // what a key adds by its distance (null: nothing)
         bool row_ok[2];
         unsigned qa[NK][4];
 #pragma unroll
@@ -186,6 +187,7 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
             const int head = kvh * G + (row_ok[h] ? r % G : 0);
             row_pos[h] = b.positions[tok];
             row_slope[h] = slope_of(p, head);
+            row_dist[h] = distance_row_of(p, head);
             row_lo[h] = window_lowest(p.window_kind, p.window_size, row_pos[h]);
             const __nv_bfloat16* qrow = (const __nv_bfloat16*)p.q + ((size_t)tok * nq + head) * HD;
 #pragma unroll
@@ -235,7 +237,7 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
                         for (int e = 0; e < 2; ++e) {
                             const int j = j0 + 8 * n + 2 * cc + e;
                             const bool vis = row_ok[h] && j >= row_lo[h] && j <= row_pos[h];
-                            const float v = vis ? capped_if<CAP>(p, sc[n][2 * h + e] * p.softmax_scale) - row_slope[h] * (float)(row_pos[h] - j) : -INFINITY;
+                            const float v = vis ? score_of<FORM>(p, sc[n][2 * h + e] * p.softmax_scale, row_slope[h], row_dist[h], row_pos[h] - j) : -INFINITY;
                             sc[n][2 * h + e] = v;
                             mx = fmaxf(mx, v);
                         }
@@ -431,7 +433,8 @@ int launch(const AttentionParams& p, const StepTokens& b, const PagedCache& c, c
     ring = (ring + 15) & ~(size_t)15;
     const size_t smem = ring + sizeof(Tail) + 1024;
     if (smem > 227 * 1024) return SPITE_UNSUPPORTED;
-    auto k = p.score_softcap > 0.f ? attn_decode_kernel<NKB, true> : attn_decode_kernel<NKB, false>;
+    const int form = score_form_of(p);
+    auto k = form == FORM_DISTANCE ? attn_decode_kernel<NKB, FORM_DISTANCE> : form == FORM_CAP ? attn_decode_kernel<NKB, FORM_CAP> : attn_decode_kernel<NKB, FORM_PLAIN>;
     if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
         cudaFuncSetAttribute(k, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared) != cudaSuccess)
         return SPITE_LAUNCH_FAILED;
@@ -454,6 +457,7 @@ SPITE_API int spite_paged_attention_decode(const AttentionParams* p, const StepT
     if (p->num_heads < 1 || c->num_kv_heads < 1 || p->num_heads % c->num_kv_heads) return SPITE_BAD_ARG;
     if (p->window_kind < 0 || p->window_kind > 2) return SPITE_BAD_ARG;
     if (p->window_kind != SPITE_WINDOW_FULL && p->window_size < 1) return SPITE_BAD_ARG;
+    if (!distance_bias_ok(p)) return SPITE_BAD_ARG;
     if (x->n_splits < 1 || x->n_segments < 1 || x->tokens_per_block < 1 || n_blocks < 0) return SPITE_BAD_ARG;
     if (c->n_pages < 1 || c->page_size < 1 || n_stages < 2 || n_stages > MAX_STAGES) return SPITE_BAD_ARG;
     const int G = p->num_heads / c->num_kv_heads;

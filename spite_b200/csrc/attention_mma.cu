@@ -53,7 +53,7 @@ __device__ __forceinline__ unsigned pack_bf16(float a, float b) {
 }
 
 // NK = head_dim / 16
-template <int NK, bool CAP>
+template <int NK, int FORM>
 __global__ void __launch_bounds__(WARPS * 32) attn_mma_kernel(const AttentionParams p, const StepTokens b,
                                                               const PagedCache c, const AttnMmaExtra x) {
     constexpr int HD = 16 * NK;
@@ -85,6 +85,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_mma_kernel(const AttentionPar
     // the two rows of this lane: g and g + 8
     int row_pos[2], row_lo[2];
     float row_slope[2];                                     // what a key costs per position of distance (0: no bias)
+    const float* row_dist[2];                               // what a key adds by its distance (null: nothing)
     bool row_ok[2];
     const __nv_bfloat16* qrow[2];
 #pragma unroll
@@ -95,6 +96,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_mma_kernel(const AttentionPar
         const int head = kvh * G + (row_ok[h] ? r % G : 0);
         row_pos[h] = b.positions[tok];
         row_slope[h] = slope_of(p, head);
+        row_dist[h] = distance_row_of(p, head);
         row_lo[h] = window_lowest(p.window_kind, p.window_size, row_pos[h]);
         qrow[h] = (const __nv_bfloat16*)p.q + ((size_t)tok * nq + head) * HD;
     }
@@ -190,7 +192,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_mma_kernel(const AttentionPar
                 for (int e = 0; e < 2; ++e) {
                     const int j = j0 + 8 * n + 2 * cc + e;
                     const bool ok = row_ok[h] && j >= row_lo[h] && j <= row_pos[h];
-                    const float v = ok ? capped_if<CAP>(p, s[n][2 * h + e] * p.softmax_scale) - row_slope[h] * (float)(row_pos[h] - j) : -INFINITY;
+                    const float v = ok ? score_of<FORM>(p, s[n][2 * h + e] * p.softmax_scale, row_slope[h], row_dist[h], row_pos[h] - j) : -INFINITY;
                     s[n][2 * h + e] = v;
                     mx = fmaxf(mx, v);
                 }
@@ -340,7 +342,8 @@ int launch(const AttentionParams& p, const StepTokens& b, const PagedCache& c, c
     const size_t tiles = (size_t)WARPS * 4 * TILE * 16 * NK * 2;
     const size_t merge = (size_t)WARPS * 16 * 16 * NK * 4 + WARPS * 16 * 2 * 4;
     const size_t smem = tiles > merge ? tiles : merge;
-    auto k = p.score_softcap > 0.f ? attn_mma_kernel<NK, true> : attn_mma_kernel<NK, false>;
+    const int form = score_form_of(p);
+    auto k = form == FORM_DISTANCE ? attn_mma_kernel<NK, FORM_DISTANCE> : form == FORM_CAP ? attn_mma_kernel<NK, FORM_CAP> : attn_mma_kernel<NK, FORM_PLAIN>;
     if (smem > 48 * 1024 &&
         cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
         return SPITE_LAUNCH_FAILED;
@@ -362,6 +365,7 @@ SPITE_API int spite_paged_attention_mma(const AttentionParams* p, const StepToke
     if (p->num_heads < 1 || c->num_kv_heads < 1 || p->num_heads % c->num_kv_heads) return SPITE_BAD_ARG;
     if (p->window_kind < 0 || p->window_kind > 2) return SPITE_BAD_ARG;
     if (p->window_kind != SPITE_WINDOW_FULL && p->window_size < 1) return SPITE_BAD_ARG;
+    if (!distance_bias_ok(p)) return SPITE_BAD_ARG;
     if (x->n_splits < 1 || x->n_segments < 1 || x->tokens_per_block < 1 || n_blocks < 0) return SPITE_BAD_ARG;
     const int G = p->num_heads / c->num_kv_heads;
     if (c->head_dim % 16 || c->head_dim > 128 || G > 16 || c->page_size % 16) return SPITE_UNSUPPORTED;

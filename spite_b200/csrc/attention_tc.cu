@@ -81,7 +81,7 @@ __device__ __forceinline__ unsigned pack_bf16(float a, float b) {
 }
 
 // NKB = head_dim / 64.  grid (blocks over (request, pair of token tiles), kv heads).
-template <int NKB, bool CAP>
+template <int NKB, int FORM>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                const __grid_constant__ CUtensorMap map_v, const AttentionParams p, const StepTokens b,
@@ -309,6 +309,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 // a cap on the scaled scores, in units of the raw ones; the argument of 2^x that gives e^(2 s scale / cap)
                 const float cap_raw = p.score_softcap > 0.f ? p.score_softcap / p.softmax_scale : 0.f;
                 const float cap_arg = p.score_softcap > 0.f ? 2.f * LOG2E * p.softmax_scale / p.score_softcap : 0.f;
+                // a number per distance, brought into the units of the raw scores as it is added
+                const float* dist_row = FORM == FORM_DISTANCE ? distance_row_of(p, head) : nullptr;
+                const float per_scale = 1.f / p.softmax_scale;
                 const unsigned lane_base = tmem_g + ((unsigned)(quarter * 32) << 16);
                 float m_ref = -INFINITY, l = 0.f;
                 bool ok = true;
@@ -326,8 +329,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                     // The bias of key j0 + e is bias_raw * (j0 - pos) + bias_raw * e: the second term is one multiply-add an
                     // element with a constant that the compiler knows; the first is the same for the whole tile and joins
                     // the maximum and the exponent's offset below.
-                    const float tile_bias = biased ? bias_raw * (float)(j0 - pos) : 0.f;
-                    if constexpr (CAP) {
+                    float tile_bias = biased ? bias_raw * (float)(j0 - pos) : 0.f;
+                    if (FORM == FORM_CAP || (FORM == FORM_DISTANCE && cap_raw > 0.f)) {
                         // cap tanh(s scale / cap) in units of the raw scores: tanh(x) = 1 - 2 / (e^(2x) + 1), whose absolute
                         // error (a few float32 roundings of a number below one) times the cap is far below a bfloat16 weight's
 #pragma unroll
@@ -337,6 +340,20 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                     if (biased) {
 #pragma unroll
                         for (int e = 0; e < BN; ++e) s[e] = fmaf(bias_raw, (float)e, s[e]);
+                    }
+                    if constexpr (FORM == FORM_DISTANCE) {
+                        // The numbers change with the distance near the query and hardly further away: where every row of the
+                        // warp has one number for its whole tile, that joins the tile's common term; else each key's is read
+                        // (a row's distances lie side by side, the repeated ends take the tile's overhang).
+                        const int n = pos - j0, len1 = p.distance_len - 1;       // the distance of the tile's first key
+                        const int n_hi = max(min(n, len1), 0), n_lo = max(min(n - BN + 1, len1), 0);
+                        if (__all_sync(0xffffffffu, p.distance_runs[n_hi] <= n_lo)) {
+                            tile_bias = fmaf(dist_row[n_lo], per_scale, tile_bias);
+                        } else {
+                            const float* d = dist_row + min(max(n, -1), len1 + SPITE_DISTANCE_PAD);
+#pragma unroll
+                            for (int e = 0; e < BN; ++e) s[e] = fmaf(d[-e], per_scale, s[e]);
+                        }
                     }
                     if (!open) {                                   // a tile on a window's edge or on the diagonal
 #pragma unroll
@@ -460,7 +477,8 @@ int launch(const AttentionParams& p, const StepTokens& b, const PagedCache& c, c
         if (!make_map(&mv, (const __nv_bfloat16*)c.kv + c.v_offset, 2, dims, strides, box)) return SPITE_LAUNCH_FAILED;
     }
     const size_t smem = 2 * (size_t)NKB * BM * 128 + 2 * ST * (size_t)NKB * BN * 128;
-    auto k = p.score_softcap > 0.f ? attn_tc_kernel<NKB, true> : attn_tc_kernel<NKB, false>;
+    const int form = score_form_of(p);
+    auto k = form == FORM_DISTANCE ? attn_tc_kernel<NKB, FORM_DISTANCE> : form == FORM_CAP ? attn_tc_kernel<NKB, FORM_CAP> : attn_tc_kernel<NKB, FORM_PLAIN>;
     if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
         return SPITE_LAUNCH_FAILED;
     const long long items = (long long)n_blocks * nkv;
@@ -482,6 +500,7 @@ SPITE_API int spite_paged_attention_tc(const AttentionParams* p, const StepToken
     if (p->num_heads < 1 || c->num_kv_heads < 1 || p->num_heads % c->num_kv_heads) return SPITE_BAD_ARG;
     if (p->window_kind < 0 || p->window_kind > 2) return SPITE_BAD_ARG;
     if (p->window_kind != SPITE_WINDOW_FULL && p->window_size < 1) return SPITE_BAD_ARG;
+    if (!distance_bias_ok(p)) return SPITE_BAD_ARG;
     if (x->n_segments < 1 || x->tokens_per_block < 1 || n_blocks < 0 || c->n_pages < 1 || c->page_size < 1) return SPITE_BAD_ARG;
     const int G = p->num_heads / c->num_kv_heads;
     if ((c->head_dim != 64 && c->head_dim != 128) || G > BM || c->page_size % BN) return SPITE_UNSUPPORTED;

@@ -467,22 +467,39 @@ SPITE_API int spite_rms_norm_residual(int out_dtype, const float* y, const float
     return spite_launch_status();
 }
 
-// out[m, :] (=|+=) vec: a bias that a product then adds its rows to (float32 [n_rows, d]).
-__global__ void fill_rows_kernel(float* __restrict__ out, const float* __restrict__ vec, long long n, int d, int accumulate) {
+// out[m, :] (=|+=) [other[m, :] +] vec: a bias that a product then adds its rows to, or what is mixed into the residual stream
+// between two layers (float32 [n_rows, d]; the sum in the order out, other, vec).  One block a row.
+__global__ void __launch_bounds__(256) fill_rows_kernel(float* __restrict__ out, const float* __restrict__ vec,
+                                                        const float* __restrict__ other, int d, int accumulate, int vec4) {
     pdl_wait();
     pdl_launch_dependents();
-    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
-        const float b = vec[i % d];
-        out[i] = accumulate ? out[i] + b : b;
+    const size_t row = (size_t)blockIdx.x * d;
+    if (vec4) {
+        for (int c = 4 * threadIdx.x; c < d; c += 4 * blockDim.x) {
+            float4 v = accumulate ? *(const float4*)(out + row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 b = *(const float4*)(vec + c);
+            if (other) {
+                const float4 o = *(const float4*)(other + row + c);
+                v.x += o.x; v.y += o.y; v.z += o.z; v.w += o.w;
+            }
+            v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+            *(float4*)(out + row + c) = v;
+        }
+        return;
+    }
+    for (int c = threadIdx.x; c < d; c += blockDim.x) {
+        float v = accumulate ? out[row + c] : 0.f;
+        if (other) v += other[row + c];
+        out[row + c] = v + vec[c];
     }
 }
 
-SPITE_API int spite_fill_rows(float* out, const float* vec, int n_rows, int d, int accumulate, void* stream) {
+SPITE_API int spite_fill_rows(float* out, const float* vec, const float* other, int n_rows, int d, int accumulate, void* stream) {
     if (!out || !vec || n_rows < 0 || d <= 0) return SPITE_BAD_ARG;
     if (n_rows == 0) return SPITE_OK;
-    const long long n = (long long)n_rows * d;
-    const long long blocks = (n + 255) / 256;
-    SPITE_LAUNCH(fill_rows_kernel, (int)(blocks < 8192 ? blocks : 8192), 256, 0, (cudaStream_t)stream, out, vec, n, d, accumulate);
+    const int vec4 = d % 4 == 0 && (((uintptr_t)out | (uintptr_t)vec | (uintptr_t)other) & 15) == 0;
+    const int threads = (vec4 ? d / 4 : d) > 128 ? 256 : 128;
+    SPITE_LAUNCH(fill_rows_kernel, n_rows, threads, 0, (cudaStream_t)stream, out, vec, other, d, accumulate, vec4);
     return spite_launch_status();
 }
 

@@ -104,7 +104,7 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const GemmParams p) {
             if (EPI == EPI_STORE) ((T*)p.C)[o] = from_f32<T>(finish_store(p, acc[0][i][j] * s, n));
             else if (EPI == EPI_STORE_F32) ((float*)p.C)[o] = acc[0][i][j] * s;
             else if (EPI == EPI_ADD_F32) ((float*)p.C)[o] += acc[0][i][j] * s;
-            else ((T*)p.C)[o] = from_f32<T>(silu_f32(acc[0][i][j] * s) * (acc[DUAL ? 1 : 0][i][j] * s));
+            else ((T*)p.C)[o] = from_f32<T>(gate_factor(p, acc[0][i][j] * s) * (acc[DUAL ? 1 : 0][i][j] * s));
         }
     }
 }

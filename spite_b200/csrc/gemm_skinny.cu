@@ -256,7 +256,7 @@ __global__ void __launch_bounds__(WARPS * 32, (NT <= 1 ? 2 : 1)) gemm_skinny_ker
             if (EPI == EPI_STORE) ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(finish_store(p, v * sc, n));
             else if (EPI == EPI_STORE_F32) ((float*)p.C)[o] = v * sc;
             else if (EPI == EPI_ADD_F32) ((float*)p.C)[o] += v * sc;
-            else ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(silu_f32(v * sc) * (v2 * sc));
+            else ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(gate_factor(p, v * sc) * (v2 * sc));
         }
     }
 }

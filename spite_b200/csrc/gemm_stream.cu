@@ -353,7 +353,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const GemmParams p
                 if (EPI == EPI_STORE) ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(finish_store(p, v * sc, n));
                 else if (EPI == EPI_STORE_F32) ((float*)p.C)[o] = v * sc;
                 else if (EPI == EPI_ADD_F32) ((float*)p.C)[o] += v * sc;
-                else ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(silu_f32(v * sc) * (v2 * sc));
+                else ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(gate_factor(p, v * sc) * (v2 * sc));
             };
             if (CL) {
                 // the k loops of all the cluster's blocks have ended (the first block's ring is free: the others'

@@ -289,7 +289,7 @@ gemm_tc_experts_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_c
 #pragma unroll
                     for (int t = 0; t < 32; ++t) {
                         const float s = __shfl_sync(0xffffffffu, sc, t);
-                        if (c0 + t < it.rows && n_ok) out[(size_t)t * p.ldc] = __float2bfloat16_rn(silu_f32(v[t] * s) * (u[t] * s));
+                        if (c0 + t < it.rows && n_ok) out[(size_t)t * p.ldc] = __float2bfloat16_rn(gate_factor(p, v[t] * s) * (u[t] * s));
                     }
                 } else {
                     int crow = 0;

@@ -45,7 +45,7 @@ __device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&v)[4]) {
 template <typename T>
 __global__ void __launch_bounds__(WARPS * 32) route_logits_kernel(const T* __restrict__ x, const float* __restrict__ wr,
                                                                  int n_tokens, int d, int n_experts, int experts_per_block,
-                                                                 float* __restrict__ logits) {
+                                                                 float* __restrict__ logits, const float* __restrict__ bias) {
     __shared__ float part[WARPS][EB * TB];
     pdl_wait();
     pdl_launch_dependents();
@@ -111,7 +111,7 @@ __global__ void __launch_bounds__(WARPS * 32) route_logits_kernel(const T* __res
                 float s = 0.f;
 #pragma unroll
                 for (int w = 0; w < WARPS; ++w) s += part[w][threadIdx.x];
-                logits[(size_t)(t0 + t) * n_experts + e0 + e] = s;
+                logits[(size_t)(t0 + t) * n_experts + e0 + e] = bias ? s + bias[e0 + e] : s;
             }
         }
     }
@@ -221,11 +221,11 @@ __global__ void __launch_bounds__(1024) select_and_sort_kernel(const float* __re
 
 }  // namespace
 
-// `logits` [tokens, experts] float32 is always written (the caller owns it).
+// `logits` [tokens, experts] float32 is always written (the caller owns it); `logit_bias` [experts] or null is added to them.
 SPITE_API int spite_moe_route(int dtype, const void* x, const float* w_router, int n_tokens, int d,
                               int n_experts, int top_k, int* expert_ids, float* weights,
                               float* logits, int* offsets, int* sorted_rows, int scoring, float* sorted_weights,
-                              const float* choice_bias, void* stream) {
+                              const float* choice_bias, const float* logit_bias, void* stream) {
     if (!x || !w_router || !expert_ids || !weights || !logits || !offsets || !sorted_rows) return SPITE_BAD_ARG;
     if (scoring != SCORE_SIGMOID && scoring != SCORE_SOFTMAX_RENORM && scoring != SCORE_SOFTMAX_BIASED) return SPITE_BAD_ARG;
     if (scoring == SCORE_SOFTMAX_BIASED && !choice_bias) return SPITE_BAD_ARG;
@@ -240,10 +240,10 @@ SPITE_API int spite_moe_route(int dtype, const void* x, const float* w_router, i
         if (grid.y > 65535) return SPITE_UNSUPPORTED;
         if (dtype == SPITE_DT_F32)
             SPITE_LAUNCH(route_logits_kernel<float>, grid, WARPS * 32, 0, st, (const float*)x, w_router, n_tokens, d,
-                         n_experts, per_block, logits);
+                         n_experts, per_block, logits, logit_bias);
         else if (dtype == SPITE_DT_BF16)
             SPITE_LAUNCH(route_logits_kernel<__nv_bfloat16>, grid, WARPS * 32, 0, st, (const __nv_bfloat16*)x, w_router,
-                         n_tokens, d, n_experts, per_block, logits);
+                         n_tokens, d, n_experts, per_block, logits, logit_bias);
         else
             return SPITE_BAD_ARG;
         if (cudaGetLastError() != cudaSuccess) return SPITE_LAUNCH_FAILED;

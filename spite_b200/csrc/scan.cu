@@ -1,10 +1,12 @@
 // Recurrent mixers whose state is a matrix per head that decays and takes one outer product a token, carried from token to
-// token in float32 in the request's state slot.  One walk serves two designs:
+// token in float32 in the request's state slot.  One walk serves three designs:
 //
 //   state space (Mamba-2):   dt = softplus(a + dt_bias),  S <- exp(-exp(A_log) dt) S + dt k v^T,   o = S^T q + D v
 //                            (one decay a head and token; q and k shared by a group of heads; read after the write)
 //   decaying memory (RWKV):  o = S^T q + (sum_i q_i u_i k_i) v,   S <- diag(w) S + k v^T,   w = exp(-exp(z + w0))
 //                            (a decay per key channel; the token itself enters the read-out through the bonus u)
+//   gated linear attention:  S <- diag(w) S + k v^T,   o = c S^T q,   w = sigmoid(z)^(1/tau),   z = A_2 a + b
+//                            (a decay per key channel from a short vector a; read after the write)
 //
 // S is [dim keys, vdim values], zeros at the start of a sequence.  Everything is float32.
 //
@@ -25,12 +27,14 @@ struct ScanParams {
     const float* q; const float* k; const float* v;       // first element of token 0's q, k [kv_heads * dim], v [heads * vdim]
     long long q_stride, k_stride, v_stride;               // floats between two tokens' rows
     const float* w; long long w_stride;                   // decay per key channel [tokens, heads * dim], or null: per head
-    const float* scalars;                                 // [tokens, heads, 4]: (decay, dt, -, -) without w; (bonus, -, -, -) with w
+    const float* scalars;                                 // [tokens, heads, 4]: (decay, dt, -, -) without w; (bonus, -, -, -) with w;
+                                                          // not read (null) by gated linear attention
     const float* skip;                                    // [heads] the factor D on v in the read-out, or null
     float* out; long long out_stride;                     // [tokens, heads * vdim]
     float* state; long long slot_stride;                  // state + slot * slot_stride + head * vdim * dim4
     const int* cu_seqlens; const int* slots;
     int n_segments, n_tokens, heads, kv_heads, dim, vdim;
+    float out_scale;                                      // gated linear attention: the factor c on the read-out
 };
 
 namespace {
@@ -69,8 +73,13 @@ constexpr int RING = 4;
 
 constexpr int MAX_WARPS = 4;                              // walking warps a block
 
-template <int LR, int RPV, int CC, int TB, bool CH>
+// the three designs
+enum Walk { PER_HEAD = 0, PER_CHANNEL_BONUS = 1, PER_CHANNEL = 2 };
+
+template <int LR, int RPV, int CC, int TB, int WALK>
 struct Shape {
+    static constexpr bool CH = WALK != PER_HEAD;          // a decay per key channel
+    static constexpr bool SCALARS = WALK != PER_CHANNEL;  // a token brings scalars
     static constexpr int DP = LR * RPV * 4;               // key rows a warp covers
     static constexpr int WC = 32 / LR * CC;               // value columns a warp covers
     static constexpr int ROWS = CH ? 3 : 2;               // q, k (and w) of a token
@@ -103,7 +112,7 @@ struct Bringer {
             else if (e < 2 * du) { src[s] = kp + 4 * (e - du); stride[s] = p.k_stride; dst[s] = SH::DP + 4 * (e - du); }
             else if (CH && e < 3 * du) { src[s] = wp + 4 * (e - 2 * du); stride[s] = p.w_stride; dst[s] = 2 * SH::DP + 4 * (e - 2 * du); }
             else if (e < rows + vu) { src[s] = vp + 4 * (e - rows); stride[s] = p.v_stride; dst[s] = V + 4 * (e - rows); }
-            else if (e == rows + vu) { src[s] = sp; stride[s] = 4 * p.heads; dst[s] = SH::TOKEN - 4; }
+            else if (SH::SCALARS && e == rows + vu) { src[s] = sp; stride[s] = 4 * p.heads; dst[s] = SH::TOKEN - 4; }
             if (dst[s] >= 0) src[s] += t0 * stride[s];
         }
     }
@@ -139,14 +148,15 @@ __device__ __forceinline__ void bring_elements(const ScanParams& p, const float*
             if constexpr (CH) cp_async4(d + 2 * SH::DP + e, wp + t * p.w_stride + e);
         }
         for (int e = lane; e < n_cols; e += 32) cp_async4(d + V + e, vp + t * p.v_stride + e);
-        if (lane < 2) cp_async4(d + SH::TOKEN - 4 + lane, sp + t * (4 * p.heads) + lane);
+        if (SH::SCALARS && lane < 2) cp_async4(d + SH::TOKEN - 4 + lane, sp + t * (4 * p.heads) + lane);
     }
 }
 
 // grid (ceil(vdim / (WC * warps)), heads, segments), block 32 * (warps + 1)
-template <int LR, int RPV, int CC, int TB, bool CH>
+template <int LR, int RPV, int CC, int TB, int WALK>
 __global__ void __launch_bounds__(32 * (MAX_WARPS + 1)) scan_kernel(const ScanParams p, const int wide) {
-    using SH = Shape<LR, RPV, CC, TB, CH>;
+    using SH = Shape<LR, RPV, CC, TB, WALK>;
+    constexpr bool CH = SH::CH;
     constexpr int DP = SH::DP, WC = SH::WC, NP = RPV * 2, TOKEN = SH::TOKEN, V = SH::ROWS * DP;
     extern __shared__ __align__(16) float ring[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = (blockDim.x >> 5) - 1;
@@ -179,7 +189,7 @@ __global__ void __launch_bounds__(32 * (MAX_WARPS + 1)) scan_kernel(const ScanPa
         const float* kp = p.k + (size_t)kvh * dim;
         const float* vp = p.v + (size_t)head * vdim + c0;
         const float* wp = CH ? p.w + (size_t)head * dim : nullptr;
-        const float* sp = p.scalars + 4 * head;
+        const float* sp = SH::SCALARS ? p.scalars + 4 * head : nullptr;
         const auto pump = [&](auto&& bring) {             // bring(batch): starts its copies
 #pragma unroll 1
             for (int b = 0; b < RING - 1; ++b) { bring(b); cp_commit(); }
@@ -249,9 +259,12 @@ __global__ void __launch_bounds__(32 * (MAX_WARPS + 1)) scan_kernel(const ScanPa
             f2 acc = 0;
 #pragma unroll
             for (int i = 0; i < NP; ++i) {
-                if constexpr (CH) {
+                if constexpr (WALK == PER_CHANNEL_BONUS) {
                     acc = fma2(q[i], S[i][c], acc);
                     S[i][c] = fma2(w[i], S[i][c], mul2(k[i], v2));
+                } else if constexpr (WALK == PER_CHANNEL) {
+                    S[i][c] = fma2(w[i], S[i][c], mul2(k[i], v2));
+                    acc = fma2(q[i], S[i][c], acc);
                 } else {
                     S[i][c] = fma2(k[i], v2, mul2(decay, S[i][c]));
                     acc = fma2(q[i], S[i][c], acc);
@@ -298,7 +311,8 @@ __global__ void __launch_bounds__(32 * (MAX_WARPS + 1)) scan_kernel(const ScanPa
             const int num = r * SH::KEEP + i, tt = num / CC, c = num % CC;
             if (tt < left && j0 + c < n_cols) {
                 const float* tok = in + tt * TOKEN;
-                out[(long long)tt * p.out_stride + c] = fmaf(CH ? tok[TOKEN - 4] : skip, tok[V + j0 + c], o[i]);
+                out[(long long)tt * p.out_stride + c] =
+                    WALK == PER_CHANNEL ? p.out_scale * o[i] : fmaf(CH ? tok[TOKEN - 4] : skip, tok[V + j0 + c], o[i]);
             }
         }
         out += TB * p.out_stride;
@@ -358,15 +372,55 @@ __global__ void __launch_bounds__(128) memory_gates_kernel(float* __restrict__ w
     if (lane == 0) *(float4*)(scalars + 4 * row) = make_float4(s, 0.f, 0.f, 0.f);
 }
 
-template <int LR, int RPV, int CC, int TB, bool CH>
+// gated linear attention: w[t, c] = sigmoid(z)^(1/tau) with z = sum_r a[t, r] A_2[r, c] + b[c] for the channels c of all heads.
+// A thread has one channel of DECAY_TOKENS tokens; the sum runs over r in ascending order.
+constexpr int DECAY_TOKENS = 8, DECAY_RANK = 64;          // (the short vectors of a block's tokens pass through in pieces)
+__global__ void __launch_bounds__(128) channel_decays_kernel(const float* __restrict__ a, long long a_stride, const float* __restrict__ a2,
+                                                             const float* __restrict__ b, float* __restrict__ w, long long w_stride,
+                                                             int n_tokens, int n, int rank, float inv_tau) {
+    __shared__ float a_s[DECAY_TOKENS][DECAY_RANK];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int c = blockIdx.x * 128 + threadIdx.x, t0 = blockIdx.y * DECAY_TOKENS, nt = min(DECAY_TOKENS, n_tokens - t0);
+    float z[DECAY_TOKENS];
+#pragma unroll
+    for (int t = 0; t < DECAY_TOKENS; ++t) z[t] = 0.f;
+    for (int r0 = 0; r0 < rank; r0 += DECAY_RANK) {
+        const int nr = min(DECAY_RANK, rank - r0);
+        if (r0 > 0) __syncthreads();
+        for (int e = threadIdx.x; e < DECAY_TOKENS * nr; e += 128) {
+            const int t = e / nr, r = e % nr;
+            a_s[t][r] = t < nt ? a[(long long)(t0 + t) * a_stride + r0 + r] : 0.f;
+        }
+        __syncthreads();
+        if (c < n) {
+#pragma unroll 4
+            for (int r = 0; r < nr; ++r) {
+                const float v = a2[(size_t)(r0 + r) * n + c];
+#pragma unroll
+                for (int t = 0; t < DECAY_TOKENS; ++t) z[t] = fmaf(a_s[t][r], v, z[t]);
+            }
+        }
+    }
+    if (c >= n) return;
+    const float bias = b[c];
+#pragma unroll
+    for (int t = 0; t < DECAY_TOKENS; ++t) {
+        if (t >= nt) break;
+        const float y = z[t] + bias;                      // log sigmoid(y) = -(max(-y, 0) + log(1 + e^-|y|))
+        w[(long long)(t0 + t) * w_stride + c] = expf(-inv_tau * (fmaxf(-y, 0.f) + log1pf(expf(-fabsf(y)))));
+    }
+}
+
+template <int LR, int RPV, int CC, int TB, int WALK>
 int launch_scan(const ScanParams& p, int wide, cudaStream_t st) {
-    using SH = Shape<LR, RPV, CC, TB, CH>;
+    using SH = Shape<LR, RPV, CC, TB, WALK>;
     // four walking warps a block, fewer where a step has so few (segment, head) pairs that more and smaller blocks spread better
     int warps = MAX_WARPS;
     while (warps > 1 && ((long long)((p.vdim + SH::WC * warps - 1) / (SH::WC * warps)) * p.heads * p.n_segments < 148 ||
                          SH::WC * (warps / 2) >= p.vdim)) warps /= 2;
     const size_t bytes = (size_t)RING * TB * SH::TOKEN * sizeof(float);
-    auto kernel = scan_kernel<LR, RPV, CC, TB, CH>;
+    auto kernel = scan_kernel<LR, RPV, CC, TB, WALK>;
     if (bytes > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess)
         return SPITE_LAUNCH_FAILED;
     dim3 grid((p.vdim + SH::WC * warps - 1) / (SH::WC * warps), p.heads, p.n_segments);
@@ -377,20 +431,21 @@ int launch_scan(const ScanParams& p, int wide, cudaStream_t st) {
     return spite_launch_status();
 }
 
-template <bool CH>
+template <int WALK>
 int choose_scan(const ScanParams& p, cudaStream_t st) {
+    constexpr bool CH = WALK != PER_HEAD;
     const auto al = [](const void* x) { return ((uintptr_t)x & 15) == 0; };
     const int wide = p.dim % 4 == 0 && p.vdim % 4 == 0 && p.q_stride % 4 == 0 && p.k_stride % 4 == 0 && p.v_stride % 4 == 0 &&
-                     al(p.q) && al(p.k) && al(p.v) && al(p.scalars) && (!CH || (p.w_stride % 4 == 0 && al(p.w)));
-    if (p.dim <= 32) return launch_scan<8, 1, 2, 8, CH>(p, wide, st);
-    if (p.dim <= 64) return launch_scan<8, 2, 2, 8, CH>(p, wide, st);
-    if (p.dim <= 128) return launch_scan<8, 4, 2, 8, CH>(p, wide, st);
-    if (p.dim <= 256) return launch_scan<16, 4, 2, 8, CH>(p, wide, st);
-    return launch_scan<32, 4, 4, 8, CH>(p, wide, st);
+                     al(p.q) && al(p.k) && al(p.v) && (WALK == PER_CHANNEL || al(p.scalars)) && (!CH || (p.w_stride % 4 == 0 && al(p.w)));
+    if (p.dim <= 32) return launch_scan<8, 1, 2, 8, WALK>(p, wide, st);
+    if (p.dim <= 64) return launch_scan<8, 2, 2, 8, WALK>(p, wide, st);
+    if (p.dim <= 128) return launch_scan<8, 4, 2, 8, WALK>(p, wide, st);
+    if (p.dim <= 256) return launch_scan<16, 4, 2, 8, WALK>(p, wide, st);
+    return launch_scan<32, 4, 4, 8, WALK>(p, wide, st);
 }
 
 int check_scan(const ScanParams* p) {
-    if (!p || !p->q || !p->k || !p->v || !p->out || !p->state || !p->cu_seqlens || !p->slots || !p->scalars) return SPITE_BAD_ARG;
+    if (!p || !p->q || !p->k || !p->v || !p->out || !p->state || !p->cu_seqlens || !p->slots) return SPITE_BAD_ARG;
     if (p->n_segments < 0 || p->n_tokens < 0 || p->heads < 1 || p->kv_heads < 1 || p->heads % p->kv_heads || p->dim < 1 || p->vdim < 1)
         return SPITE_BAD_ARG;
     const long long dim4 = (p->dim + 3) & ~3;
@@ -408,20 +463,20 @@ SPITE_API int spite_state_space_scan(const ScanParams* p, const float* a, long l
                                      const float* dt_bias, void* stream) {
     const int chk = check_scan(p);
     if (chk != SPITE_OK) return chk;
-    if (!a || !a_log || !dt_bias || p->w || a_stride < p->heads) return SPITE_BAD_ARG;
+    if (!a || !a_log || !dt_bias || !p->scalars || p->w || a_stride < p->heads) return SPITE_BAD_ARG;
     if (p->n_segments == 0 || p->n_tokens == 0) return SPITE_OK;
     cudaStream_t st = (cudaStream_t)stream;
     const long long n = (long long)p->n_tokens * p->heads;
     SPITE_LAUNCH(state_space_gates_kernel, (int)((n + 127) / 128), 128, 0, st, a, a_stride, a_log, dt_bias, (float*)p->scalars, n, p->heads);
     if (cudaGetLastError() != cudaSuccess) return SPITE_LAUNCH_FAILED;
-    return choose_scan<false>(*p, st);
+    return choose_scan<PER_HEAD>(*p, st);
 }
 
 // p->w holds the decay's pre-activations on entry and the decays afterwards; `u` and `w0` [heads * dim]
 SPITE_API int spite_decay_scan(const ScanParams* p, const float* w0, const float* u, void* stream) {
     const int chk = check_scan(p);
     if (chk != SPITE_OK) return chk;
-    if (!w0 || !u || !p->w || p->w_stride < (long long)p->heads * p->dim || p->kv_heads != p->heads || p->skip) return SPITE_BAD_ARG;
+    if (!w0 || !u || !p->scalars || !p->w || p->w_stride < (long long)p->heads * p->dim || p->kv_heads != p->heads || p->skip) return SPITE_BAD_ARG;
     if (p->n_segments == 0 || p->n_tokens == 0) return SPITE_OK;
     cudaStream_t st = (cudaStream_t)stream;
     const long long rows = (long long)p->n_tokens * p->heads;
@@ -429,5 +484,23 @@ SPITE_API int spite_decay_scan(const ScanParams* p, const float* w0, const float
     SPITE_LAUNCH(memory_gates_kernel, (int)((rows + 3) / 4), 128, 0, st, (float*)p->w, p->w_stride, w0, p->q, p->q_stride, p->k,
                  p->k_stride, u, (float*)p->scalars, rows, p->heads, p->dim);
     if (cudaGetLastError() != cudaSuccess) return SPITE_LAUNCH_FAILED;
-    return choose_scan<true>(*p, st);
+    return choose_scan<PER_CHANNEL_BONUS>(*p, st);
+}
+
+// p->w [tokens, heads * dim] receives the decays, from the short vectors `a` [tokens, rank] (rows of a_stride), `a2` [rank,
+// heads * dim] and `b` [heads * dim]
+SPITE_API int spite_gated_linear_scan(const ScanParams* p, const float* a, long long a_stride, const float* a2, const float* b,
+                                      int rank, float tau, void* stream) {
+    const int chk = check_scan(p);
+    if (chk != SPITE_OK) return chk;
+    if (!a || !a2 || !b || rank < 1 || a_stride < rank || !(tau > 0.f) || !(p->out_scale == p->out_scale)) return SPITE_BAD_ARG;
+    if (!p->w || p->w_stride < (long long)p->heads * p->dim || p->kv_heads != p->heads || p->skip) return SPITE_BAD_ARG;
+    if (p->n_segments == 0 || p->n_tokens == 0) return SPITE_OK;
+    cudaStream_t st = (cudaStream_t)stream;
+    const int n = p->heads * p->dim;
+    dim3 grid((n + 127) / 128, (p->n_tokens + DECAY_TOKENS - 1) / DECAY_TOKENS);
+    if (grid.y > 65535) return SPITE_UNSUPPORTED;
+    SPITE_LAUNCH(channel_decays_kernel, grid, 128, 0, st, a, a_stride, a2, b, (float*)p->w, p->w_stride, p->n_tokens, n, rank, 1.f / tau);
+    if (cudaGetLastError() != cudaSuccess) return SPITE_LAUNCH_FAILED;
+    return choose_scan<PER_CHANNEL>(*p, st);
 }

@@ -37,6 +37,32 @@ class Routing:
     sorted_weights: Optional[torch.Tensor] = None   # [k, M] float32: weights[slot][sorted_rows[slot][i]] at place i
 
 
+@dataclass(frozen=True)
+class DistanceBias:
+    """A number per head and distance for attention scores: head h's score of a key n positions before the query gets
+    padded[h, PAD + min(n, length - 1)].  The rows' ends are repeated PAD times on either side (a kernel reads whole tiles of
+    keys around them); `runs`[n] is the smallest distance from which up to n every head's number stays the same."""
+    PAD = 64
+    padded: torch.Tensor         # float32 [heads, PAD + length + PAD]
+    runs: torch.Tensor           # int32 [length]
+
+    @property
+    def length(self) -> int:
+        return self.runs.numel()
+
+    @classmethod
+    def from_rows(cls, table: torch.Tensor, row_of: list) -> "DistanceBias":
+        """`table` [rows, heads]: row row_of[n] serves distance n, the last entry every distance from there on."""
+        dev = table.device
+        index = torch.tensor([row_of[0]] * cls.PAD + list(row_of) + [row_of[-1]] * cls.PAD, dtype=torch.long, device=dev)
+        runs, start = [], 0
+        for n, row in enumerate(row_of):
+            if n and row != row_of[n - 1]:
+                start = n
+            runs.append(start)
+        return cls(table.to(torch.float32)[index].t().contiguous(), torch.tensor(runs, dtype=torch.int32, device=dev))
+
+
 class KernelSet:
     """Interface; see `CudaKernels` for the product implementation."""
 
@@ -92,8 +118,9 @@ class KernelSet:
         With one tap nothing is carried and `state` may be None."""
         raise NotImplementedError
 
-    def fill_rows(self, out, vec, *, accumulate=False):
-        """out[m, :] (float32 [M, d]) = vec (float32 [d]), or += vec: a bias laid down for a product that adds to it."""
+    def fill_rows(self, out, vec, *, accumulate=False, other=None):
+        """out[m, :] (float32 [M, d]) = vec (float32 [d]), or += vec: a bias laid down for a product that adds to it.  `other`
+        (float32 [M, d]) is added row by row ahead of the vector."""
         raise NotImplementedError
 
     def head_norm_gate(self, x, out, *, heads, size, gates=None, gate_column=0, gain=None, eps=None, gate_activation="sigmoid",
@@ -102,7 +129,8 @@ class KernelSet:
         result of a recurrence), out [M, heads * size] (T; may be x):
         out[m, h, j] = x[m, h, j] * r * gain[h * size + j] * sigmoid(gates[m, gate_column + h * size + j]) with
         r = rsqrt(mean_j x[m, h, :]^2 + eps) if `eps` is given (a norm of every head without a gain of its own), else 1;
-        `gates` (a 2-D tensor of x's type, the gate columns of a wider product) and `gain` (float32) may be left out.
+        `gates` (a 2-D tensor of x's type, the gate columns of a wider product) and `gain` (float32) may be left out; a gain
+        of `size` elements is shared by the heads.
         `gate_activation` "silu": the factor is z * sigmoid(z) of the gate column z instead of sigmoid(z).
         `out_column` c: out is a wider 2-D tensor and the result goes into its columns from c on."""
         raise NotImplementedError
@@ -152,8 +180,9 @@ class KernelSet:
         on the device holds g * M."""
         raise NotImplementedError
 
-    def linear_swiglu(self, x, w_gate_up, out, *, row_scale=None):
-        """out[M, F] (T) = silu(s g) * (s u) with g = x @ w[:F]^T, u = x @ w[F:]^T, s = row_scale or 1."""
+    def linear_swiglu(self, x, w_gate_up, out, *, row_scale=None, activation="silu"):
+        """out[M, F] (T) = silu(s g) * (s u) with g = x @ w[:F]^T, u = x @ w[F:]^T, s = row_scale or 1; `activation`
+        "gelu_tanh": the gate's function is gelu in its tanh form (as in `linear`) instead of silu."""
         raise NotImplementedError
 
     def grouped_linear_swiglu(self, x, w_gate_up, sorted_rows, offsets, row_scale, out):
@@ -187,7 +216,8 @@ class KernelSet:
 
     # ---- attention
     def qk_prepare(self, qkv, q_out, batch, cache, *, num_heads, rotation, qk_norm, temperature,
-                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None, value_rotation=None):
+                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None, value_rotation=None,
+                   values_are_keys=False):
         """Encode positions of q and k, normalise, scale q, append k and v to the cache.
         `bias` float32 [(nq + 2 nkv) hd]: added to the projection's columns before anything else.  `q_only`: a row of
         qkv holds the q heads alone (and `bias` theirs): the layer reads keys and values that another layer cached.
@@ -201,12 +231,13 @@ class KernelSet:
         `norm_dim`: a q or k head has this many elements and zeros behind them up to hd (a cache row wider than the key):
         the per-head norm takes its mean over them.
         `value_rotation`: a `parts.Rotation` over the leading elements of a value head: a value turns by its own position
-        before it is cached."""
+        before it is cached.  `values_are_keys`: a row of qkv holds q and k heads alone ((nq + nkv) hd columns, `bias` too),
+        and the value of a position is its key as projected (with its bias, before norm and rotation)."""
         raise NotImplementedError
 
     def paged_attention(self, q, out, batch, cache, *, num_heads, window, softmax_scale, cache_settled=False,
                         sink_logit=None, head_sinks=None, head_slopes=None, head_gates=None, out_by_head=False,
-                        score_softcap=None):
+                        score_softcap=None, distance_bias=None):
         """out[M, nq hd] = softmax(q K^T * scale over the visible cached keys) V.
         `score_softcap` c: a scaled score s becomes c * tanh(s / c) before anything else happens to it.
         `out_by_head`: the result is laid out head by head instead, out[nq, M, hd] (the order in which a product per
@@ -214,6 +245,7 @@ class KernelSet:
         `sink_logit`: the softmax's denominator also holds exp(sink_logit), a key without a value;
         `head_sinks` float32 [nq]: the same with a score of its own for every head.
         `head_slopes` float32 [nq]: slope_h * (query position - key position) is taken off head h's scores.
+        `distance_bias`, a `DistanceBias`: a number per head and distance is added to a score (behind scale and cap).
         `head_gates` float32 [M, nq]: head h's output for token m is multiplied by head_gates[m, h].
         A cache with one plane (`cache.kv.shape[0] == 1`) holds keys only, and the value of a position is its key row.
         `cache_settled`: the caller promises that the cache rows of positions before each request's first
@@ -294,6 +326,13 @@ class KernelSet:
         overwritten with the decays; w0, u float32 [heads * dim]."""
         raise NotImplementedError
 
+    def gated_linear_scan(self, q, k, v, a, w, out, batch, state, *, heads, dim, vdim, a2, a2_bias, tau, q_scale, state_offset=0):
+        """Gated linear attention, walked and kept as above: S <- diag(w) S + k v^T, then out = q_scale S^T q, with the decays
+        w = sigmoid(a A_2 + a2_bias)^(1 / tau) per head and key channel made first.  q, k, v and a (the short vectors of
+        a2.shape[0] elements) are pairs (float32 tensor, first column); a2 float32 [rank, heads * dim] (input-major), a2_bias
+        float32 [heads * dim]; w float32 [M, heads * dim] receives the decays."""
+        raise NotImplementedError
+
     # ---- mixture of experts
     def moe_identity(self, x, routing, first_identity, out, *, accumulate=True):
         """Experts that return their input: out[m, :] (float32) (+)= sum over the choice slots s whose expert id
@@ -301,8 +340,8 @@ class KernelSet:
         every row of out is written (zeros where no such expert was chosen)."""
         raise NotImplementedError
 
-    def moe_route(self, x, w_router, top_k, want_logits=False, scoring="sigmoid", choice_bias=None) -> Routing:
-        """Router logits in float32, the `top_k` largest per token (equal ones: the lower expert first), the
+    def moe_route(self, x, w_router, top_k, want_logits=False, scoring="sigmoid", choice_bias=None, logit_bias=None) -> Routing:
+        """Router logits in float32 (plus `logit_bias`, float32 [E], if given), the `top_k` largest per token (equal ones: the lower expert first), the
         tokens sorted by expert for every choice slot.  `scoring` "sigmoid": the weight of a choice is the sigmoid
         of its logit; "softmax_renorm": its share of the softmax over all experts, divided by the sum of the
         chosen shares (+ 1e-20); `sorted_weights` is filled for it.  "softmax_biased": the experts are ordered by their

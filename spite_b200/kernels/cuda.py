@@ -54,7 +54,7 @@ class QkPrepareParams(C.Structure):
                 ("v_mix_dim", C.c_int), ("v_mix", C.c_float), ("gates_out", C.c_void_p),
                 ("bias", C.c_void_p), ("q_only", C.c_int), ("norm_dim", C.c_int),
                 ("v_inv_freq", C.c_void_p), ("v_rotary_dim", C.c_int), ("v_pairing", C.c_int),
-                ("inv_freq_low", C.c_void_p), ("v_inv_freq_low", C.c_void_p)]
+                ("inv_freq_low", C.c_void_p), ("v_inv_freq_low", C.c_void_p), ("values_are_keys", C.c_int)]
 
 
 class AttentionParams(C.Structure):
@@ -62,7 +62,8 @@ class AttentionParams(C.Structure):
                 ("window_kind", C.c_int), ("window_size", C.c_int), ("softmax_scale", C.c_float),
                 ("has_sink", C.c_int), ("sink_logit", C.c_float),
                 ("head_sinks", C.c_void_p), ("head_slopes", C.c_void_p), ("head_gates", C.c_void_p),
-                ("out_by_head_tokens", C.c_int), ("score_softcap", C.c_float)]
+                ("out_by_head_tokens", C.c_int), ("score_softcap", C.c_float),
+                ("distance_bias", C.c_void_p), ("distance_runs", C.c_void_p), ("distance_len", C.c_int)]
 
 
 class LatentPrepareParams(C.Structure):
@@ -108,7 +109,7 @@ class ScanParams(C.Structure):
                 ("w", C.c_void_p), ("w_stride", C.c_longlong), ("scalars", C.c_void_p), ("skip", C.c_void_p),
                 ("out", C.c_void_p), ("out_stride", C.c_longlong), ("state", C.c_void_p), ("slot_stride", C.c_longlong),
                 ("cu_seqlens", C.c_void_p), ("slots", C.c_void_p), ("n_segments", C.c_int), ("n_tokens", C.c_int),
-                ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int)]
+                ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("out_scale", C.c_float)]
 
 
 class DeltaParams(C.Structure):
@@ -476,13 +477,15 @@ class CudaKernels(KernelSet):
         self._count("elementwise", 1)
         _check(st, "short_conv")
 
-    def fill_rows(self, out, vec, *, accumulate=False):
+    def fill_rows(self, out, vec, *, accumulate=False, other=None):
         self._t(out, torch.float32, "out"); self._t(vec, torch.float32, "vec")
         M, d = out.shape
         if vec.numel() != d:
             raise KernelError("fill_rows: the vector must have the rows' width")
-        st = self._lib("elementwise").spite_fill_rows(C.c_void_p(out.data_ptr()), C.c_void_p(vec.data_ptr()), M, d,
-                                                      int(bool(accumulate)), self._stream())
+        if other is not None and self._t(other, torch.float32, "other").shape != out.shape:
+            raise KernelError("fill_rows: what is added row by row must have the output's shape")
+        st = self._lib("elementwise").spite_fill_rows(C.c_void_p(out.data_ptr()), C.c_void_p(vec.data_ptr()), C.c_void_p(_ptr(other)),
+                                                      M, d, int(bool(accumulate)), self._stream())
         self._count("elementwise", 1)
         _check(st, "fill_rows")
 
@@ -503,12 +506,12 @@ class CudaKernels(KernelSet):
             if gates.dim() != 2 or gates.shape[0] != M or gate_column < 0 or gate_column + heads * size > gates.shape[1]:
                 raise KernelError("head_norm_gate: the gate columns do not fit")
             g_ptr, g_stride = gates.data_ptr() + int(gate_column) * gates.element_size(), gates.shape[1]
-        if gain is not None and self._t(gain, torch.float32, "gain").numel() != heads * size:
-            raise KernelError("head_norm_gate: the gain must have heads * size elements")
+        if gain is not None and self._t(gain, torch.float32, "gain").numel() not in (heads * size, size):
+            raise KernelError("head_norm_gate: the gain must have heads * size elements, or a head's")
         st = self._lib("elementwise").spite_head_norm_gate(
             _DT[x.dtype], self._dt, C.c_void_p(x.data_ptr()), C.c_void_p(g_ptr), C.c_longlong(g_stride),
             C.c_void_p(_ptr(gain)), C.c_void_p(o_ptr), C.c_longlong(out.shape[1]), M, int(heads), int(size), C.c_float(eps or 0.0),
-            int(gate_activation == "silu"), 1, self._stream())
+            int(gate_activation == "silu"), int(gain is not None and gain.numel() == heads * size), self._stream())
         self._count("elementwise", 1)
         _check(st, "head_norm_gate")
 
@@ -758,15 +761,18 @@ class CudaKernels(KernelSet):
                        bias=_ptr(bias), act_pos=float(pos), act_neg=float(neg))
         self._gemm(p, "linear", M)
 
-    def linear_swiglu(self, x, w_gate_up, out, *, row_scale=None):
+    def linear_swiglu(self, x, w_gate_up, out, *, row_scale=None, activation="silu"):
         self._t(x, self.dtype, "x"); self._t(w_gate_up, self.dtype, "w"); self._t(out, self.dtype, "out")
         M, K = x.shape
         F = w_gate_up.shape[0] // 2
         if w_gate_up.shape != (2 * F, K) or tuple(out.shape) != (M, F):
             raise KernelError("linear_swiglu: shapes do not fit")
+        if activation not in ("silu", "gelu_tanh"):
+            raise KernelError(f"linear_swiglu: unknown gate function {activation!r}")
         p = GemmParams(A=x.data_ptr(), W=w_gate_up.data_ptr(), C=out.data_ptr(), a_rows=None, c_rows=None,
                        group_offsets=None, row_scale=_ptr(row_scale), lda=K, ldc=F, w_group_stride=0,
-                       n_groups=1, M=M, N=F, K=K, epilogue=EPI_SWIGLU, scale_by_a_row=0)
+                       n_groups=1, M=M, N=F, K=K, epilogue=EPI_SWIGLU, scale_by_a_row=0,
+                       activation=0 if activation == "silu" else _ACTIVATION[activation])
         self._gemm(p, "linear_swiglu", M)
 
     def grouped_linear_swiglu(self, x, w_gate_up, sorted_rows, offsets, row_scale, out):
@@ -854,10 +860,13 @@ class CudaKernels(KernelSet):
                           page_size=kv.shape[3], num_kv_heads=kv.shape[2], head_dim=kv.shape[4])
 
     def qk_prepare(self, qkv, q_out, batch, cache, *, num_heads, rotation, qk_norm, temperature,
-                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None, value_rotation=None):
+                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None, value_rotation=None,
+                   values_are_keys=False):
         self._t(qkv, self.dtype, "qkv"); self._t(q_out, self.dtype, "q_out")
         head_dim = cache.kv.shape[4]
-        n_cols = (num_heads + (0 if q_only else 2 * cache.kv.shape[2])) * head_dim
+        if values_are_keys and (q_only or value_mix is not None or value_rotation is not None):
+            raise KernelError("qk_prepare: values that are the keys are neither borrowed, blended nor rotated")
+        n_cols = (num_heads + (0 if q_only else (1 if values_are_keys else 2) * cache.kv.shape[2])) * head_dim
         if qkv.shape[1] < n_cols:
             raise KernelError(f"qk_prepare: rows of {qkv.shape[1]} elements cannot hold the heads' {n_cols}")
         if bias is not None and self._t(bias, torch.float32, "bias").numel() != n_cols:
@@ -909,7 +918,7 @@ class CudaKernels(KernelSet):
                             v_other=v_other, v_other_stride=v_stride, v_other_head=int(v_head), v_mix_dim=int(v_dim),
                             v_mix=float(v_lam), gates_out=_ptr(gates_out), bias=_ptr(bias), q_only=int(bool(q_only)),
                             norm_dim=int(norm_dim or 0), v_inv_freq=v_freq, v_rotary_dim=v_dims, v_pairing=v_pairing,
-                            inv_freq_low=low, v_inv_freq_low=v_low)
+                            inv_freq_low=low, v_inv_freq_low=v_low, values_are_keys=int(bool(values_are_keys)))
         b, c = self._step_tokens(batch, cache.group), self._paged(cache)
         st = self._lib("attention").spite_qk_prepare(self._dt, C.byref(p), C.byref(b), C.byref(c), self._stream())
         self._count("attention", 1)
@@ -945,7 +954,7 @@ class CudaKernels(KernelSet):
 
     def paged_attention(self, q, out, batch, cache, *, num_heads, window, softmax_scale, cache_settled=False,
                         sink_logit=None, head_sinks=None, head_slopes=None, head_gates=None, out_by_head=False,
-                        score_softcap=None):
+                        score_softcap=None, distance_bias=None):
         self._t(q, self.dtype, "q"); self._t(out, self.dtype, "out")
         if score_softcap is not None and not score_softcap > 0:
             raise KernelError("paged_attention: the cap of the scores must be positive")
@@ -957,6 +966,11 @@ class CudaKernels(KernelSet):
                 raise KernelError(f"paged_attention: {name} has {t.numel()} elements, {n} are needed")
         if not softmax_scale > 0:
             raise KernelError("paged_attention: the score scale must be positive")
+        if distance_bias is not None:
+            self._t(distance_bias.runs, torch.int32, "distance_bias.runs")
+            if tuple(self._t(distance_bias.padded, torch.float32, "distance_bias.padded").shape) != \
+                    (num_heads, distance_bias.length + 2 * distance_bias.PAD):
+                raise KernelError("paged_attention: one row of numbers by distance per head")
         p = AttentionParams(q=q.data_ptr(), out=out.data_ptr(), num_heads=num_heads,
                             window_kind=_WINDOW[window.kind], window_size=int(window.size),
                             softmax_scale=float(softmax_scale),
@@ -964,6 +978,9 @@ class CudaKernels(KernelSet):
                             sink_logit=float(sink_logit or 0.0), head_sinks=_ptr(head_sinks),
                             head_slopes=_ptr(head_slopes), head_gates=_ptr(head_gates),
                             out_by_head_tokens=q.shape[0] if out_by_head else 0, score_softcap=float(score_softcap or 0.0))
+        if distance_bias is not None:
+            p.distance_bias, p.distance_runs = distance_bias.padded.data_ptr(), distance_bias.runs.data_ptr()
+            p.distance_len = distance_bias.length
         b, c = self._step_tokens(batch, cache.group), self._paged(cache)
         group = num_heads // c.num_kv_heads
         if (self.dtype == torch.bfloat16 and c.head_dim % 16 == 0 and c.head_dim <= 128 and group <= 16
@@ -1184,8 +1201,8 @@ class CudaKernels(KernelSet):
         self._count("delta", 2)
         _check(st, "delta_scan")
 
-    def _scan(self, what, q, k, v, out, batch, state, *, heads, kv_heads, dim, vdim, state_offset):
-        """The argument block that both scans share; q, k, v are (float32 tensor [M, *], first column)."""
+    def _scan(self, what, q, k, v, out, batch, state, *, heads, kv_heads, dim, vdim, state_offset, scalars=True):
+        """The argument block that the scans share; q, k, v are (float32 tensor [M, *], first column)."""
         self._t(out, torch.float32, "out"); self._t(state, torch.float32, "state")
         M = out.shape[0]
         slot_stride = state[0].numel()
@@ -1196,9 +1213,9 @@ class CudaKernels(KernelSet):
         for name, (t, column), width in (("q", q, kv_heads * dim), ("k", k, kv_heads * dim), ("v", v, heads * vdim)):
             self._t(t, torch.float32, name)
             at.append((self._columns(t, column, width, M, f"{what}: {name}"), t.shape[1]))
-        scalars = torch.empty((M, heads, 4), dtype=torch.float32, device=out.device)
+        scalars = torch.empty((M, heads, 4), dtype=torch.float32, device=out.device) if scalars else None
         p = ScanParams(q=at[0][0], k=at[1][0], v=at[2][0], q_stride=at[0][1], k_stride=at[1][1], v_stride=at[2][1],
-                       w=None, w_stride=0, scalars=scalars.data_ptr(), skip=None, out=out.data_ptr(), out_stride=out.shape[1],
+                       w=None, w_stride=0, scalars=_ptr(scalars), skip=None, out=out.data_ptr(), out_stride=out.shape[1],
                        state=state.data_ptr() + 4 * int(state_offset), slot_stride=slot_stride,
                        cu_seqlens=batch.cu_seqlens.data_ptr(), slots=batch.slots.data_ptr(),
                        n_segments=batch.cu_seqlens.numel() - 1, n_tokens=M, heads=int(heads), kv_heads=int(kv_heads),
@@ -1235,6 +1252,22 @@ class CudaKernels(KernelSet):
         self._count("scan", 2)
         _check(st, "decay_scan")
 
+    def gated_linear_scan(self, q, k, v, a, w, out, batch, state, *, heads, dim, vdim, a2, a2_bias, tau, q_scale, state_offset=0):
+        p, _ = self._scan("gated_linear_scan", q, k, v, out, batch, state, heads=heads, kv_heads=heads, dim=dim, vdim=vdim,
+                          state_offset=state_offset, scalars=False)
+        self._t(w, torch.float32, "w"); self._t(a2, torch.float32, "a2")
+        n, rank = heads * dim, a2.shape[0]
+        if tuple(w.shape) != (out.shape[0], n) or tuple(a2.shape) != (rank, n) or self._t(a2_bias, torch.float32, "a2_bias").numel() != n:
+            raise KernelError("gated_linear_scan: w is [tokens, heads * dim], a2 [rank, heads * dim], its bias [heads * dim]")
+        t, column = a
+        self._t(t, torch.float32, "a")
+        at = self._columns(t, column, rank, out.shape[0], "gated_linear_scan: a")
+        p.w, p.w_stride, p.out_scale = w.data_ptr(), n, float(q_scale)
+        st = self._lib("scan").spite_gated_linear_scan(C.byref(p), C.c_void_p(at), C.c_longlong(t.shape[1]), C.c_void_p(a2.data_ptr()),
+                                                       C.c_void_p(a2_bias.data_ptr()), int(rank), C.c_float(tau), self._stream())
+        self._count("scan", 2)
+        _check(st, "gated_linear_scan")
+
     # ------------------------------------------------------------------ mixture of experts
     def moe_identity(self, x, routing, first_identity, out, *, accumulate=True):
         self._t(x, self.dtype, "x"); self._t(out, torch.float32, "out")
@@ -1248,13 +1281,15 @@ class CudaKernels(KernelSet):
         self._count("moe", 1)
         _check(st, "moe_identity")
 
-    def moe_route(self, x, w_router, top_k, want_logits=False, scoring="sigmoid", choice_bias=None) -> Routing:
+    def moe_route(self, x, w_router, top_k, want_logits=False, scoring="sigmoid", choice_bias=None, logit_bias=None) -> Routing:
         if scoring not in ("sigmoid", "softmax_renorm", "softmax_biased"):
             raise KernelError(f"moe_route: unknown scoring {scoring!r}")
         if (scoring == "softmax_biased") != (choice_bias is not None):
             raise KernelError("moe_route: `choice_bias` goes with the scoring 'softmax_biased'")
         if choice_bias is not None and self._t(choice_bias, torch.float32, "choice_bias").numel() != w_router.shape[0]:
             raise KernelError("moe_route: one choice bias per expert")
+        if logit_bias is not None and self._t(logit_bias, torch.float32, "logit_bias").numel() != w_router.shape[0]:
+            raise KernelError("moe_route: one logit bias per expert")
         self._t(x, self.dtype, "x"); self._t(w_router, torch.float32, "w_router")
         M, d = x.shape
         E = w_router.shape[0]
@@ -1270,7 +1305,7 @@ class CudaKernels(KernelSet):
             self._dt, C.c_void_p(x.data_ptr()), C.c_void_p(w_router.data_ptr()), M, d, E, top_k,
             C.c_void_p(ids.data_ptr()), C.c_void_p(wts.data_ptr()), C.c_void_p(_ptr(logits)),
             C.c_void_p(offsets.data_ptr()), C.c_void_p(rows.data_ptr()), int(renorm), C.c_void_p(_ptr(sorted_w)),
-            C.c_void_p(_ptr(choice_bias)), self._stream())
+            C.c_void_p(_ptr(choice_bias)), C.c_void_p(_ptr(logit_bias)), self._stream())
         self._count("moe", 2)
         _check(st, "moe_route")
         return Routing(ids, wts, offsets, rows, logits if want_logits else None, sorted_w)

@@ -5,7 +5,8 @@ the query's chunk, the last W keys), the position encoding, the per-head norm of
 q and k (after or before the rotation, with gains or without), the
 temperature factor, a value size that differs from the key size, a sink in
 the softmax (an extra term exp(sink) in the sum, with nothing behind it; one score for all heads or a learned
-one per head), a bias that grows with the distance between query and key, a gate on every head's output (one
+one per head), a bias that grows with the distance between query and key, a learned number per head and bucket of distances,
+values that are the projected keys, a gate on every head's output (one
 number a head, or one for every element of the concatenated heads), biases on the four projections, the
 blending of the values with those of another layer, values cached rotated by their own position (and every head's
 result turned back by the query's), and keys and values that are not the layer's own but those
@@ -24,7 +25,9 @@ import torch
 
 from ..cache import FixedState, PagedKV, Window
 from ..config.specs import ConfigError, PartSpec
+from ..kernels.api import DistanceBias
 from .base import Mixer, ParamSpec, QkNorm, build_part, register_mixer
+from .position import distance_rows
 
 
 @register_mixer("paged_attention")
@@ -38,7 +41,7 @@ class PagedAttention(Mixer):
                  qk_norm_before_rotation=False, temperature_tuning=None, softmax_scale=None,
                  value_dim=None, sink_logit=None, head_sinks=False, distance_slopes=None, head_gate=False,
                  value_mix=None, bias=False, output_gate=False, kv_shared=False, conv_taps=None, score_softcap=None,
-                 value_rotation: PartSpec | None = None):
+                 value_rotation: PartSpec | None = None, output_bias=None, values_are_keys=False, distance_table=None):
         """`head_dim` is the size of a query and a key head, `value_dim` that of a value head (default: the
         same).  `sink_logit`, if given, is the score of a sink: a term exp(sink) in every softmax's sum that adds
         nothing to the output, p_j = exp(s_j) / (exp(sink) + sum exp(s_j')); with `head_sinks` the score is a
@@ -58,7 +61,11 @@ class PagedAttention(Mixer):
         becomes c tanh(s / c) before the softmax.
         `value_rotation`, a position part that rotates the whole value head: value j turns by its position j before it is
         cached, and a head's result at position i is turned back by i before the output projection (so a value
-        enters turned by its distance, and nothing else of the attention knows about it)."""
+        enters turned by its distance, and nothing else of the attention knows about it).
+        `output_bias` (default: as `bias`): whether the output projection has one.  `values_are_keys`: there is no value
+        projection; a position's value is its key as projected, bias included, before norm and rotation.
+        `distance_table` (rows, far): the parameter `distance_bias` [rows, heads] is added to the scores (behind scale and cap),
+        the row by the distance between query and key as `distance_rows` says."""
         super().__init__(ctx)
         self.conv_taps = None if conv_taps is None else int(conv_taps)
         if self.conv_taps is not None and (self.conv_taps < 1 or self.conv_taps > 8):
@@ -69,6 +76,12 @@ class PagedAttention(Mixer):
         if self.score_softcap is not None and not self.score_softcap > 0:
             raise ConfigError("score_softcap must be positive")
         self.has_bias, self.output_gate, self.kv_shared = bool(bias), bool(output_gate), bool(kv_shared)
+        self.has_output_bias = self.has_bias if output_bias is None else bool(output_bias)
+        self.values_are_keys = bool(values_are_keys)
+        if self.values_are_keys and (kv_shared or value_mix or conv_taps is not None or value_rotation is not None):
+            raise ConfigError("values that are the keys cannot be borrowed, blended, convolved or rotated")
+        if self.values_are_keys and value_dim not in (None, head_dim):
+            raise ConfigError(f"values that are the keys have the keys' size {head_dim}, not {value_dim}")
         if self.kv_shared and value_mix:
             raise ConfigError("a layer that reads another layer's keys and values has no values to blend")
         if self.output_gate and head_gate:
@@ -142,17 +155,31 @@ class PagedAttention(Mixer):
             temperature_tuning = (int(floor), float(scale))
         self.temperature = temperature_tuning
         self.softmax_scale = float(softmax_scale) if softmax_scale is not None else 1.0 / math.sqrt(self.kd)
+        self.distance_table = None if distance_table is None else (int(distance_table[0]), int(distance_table[1]))
+        self._distance_rows = self.distance_bias = None
+        if self.distance_table is not None:
+            rows, far = self.distance_table
+            # what lies beyond `far` shares its row; a window may end before that
+            self._distance_rows = distance_rows(rows, far, far + 1 if self.window.kind == "full" else min(self.window.size, far + 1))
         self.wqkv = self.wo = None
 
     def param_specs(self):
         d, nq, nkv, kd, vd = self.d, self.nq, self.nkv, self.kd, self.vd
         specs = {"q_proj": ParamSpec((nq * kd, d)), "o_proj": ParamSpec((d, nq * vd))}
         if not self.kv_shared:
-            specs.update({"k_proj": ParamSpec((nkv * kd, d)), "v_proj": ParamSpec((nkv * vd, d))})
+            specs["k_proj"] = ParamSpec((nkv * kd, d))
+            if not self.values_are_keys:
+                specs["v_proj"] = ParamSpec((nkv * vd, d))
         if self.has_bias:
-            specs.update({"q_bias": ParamSpec((nq * kd,)), "o_bias": ParamSpec((d,))})
+            specs["q_bias"] = ParamSpec((nq * kd,))
             if not self.kv_shared:
-                specs.update({"k_bias": ParamSpec((nkv * kd,)), "v_bias": ParamSpec((nkv * vd,))})
+                specs["k_bias"] = ParamSpec((nkv * kd,))
+                if not self.values_are_keys:
+                    specs["v_bias"] = ParamSpec((nkv * vd,))
+        if self.has_output_bias:
+            specs["o_bias"] = ParamSpec((d,))
+        if self.distance_table is not None:
+            specs["distance_bias"] = ParamSpec((self.distance_table[0], nq))
         if self.output_gate:
             specs["out_gate_proj"] = ParamSpec((nq * vd, d))
         if self.qk_norm_gain:
@@ -181,8 +208,9 @@ class PagedAttention(Mixer):
         # q, k and v rows in one matrix: one product per layer instead of three
         rows = [self._pad_heads(params["q_proj"].to(dt), self.nq, self.kd)]
         if not self.kv_shared:
-            rows += [self._pad_heads(params["k_proj"].to(dt), self.nkv, self.kd),
-                     self._pad_heads(params["v_proj"].to(dt), self.nkv, self.vd)]
+            rows.append(self._pad_heads(params["k_proj"].to(dt), self.nkv, self.kd))
+            if not self.values_are_keys:
+                rows.append(self._pad_heads(params["v_proj"].to(dt), self.nkv, self.vd))
         self.head_columns = sum(r.shape[0] for r in rows)       # the gates' columns of the product follow the heads'
         self.conv_w = None
         if self.conv_taps is not None:
@@ -198,8 +226,11 @@ class PagedAttention(Mixer):
                 return self._pad_heads(params[name].to(torch.float32).reshape(-1, 1), heads, size).reshape(-1)
             cols = [column("q_bias", self.nq, self.kd)]
             if not self.kv_shared:
-                cols += [column("k_bias", self.nkv, self.kd), column("v_bias", self.nkv, self.vd)]
+                cols.append(column("k_bias", self.nkv, self.kd))
+                if not self.values_are_keys:
+                    cols.append(column("v_bias", self.nkv, self.vd))
             self.qkv_bias = torch.cat(cols).contiguous()
+        if self.has_output_bias:
             self.o_bias = params["o_bias"].to(torch.float32).contiguous()
         if self.output_gate:
             # a gate per element of the concatenated heads: its rows ride in the same product, laid out like the
@@ -210,6 +241,8 @@ class PagedAttention(Mixer):
             g = params["gate_proj"].to(dt)
             rows += [g, torch.zeros((-self.nq % 8, self.d), dtype=dt, device=g.device)]
         self.wqkv = torch.cat(rows, 0).contiguous()
+        if self.distance_table is not None:
+            self.distance_bias = DistanceBias.from_rows(params["distance_bias"], self._distance_rows)
         if self.has_head_sinks:
             self.head_sinks = params["sinks"].to(torch.float32).contiguous()
         if self.value_mix == "blend":
@@ -235,7 +268,7 @@ class PagedAttention(Mixer):
 
     @property
     def heads_size(self):
-        return None if self.has_bias else self.nq * self.vd
+        return None if self.has_output_bias else self.nq * self.vd
 
     def heads(self, x, out, column, batch, cache, scale=1.0):
         o = self._attend(x, batch, cache)
@@ -290,6 +323,8 @@ class PagedAttention(Mixer):
             extra["q_only"] = True
         if self.value_rotation is not None:
             extra["value_rotation"] = self.value_rotation
+        if self.values_are_keys:
+            extra["values_are_keys"] = True
         k.qk_prepare(qkv, q, batch, cache, num_heads=self.nq, rotation=self.position.rotation(),
                      qk_norm=self.qk_norm, temperature=self.temperature, **extra)
         o = torch.empty_like(q)
@@ -304,6 +339,8 @@ class PagedAttention(Mixer):
             more["head_gates"] = gates
         if self.score_softcap is not None:
             more["score_softcap"] = self.score_softcap
+        if self.distance_bias is not None:
+            more["distance_bias"] = self.distance_bias
         k.paged_attention(q, o, batch, cache, num_heads=self.nq, window=self.window,
                           softmax_scale=self.softmax_scale, cache_settled=True, sink_logit=self.sink_logit, **more)
         if self.output_gate:

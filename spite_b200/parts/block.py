@@ -5,6 +5,9 @@
 The residual stream h stays float32; the sums are done by the epilogues of the
 mixer's and the feed-forward's last products.
 
+`parallel_residual`: one norm, whose output both sublayers read, and both add to the stream (the feed-forward may be left out):
+    n = norm(h);  h += mixer(n) + feed_forward(n)
+
 `sandwich_residual`: a norm before and a norm behind every sublayer, and a factor on what joins the stream:
     h += mult * norm_c(mixer(norm_a(h)));  h += mult * norm_d(feed_forward(norm_b(h)))
 The sublayer's output goes to a float32 buffer of its own; one kernel norms it, adds it to the stream and, where
@@ -36,6 +39,20 @@ class PreNormResidual(Block):
         self.mixer.forward(x, h, batch, cache)
         if self.ffn is not None:
             self.ffn_norm.forward(h, x)
+            self.ffn.forward(x, h, batch)
+
+
+@register_block("parallel_residual")
+class ParallelResidual(Block):
+    graph_safe = True
+    places = {"norm": "norm", "mixer": "mixer", "ffn": "feed_forward"}
+    optional = ("ffn",)
+
+    def forward(self, h, batch, cache):
+        x = torch.empty(h.shape, dtype=self.ctx.dtype, device=h.device)
+        self.norm.forward(h, x)
+        self.mixer.forward(x, h, batch, cache)
+        if self.ffn is not None:
             self.ffn.forward(x, h, batch)
 
 

@@ -17,12 +17,18 @@ from .base import FeedForward, ParamSpec, register_feed_forward, side_stream
 
 @register_feed_forward("dense_swiglu")
 class DenseSwiGLU(FeedForward):
-    """h += down( silu(gate x) * (up x) )          (llama4.rs:257-271)"""
+    """h += down( silu(gate x) * (up x) )          (llama4.rs:257-271); `activation` "gelu_tanh": the gate passes gelu in its
+    tanh form instead of silu."""
     graph_safe = True
     kernel_libraries = ("gemm_simt",)
 
-    def __init__(self, ctx, hidden_size: int, intermediate_size: int):
+    ACTIVATIONS = ("silu", "gelu_tanh")
+
+    def __init__(self, ctx, hidden_size: int, intermediate_size: int, activation: str = "silu"):
         super().__init__(ctx)
+        if activation not in self.ACTIVATIONS:
+            raise ConfigError(f"unknown gate function {activation!r}; known: {', '.join(self.ACTIVATIONS)}")
+        self.activation = activation
         self.d, self.f = int(hidden_size), int(intermediate_size)
         self.w_gate_up = self.w_down = None
 
@@ -40,7 +46,7 @@ class DenseSwiGLU(FeedForward):
 
     def forward(self, x, h, batch):
         a = torch.empty((x.shape[0], self.f), dtype=x.dtype, device=x.device)
-        self.k.linear_swiglu(x, self.w_gate_up, a)
+        self.k.linear_swiglu(x, self.w_gate_up, a, activation=self.activation)
         self.k.linear(a, self.w_down, h, accumulate=True)
 
 
@@ -232,7 +238,7 @@ class MoESoftmaxTopK(FeedForward):
     The weight multiplies the float32 sums of the expert's last product as they are added to the residual
     stream, so no rounded intermediate carries it.
 
-    Variants, all parameters: `renormalize` False leaves the chosen shares as they are (w_e = s_e); `choice_bias` adds a
+    Variants, all parameters: `router_bias` adds a learned constant per expert to the logits; `renormalize` False leaves the chosen shares as they are (w_e = s_e); `choice_bias` adds a
     learned constant per expert (`choice_bias` [experts]) to the shares for the choice alone, the weights stay the
     shares; `identity_experts` n: the router has n outputs more than there are experts, and a token that draws one of
     those gets its own input back, times the weight (such an expert has no tensors)."""
@@ -241,7 +247,7 @@ class MoESoftmaxTopK(FeedForward):
     kernel_libraries = ("gemm_simt", "moe")
 
     def __init__(self, ctx, hidden_size: int, num_experts: int, top_k: int, expert_size: int, renormalize: bool = True,
-                 choice_bias: bool = False, identity_experts: int = 0):
+                 choice_bias: bool = False, identity_experts: int = 0, router_bias: bool = False):
         super().__init__(ctx)
         self.identity = int(identity_experts)
         if self.identity < 0 or num_experts < 0 or num_experts + self.identity < 1:
@@ -252,7 +258,8 @@ class MoESoftmaxTopK(FeedForward):
         if self.renormalize and (self.has_choice_bias or self.identity):
             raise ConfigError("a choice bias and identity experts go with weights that are not renormalised")
         self.d, self.E, self.top_k, self.f = int(hidden_size), int(num_experts), int(top_k), int(expert_size)
-        self.router = self.w_gate_up = self.w_down = self.choice_bias = None
+        self.has_router_bias = bool(router_bias)
+        self.router = self.w_gate_up = self.w_down = self.choice_bias = self.router_bias = None
         self.keep_router_logits = False      # `last_routing.logits` [tokens, experts] stays readable after a forward
 
     def param_specs(self):
@@ -261,11 +268,15 @@ class MoESoftmaxTopK(FeedForward):
                  "experts_up": ParamSpec((E, f, d)), "experts_down": ParamSpec((E, d, f))}
         if self.has_choice_bias:
             specs["choice_bias"] = ParamSpec((E + self.identity,))
+        if self.has_router_bias:
+            specs["router_bias"] = ParamSpec((E + self.identity,))
         return specs
 
     def bind(self, params):
         dt = self.ctx.dtype
         self.router = params["router"].to(torch.float32).contiguous()        # float32 sums of float32 weights
+        if self.has_router_bias:
+            self.router_bias = params["router_bias"].to(torch.float32).contiguous()
         if self.renormalize:
             self.choice_bias = None
         elif self.has_choice_bias:
@@ -286,11 +297,12 @@ class MoESoftmaxTopK(FeedForward):
     def forward(self, x, h, batch, accumulate=True):
         k = self.k
         M = x.shape[0]
+        more = {} if self.router_bias is None else dict(logit_bias=self.router_bias)
         if self.renormalize:
-            routing = k.moe_route(x, self.router, self.top_k, want_logits=self.keep_router_logits, scoring="softmax_renorm")
+            routing = k.moe_route(x, self.router, self.top_k, want_logits=self.keep_router_logits, scoring="softmax_renorm", **more)
         else:
             routing = k.moe_route(x, self.router, self.top_k, want_logits=self.keep_router_logits, scoring="softmax_biased",
-                                  choice_bias=self.choice_bias)
+                                  choice_bias=self.choice_bias, **more)
         self.last_routing = routing
         if self.identity:
             # the tokens that drew an identity expert get their input back, times the weight; without `accumulate` this

@@ -109,6 +109,24 @@ class RotaryYarn(PositionEncoding):
         return self._rotation
 
 
+def distance_rows(rows: int, far: int, length: int) -> list[int]:
+    """Which row of a table serves each distance 0 .. length - 1 (the T5 kind of buckets, one-sided): the first half of the
+    rows one distance each, the others ranges that grow geometrically up to the distance `far`, the last row everything
+    beyond.  With h = rows // 2: n < h: n; else min(rows - 1, h + floor(ln(n / h) / ln(far / h) (rows - h)))."""
+    half = rows // 2
+    if rows < 2 or far <= half:
+        raise ConfigError(f"a table of {rows} rows by distance needs two rows and a far distance ({far}) beyond half of them")
+    out = []
+    for n in range(length):
+        if n < half:
+            out.append(n)
+            continue
+        x = math.log(n / half) / math.log(far / half) * (rows - half)
+        # (a border that falls on a whole number belongs to the row above it, whichever way the logarithms were rounded)
+        out.append(min(rows - 1, half + math.floor(x + 1e-9)))
+    return out
+
+
 @register_position("rotary_halves")
 class RotaryHalves(PositionEncoding):
     """Rotation of the first `rotary_dim` elements of every head of q and k, element i paired with element

@@ -120,7 +120,10 @@ class TorchReferenceKernels(KernelSet):
                     out[t, a * vdim:(a + 1) * vdim] = (S.T @ q).to(out.dtype)
                 st.copy_(S.reshape(-1).to(st.dtype))
 
-    def fill_rows(self, out, vec, *, accumulate=False):
+    def fill_rows(self, out, vec, *, accumulate=False, other=None):
+        if other is not None:
+            out.copy_((out if accumulate else 0) + other)
+            accumulate = True
         if accumulate:
             out.add_(vec[None, :].to(out.dtype))
         else:
@@ -134,7 +137,7 @@ class TorchReferenceKernels(KernelSet):
             v = v * (1.0 / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps))
         v = v.reshape(M, heads * size)
         if gain is not None:
-            v = v * gain.to(self.acc)
+            v = v * (gain if gain.numel() == heads * size else gain.repeat(heads)).to(self.acc)
         if gates is not None:
             z = gates[:, gate_column:gate_column + heads * size].to(self.acc)
             v = v * (torch.sigmoid(z) * z if gate_activation == "silu" else torch.sigmoid(z))
@@ -242,6 +245,17 @@ class TorchReferenceKernels(KernelSet):
             return o, w[t, h * dim:(h + 1) * dim].to(self.acc)[:, None] * S + torch.outer(kt, vt)
         self._scan_segments(batch, state, state_offset, heads, dim, vdim, out, token)
 
+    def gated_linear_scan(self, q, k, v, a, w, out, batch, state, *, heads, dim, vdim, a2, a2_bias, tau, q_scale, state_offset=0):
+        z = a[0][:, a[1]:a[1] + a2.shape[0]].to(self.acc) @ a2.to(self.acc) + a2_bias.to(self.acc)
+        w.copy_((torch.sigmoid(z) ** (1.0 / tau)).to(w.dtype))
+
+        def token(h, t, S):
+            qt, kt = (x[0][t, x[1] + h * dim:x[1] + (h + 1) * dim].to(self.acc) for x in (q, k))
+            vt = v[0][t, v[1] + h * vdim:v[1] + (h + 1) * vdim].to(self.acc)
+            S = w[t, h * dim:(h + 1) * dim].to(self.acc)[:, None] * S + torch.outer(kt, vt)
+            return S.T @ qt * q_scale, S
+        self._scan_segments(batch, state, state_offset, heads, dim, vdim, out, token)
+
     # ---- recurrent mixers
     def mlstm_scan(self, proj, out, batch, state, *, heads, dim, vdim, gate_cap, q_scale, columns, i_bias, f_bias, chunked=None):
         qc, kc, vc, ic, fc = columns
@@ -314,12 +328,15 @@ class TorchReferenceKernels(KernelSet):
     def _silu(g):
         return g / (1.0 + torch.exp(-g))
 
-    def linear_swiglu(self, x, w_gate_up, out, *, row_scale=None):
+    def linear_swiglu(self, x, w_gate_up, out, *, row_scale=None, activation="silu"):
         F = w_gate_up.shape[0] // 2
         y = self._mm(x, w_gate_up)
         if row_scale is not None:
             y = y * row_scale.to(self.acc)[:, None]
-        out.copy_((self._silu(y[:, :F]) * y[:, F:]).to(out.dtype))
+        g = y[:, :F]
+        g = self._silu(g) if activation == "silu" else \
+            0.5 * g * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (g + 0.044715 * g ** 3)))
+        out.copy_((g * y[:, F:]).to(out.dtype))
 
     def grouped_linear_swiglu(self, x, w_gate_up, sorted_rows, offsets, row_scale, out):
         E, F2, _ = w_gate_up.shape
@@ -375,17 +392,18 @@ class TorchReferenceKernels(KernelSet):
 
     # ---- attention
     def qk_prepare(self, qkv, q_out, batch, cache, *, num_heads, rotation, qk_norm, temperature,
-                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None, value_rotation=None):
+                   value_mix=None, gates_out=None, bias=None, q_only=False, norm_dim=None, value_rotation=None,
+                   values_are_keys=False):
         kv = cache.kv
         nkv, P, hd = kv.shape[2], kv.shape[3], kv.shape[4]
         nq = num_heads
         M = qkv.shape[0]
-        cols = (nq + (0 if q_only else 2 * nkv)) * hd
+        cols = (nq + (0 if q_only else (1 if values_are_keys else 2) * nkv)) * hd
         x = qkv[:, :cols].to(self.acc)
         if bias is not None:
             x = x + bias.to(self.acc)[None, :]
         x = x.reshape(M, -1, hd)
-        q, k, v = x[:, :nq], x[:, nq:nq + nkv], x[:, nq + nkv:]
+        q, k, v = x[:, :nq], x[:, nq:nq + nkv], x[:, nq:] if values_are_keys else x[:, nq + nkv:]
         if q_only:
             assert not cache.write
             k = q[:, :0]
@@ -504,7 +522,7 @@ class TorchReferenceKernels(KernelSet):
 
     def paged_attention(self, q, out, batch, cache, *, num_heads, window, softmax_scale, cache_settled=False,
                         sink_logit=None, head_sinks=None, head_slopes=None, head_gates=None, out_by_head=False,
-                        score_softcap=None):
+                        score_softcap=None, distance_bias=None):
         kv = cache.kv
         nkv, P, hd = kv.shape[2], kv.shape[3], kv.shape[4]
         nq = num_heads
@@ -528,6 +546,8 @@ class TorchReferenceKernels(KernelSet):
                     s = score_softcap * torch.tanh(s / score_softcap)
                 if head_slopes is not None:
                     s = s - float(head_slopes[h]) * (p - js).to(self.acc)
+                if distance_bias is not None:
+                    s = s + distance_bias.padded[h, distance_bias.PAD + (p - js).clamp(max=distance_bias.length - 1)].to(self.acc)
                 sink = sink_logit if head_sinks is None else float(head_sinks[h])
                 if sink is None:
                     w = torch.softmax(s, dim=0)
@@ -550,8 +570,10 @@ class TorchReferenceKernels(KernelSet):
         else:
             out.copy_(y.to(out.dtype))
 
-    def moe_route(self, x, w_router, top_k, want_logits=False, scoring="sigmoid", choice_bias=None) -> Routing:
+    def moe_route(self, x, w_router, top_k, want_logits=False, scoring="sigmoid", choice_bias=None, logit_bias=None) -> Routing:
         logits = (x.to(torch.float32) @ w_router.to(torch.float32).T)
+        if logit_bias is not None:
+            logits = logits + logit_bias.to(torch.float32)
         order = torch.sort(logits, dim=-1, descending=True, stable=True)
         if scoring == "softmax_biased":
             share = torch.softmax(logits, -1)
