@@ -15,6 +15,7 @@ Two further workloads print a line of the same kind (they are extra modes; the d
     python bench.py --config mibezen     # the Mibezen design beside Llama 4 at equal layer sizes, measured the same way
     python bench.py --config paposun     # the Paposun design beside a dense Llama 4 at equal layer sizes, measured the same way
     python bench.py --config zuzadra     # the Zuzadra design beside Paposun at equal layer sizes, measured the same way
+    python bench.py --config fozutar     # the Fozutar design beside Gapevik at equal layer sizes, measured the same way
     python bench.py --config gapevik     # the Gapevik design beside Llama 4 at equal layer sizes, measured the same way
     python bench.py --config sezazen     # the Sezazen design beside Llama 4 at equal layer sizes (three sizes): prefill
                                          # of 2,048 tokens and decode at batch 1 and 8, each with its roofline fraction
@@ -418,6 +419,30 @@ def zuzadra_configs(size, runs=8):
     return zuz, pap
 
 
+def fozutar_configs(size, runs=8):
+    """A Fozutar model of eight layer runs (gated linear attention, then attention and gated linear attention three times on
+    one set of weights, then one more attention layer) and a Gapevik model of eight layers with a delta layer where Fozutar has
+    gated linear attention and attention where it has attention, on the same sets of weights (the loop's layers borrow), with
+    the same width, attention heads, chunk, cap, experts and vocabulary.  A gated linear attention has width / 128 heads of 64
+    key and 128 value elements with a decay of inner size 16, a delta layer width / 128 heads of 128 x 128 on half as many
+    q/k heads; the chunk is longer than the measured contexts, so every earlier key is read."""
+    name, d, nq, nkv, kd, vd, E, top, f, fs, fd, V = size
+    att = {"heads": nq, "kv_heads": nkv, "dim": kd, "vdim": kd, "scale": kd ** -0.5, "mask": {"size": 8192}, "softcap": 30.0}
+    gla = {"heads": d // 128, "dim": 64, "vdim": 128, "tau": 16.0, "rank": 16}
+    dlt = {"heads": d // 128, "kv_heads": d // 256, "dim": 128, "vdim": 128, "conv": 4}
+    moe = lambda **more: {"kind": "moe", "expert": {"ff": f}, "router": dict(more, experts=E, top=top)}
+    foz_att = dict(att, bias_max=4096, buckets=32)
+    gap_att = dict(att, conv=4, rot={"base": 500000.0, "dims": kd // 2})
+    L = lambda t, m, ff, **kw: dict({"type": t, "mixer": m, "mlp": ff}, **kw)
+    common = {"vocab": V, "width": d, "max_positions": 8192, "norm": {"eps": 1e-6}, "embedding": {"scale": d ** 0.5}}
+    foz = dict(common, architecture="Fozutar", loop={"start": 1, "stop": 3, "times": 3},
+               layers=[L("gla", gla, moe()), L("attention", foz_att, moe()), L("gla", gla, moe()), L("attention", foz_att, moe())])
+    A, D = (lambda **kw: L("attention", gap_att, moe(identity=0), **kw)), (lambda **kw: L("delta", dlt, moe(identity=0), **kw))
+    gap = dict(common, architecture="Gapevik", residual_mult=0.5,
+               layers=[D(), A(), D(), A(weights_of=1), D(weights_of=2), A(weights_of=1), D(weights_of=2), A()])
+    return foz, gap
+
+
 def design_work(model, T, contexts):
     """(flops of a prompt of T tokens, bytes a decode step over `contexts` must read), from the parts' own sizes
     as the design states them (no padding): every layer run reads its weights once; experts by the tokens' draw."""
@@ -426,11 +451,14 @@ def design_work(model, T, contexts):
     from spite_b200.parts.latent import LatentAttention
     from spite_b200.parts.mlstm import MatrixLstm
     from spite_b200.parts.delta import GatedDelta
+    from spite_b200.parts.gla import GatedLinearAttention
     from spite_b200.parts.parallel import ParallelMixers
     from spite_b200.parts.statespace import StateSpace
     es, p = 2, model.plan
     flops, nbytes = 2 * p.hidden_size * p.vocab_size, p.vocab_size * p.hidden_size * es
     for j in model.junctions:
+        if j.kind == "reinject_add":                 # two sums a row: no product, no weights to speak of
+            continue
         n = sum(1 for c in p.order if not isinstance(c, LayerCall))
         flops += n * 2 * T * 2 * j.d * j.d
         nbytes += n * 2 * j.d * j.d * es
@@ -456,6 +484,12 @@ def design_work(model, T, contexts):
             w = d * (2 * m.G * m.kd + 2 * m.H * m.vd + 2 * m.H) + m.H * m.vd * d
             flops += 2 * T * w + 4 * T * m.H * m.kd * m.vd
             nbytes += w * es + len(contexts) * 2 * m.H * m.kd * m.vd * 4
+        elif isinstance(m, GatedLinearAttention):
+            # projections (q, k, v, the gate, the decay's two) and the output; per token and head the matrix's update and its
+            # read-out, two multiply-adds an element; a decode step reads and writes the matrices
+            w = d * (2 * m.nk + 2 * m.nv + m.rank) + m.rank * m.nk + m.nv * d
+            flops += 2 * T * w + 4 * T * m.H * m.kd * m.vd
+            nbytes += w * es + len(contexts) * 2 * m.H * m.kd * m.vd * 4
         elif isinstance(m, StateSpace):
             # both projections; per token and head the matrix's update and its read-out, two multiply-adds an element
             w = d * (2 * m.inner + 2 * m.G * m.N + m.H) + m.inner * d
@@ -468,10 +502,11 @@ def design_work(model, T, contexts):
             nbytes += w * es + sum(c * a.nkv * (a.kd + a.vd) * es for c in contexts) + len(contexts) * 2 * b.n * b.dim * 4
         else:
             shared = getattr(m, "kv_shared", False)
-            w = d * (m.nq * m.kd + (0 if shared else m.nkv * (m.kd + m.vd))) + m.nq * m.vd * d + \
+            keys_alone = getattr(m, "values_are_keys", False)         # one row a position serves as key and value
+            w = d * (m.nq * m.kd + (0 if shared else m.nkv * (m.kd + (0 if keys_alone else m.vd)))) + m.nq * m.vd * d + \
                 (m.nq * d if getattr(m, "head_gate", False) else 0) + (m.nq * m.vd * d if getattr(m, "output_gate", False) else 0)
             flops += 2 * T * w + 2 * m.nq * (m.kd + m.vd) * T * (T + 1) // 2
-            nbytes += w * es + sum(c * m.nkv * (m.kd + m.vd) * es for c in contexts)
+            nbytes += w * es + sum(c * m.nkv * (m.kd + (0 if keys_alone else m.vd)) * es for c in contexts)
         f = blk.ffn
         if f is None:
             continue
@@ -509,8 +544,8 @@ def run_sezazen(args):
     the first size."""
     design = args.config
     configs_of = {"sezazen": design_configs, "mibezen": mibezen_configs, "paposun": paposun_configs,
-                  "gapevik": gapevik_configs, "zuzadra": zuzadra_configs}[design]
-    other = "paposun" if design == "zuzadra" else "llama4"
+                  "gapevik": gapevik_configs, "zuzadra": zuzadra_configs, "fozutar": fozutar_configs}[design]
+    other = {"zuzadra": "paposun", "fozutar": "gapevik"}.get(design, "llama4")
     import torch
     from spite_b200.config import config_from_dict
     from spite_b200.engine import Engine, Model, StepEntry
@@ -791,8 +826,8 @@ def main(argv=None):
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", choices=["ours", "reference"], default="ours")
-    ap.add_argument("--config", choices=["scout", "maverick", "long", "sezazen", "mibezen", "paposun", "gapevik", "zuzadra"], default="scout",
-                    help="scout: the benchmark line; maverick, long, sezazen, mibezen, paposun, gapevik, zuzadra: further workloads, one line each")
+    ap.add_argument("--config", choices=["scout", "maverick", "long", "sezazen", "mibezen", "paposun", "gapevik", "zuzadra", "fozutar"], default="scout",
+                    help="scout: the benchmark line; maverick, long, sezazen, mibezen, paposun, gapevik, zuzadra, fozutar: further workloads, one line each")
     ap.add_argument("--layers", type=int, default=FULL_LAYERS)
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=8192)
@@ -802,8 +837,8 @@ def main(argv=None):
     ap.add_argument("--only-prefill", action="store_true", help="measure the prefill step only (for profiling)")
     ap.add_argument("--verbose", action="store_true", help="print the single prefill timings to standard error")
     ap.add_argument("--size", default=None, help="--config sezazen: only this set of layer sizes (small, medium, ...)")
-    ap.add_argument("--design", choices=["both", "sezazen", "mibezen", "paposun", "gapevik", "zuzadra", "llama4"], default="both",
-                    help="--config sezazen / mibezen / paposun / gapevik / zuzadra: only this design")
+    ap.add_argument("--design", choices=["both", "sezazen", "mibezen", "paposun", "gapevik", "zuzadra", "fozutar", "llama4"], default="both",
+                    help="--config sezazen / mibezen / paposun / gapevik / zuzadra / fozutar: only this design")
     args = ap.parse_args(argv)
     if args.impl == "reference":
         return run_reference(args)
@@ -816,7 +851,7 @@ def main(argv=None):
     if args.config == "long":
         run_long(args)
         return 0
-    if args.config in ("sezazen", "mibezen", "paposun", "gapevik", "zuzadra"):
+    if args.config in ("sezazen", "mibezen", "paposun", "gapevik", "zuzadra", "fozutar"):
         run_sezazen(args)
         return 0
     if args.warmup < 3:

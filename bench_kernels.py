@@ -10,10 +10,15 @@ peak.  Also the small driver that `ncu` captures for the summaries under `profil
     python bench_kernels.py --only attention_decode,attention_prefill --sink 0   # attention with a sink in the softmax
     python bench_kernels.py --only attention_decode,attention_prefill --bias     # ... with a distance bias, learned sinks and gates per head
     python bench_kernels.py --only attention_decode,attention_prefill --latent   # ... over latent rows (one plane, 16 heads on one kv head)
+    python bench_kernels.py --only attention_decode,attention_prefill --cap 30             # ... with capped scores
+    python bench_kernels.py --only attention_decode,attention_prefill --cap 30 --distance  # ... with a number per head and distance, keys
+                                                 # that are the values (one plane) and a factor per key
     python bench_kernels.py --only gated_less    # experts without a gate (squared ReLU), the junction of a loop,
                                                  # the embedding with learned positions
     python bench_kernels.py --only recurrent     # the matrix memory's scan in prompts and decode steps, the heads' norm
-    python bench_kernels.py --only scan          # the scans of the state space and the decaying memory, streams, token shift, gated norm
+    python bench_kernels.py --only scan          # the scans of the state space, the decaying memory and gated linear attention,
+                                                 # streams, token shift, gated norm, heads' norm with a silu gate, what is added
+                                                 # between two passes, products with silu and gelu gates
     python bench_kernels.py --only delta         # the gated delta rule's scan in prompts and decode steps, the short convolution
                                                  # and gate, the norm behind a sublayer
 
@@ -50,6 +55,9 @@ def main(argv=None):
     ap.add_argument("--rows", default="1,8,64", help="token counts of the decode families")
     ap.add_argument("--sink", type=float, default=None, help="attention cases run with a sink of this score in the softmax")
     ap.add_argument("--bias", action="store_true", help="attention cases run with a distance bias, a learned sink and a gate per head")
+    ap.add_argument("--cap", type=float, default=None, help="attention cases run with scores capped at this")
+    ap.add_argument("--distance", action="store_true", help="attention cases run with a number per head and distance (32 buckets up to "
+                                                          "the context) over keys that are the values, with a factor per key")
     ap.add_argument("--latent", action="store_true", help="attention cases run on a cache of one plane: 16 query heads on one kv head "
                                                         "whose key rows (128 elements) are also the values, the result head by head")
     args = ap.parse_args(argv)
@@ -219,6 +227,8 @@ def main(argv=None):
     # ---- attention over the paged cache
     P = 64
     sink = "" if args.sink is None else f" sink={args.sink}"
+    sink += ("" if args.cap is None else f" cap={args.cap}") + (" distance, keys as values" if args.distance else "")
+    one_plane = args.latent or args.distance
     sink += (" bias+sinks+gates" if args.bias else "") + (" one plane, 16 heads on 1" if args.latent else "")
     if args.latent:
         nq, nkv, hd = 16, 1, 128
@@ -232,10 +242,15 @@ def main(argv=None):
             off += n_new
         batch = build_step_batch(segs, [[0] * n_new] * n_req, [[]] * n_req, [tables], dev)
         def make():
-            kv = (torch.randn((1 if args.latent else 2, n_req * pages_per, nkv, P, hd), device=dev) * 0.5).to(bf)
+            kv = (torch.randn((1 if one_plane else 2, n_req * pages_per, nkv, P, hd), device=dev) * 0.5).to(bf)
             q, out = rnd(off, nq * hd), torch.empty((off, nq * hd), dtype=bf, device=dev)
-            cache = LayerCache(0, kv, None, P, False)
-            more = {}
+            factors = torch.rand((n_req * pages_per, nkv, P), device=dev) + 0.5 if args.distance else None
+            cache = LayerCache(0, kv, None, P, False, factors)
+            more = {} if args.cap is None else {"score_softcap": args.cap}
+            if args.distance:
+                from spite_b200.kernels.api import DistanceBias
+                from spite_b200.parts.position import distance_rows
+                more["distance_bias"] = DistanceBias.from_rows(torch.randn((32, nq), device=dev), distance_rows(32, ctx, ctx))
             if args.bias:
                 more = {"head_sinks": torch.randn(nq, device=dev), "head_gates": torch.rand((off, nq), device=dev),
                         "head_slopes": torch.tensor([2.0 ** (-8.0 * (h + 1) / nq) for h in range(nq)], device=dev)}
@@ -246,7 +261,7 @@ def main(argv=None):
         seen = sum(min(p + 1, ctx) - win.lowest_visible(p) for p in range(ctx - n_new, ctx)) / n_new
         if n_new == 1:
             # short launches: back to back over rotating copies of the cache, so no launch gap is counted
-            nbytes = int(n_req * seen * (1 if args.latent else 2) * nkv * hd * 2)
+            nbytes = int(n_req * seen * nkv * (hd * 2 * (1 if one_plane else 2) + (4 if args.distance else 0)))
             report(fam, f"requests={n_req} context={ctx} window={window[0]}{sink}", timed_rotating(make, nbytes), nbytes=nbytes)
             return
         report(fam, f"tokens={n_new} context={ctx} window={window[0]}{sink}", timed(make()),
@@ -407,7 +422,8 @@ def main(argv=None):
             M = n_seg * n_tok
             segs = [Segment(i, i, 0, n_tok, i * n_tok, True) for i in range(n_seg)]
             batch = build_step_batch(segs, [[0] * n_tok] * n_seg, [[]] * n_seg, [[[0]] * n_seg], dev)
-            for kind, H, kd, vd in (("state_space", dm // 32, 128, 64), ("decay", dm // 64, 64, 64)):
+            for kind, H, kd, vd in (("state_space", dm // 32, 128, 64), ("decay", dm // 64, 64, 64), ("gated_linear", dm // 64, 64, 64),
+                                    ("gated_linear", dm // 128, 64, 128)):
                 G = 1 if kind == "state_space" else H
                 size = H * ks.scan_state_size(kd, vd)
                 def make_scan(M=M, batch=batch, n_seg=n_seg, kind=kind, H=H, kd=kd, vd=vd, G=G, size=size):
@@ -417,6 +433,11 @@ def main(argv=None):
                         x, step = torch.randn((M, 2 * kd + H * vd), device=dev), torch.randn((M, H), device=dev)
                         return lambda: ks.state_space_scan((x, kd), (x, 0), (x, 2 * kd), (step, 0), out, batch, state, heads=H, kv_heads=1,
                                                            dim=kd, vdim=vd, a_log=hv, dt_bias=hv, skip=hv)
+                    if kind == "gated_linear":
+                        x, w = torch.randn((M, H * (2 * kd + vd) + 16), device=dev), torch.empty((M, H * kd), device=dev)
+                        a2, b = torch.randn((16, H * kd), device=dev), torch.zeros(H * kd, device=dev)
+                        return lambda: ks.gated_linear_scan((x, 0), (x, H * kd), (x, 2 * H * kd), (x, H * (2 * kd + vd)), w, out, batch, state,
+                                                            heads=H, dim=kd, vdim=vd, a2=a2, a2_bias=b, tau=16.0, q_scale=0.125)
                     r, k, v, w = (torch.randn((M, H * kd), device=dev) for _ in range(4))
                     u = torch.zeros(H * kd, device=dev)
                     return lambda: ks.decay_scan((r, 0), (k, 0), (v, 0), w, out, batch, state, heads=H, dim=kd,
@@ -448,6 +469,26 @@ def main(argv=None):
             nbytes = M * dm * 12 + n_seg * dm * 8
             report("scan", f"token_shift {n_seg} x {n_tok} tokens, 5 mixes of {dm}", timed_rotating(make_shift, max(nbytes, 64 << 20) if n_tok == 1 else nbytes), nbytes=nbytes)
         for M in (8, 2048):
+            def make_heads(M=M):
+                o, z, g = torch.randn((M, dm), device=dev), torch.randn((M, 2 * dm), device=dev), torch.ones(128, device=dev)
+                a = torch.empty((M, dm), dtype=bf, device=dev)
+                return lambda: ks.head_norm_gate(o, a, heads=dm // 128, size=128, gates=z, gate_column=dm, gain=g, eps=1e-6, gate_activation="silu")
+            nbytes = M * dm * 10
+            report("scan", f"head_norm_gate M={M}, {dm // 128} heads of 128, silu gate", timed_rotating(make_heads, max(nbytes, 64 << 20) if M == 8 else nbytes), nbytes=nbytes)
+            def make_add(M=M):
+                h, h0, step = torch.randn((M, dm), device=dev), torch.randn((M, dm), device=dev), torch.randn(dm, device=dev)
+                return lambda: ks.fill_rows(h, step, accumulate=True, other=h0)
+            nbytes = M * dm * 12
+            report("scan", f"fill_rows M={M} d={dm}, two rows and a vector", timed_rotating(make_add, max(nbytes, 64 << 20) if M == 8 else nbytes), nbytes=nbytes)
+            for act in ("silu", "gelu_tanh"):
+                def make_gated(M=M, act=act):
+                    x, w, a = rnd(M, dm), rnd(2 * 14336, dm), torch.empty((M, 14336), dtype=bf, device=dev)
+                    return lambda: ks.linear_swiglu(x, w, a, activation=act)
+                name, flops, nbytes = f"gate and up, {act}, M={M}, 2 x 14336 x {dm}", 4 * M * 14336 * dm, 4 * 14336 * dm
+                if M == 8:
+                    report("scan", name, timed_rotating(make_gated, nbytes), nbytes=nbytes)
+                elif not args.case or args.case in name:
+                    report("scan", name, timed(make_gated()), flops=flops)
             inner = 2 * dm
             def make_norm(M=M):
                 y, z, g = torch.randn((M, inner), device=dev), torch.randn((M, inner), device=dev), torch.ones(inner, device=dev)

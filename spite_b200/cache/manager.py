@@ -83,6 +83,7 @@ class GroupKey:
     num_kv_heads: int
     head_dim: int
     planes: int = 2
+    key_scales: bool = False
 
 
 class PagePool:

@@ -3,7 +3,7 @@
 One tensor per group, `[caches of the group, planes (keys, values; or keys alone), pages, kv heads,
 page_size, head_dim]`: for one kv head the `page_size` keys of a page are
 contiguous rows of `head_dim` elements, which is the tile an attention kernel
-loads.  Per-request state of fixed size lives in one tensor per cache that asks
+loads.  A group may keep a float32 factor beside every key, `[caches, pages, kv heads, page_size]`.  Per-request state of fixed size lives in one tensor per cache that asks
 for it, `[slots, *shape]`.
 """
 from __future__ import annotations
@@ -18,11 +18,12 @@ from .manager import CacheManager, GroupKey, Window
 @dataclass(frozen=True)
 class PagedKV:
     """A mixer's request for paged keys and values.  `planes` 2: keys and values; 1: keys only (the value of a
-    position is its key row, or a leading part of it)."""
+    position is its key row, or a leading part of it).  `key_scales`: a float32 factor beside every cached key."""
     window: Window
     num_kv_heads: int
     head_dim: int
     planes: int = 2
+    key_scales: bool = False
 
 
 @dataclass(frozen=True)
@@ -36,12 +37,13 @@ class LayerCache:
     """What one run of a layer sees of the cache."""
 
     def __init__(self, group: int | None, kv: torch.Tensor | None, state: torch.Tensor | None,
-                 page_size: int, write: bool):
+                 page_size: int, write: bool, key_scale: torch.Tensor | None = None):
         self.group = group          # index of the block table to use
         self.kv = kv                # [planes, pages, kv heads, page_size, head_dim] or None
         self.state = state          # [slots, *shape] or None
         self.page_size = page_size
         self.write = write          # this run appends its keys and values
+        self.key_scale = key_scale  # float32 [pages, kv heads, page_size] or None
 
 
 class CacheStorage:
@@ -59,7 +61,7 @@ class CacheStorage:
             kv, _ = cache_specs[cid]
             if kv is None:
                 continue
-            key = GroupKey(kv.window, kv.num_kv_heads, kv.head_dim, kv.planes)
+            key = GroupKey(kv.window, kv.num_kv_heads, kv.head_dim, kv.planes, kv.key_scales)
             if key not in keys:
                 keys.append(key)
                 counts.append(0)
@@ -72,6 +74,9 @@ class CacheStorage:
             CacheManager([], page_size, [], n_slots)
         self.kv = [torch.zeros((counts[g], k.planes, pages, k.num_kv_heads, page_size, k.head_dim),
                                dtype=dtype, device=self.device) for g, k in enumerate(keys)]
+        # (a factor is only read where its key is visible: a page that is handed out again needs no clearing here)
+        self.key_scales = [torch.zeros((counts[g], pages, k.num_kv_heads, page_size), dtype=torch.float32, device=self.device)
+                           if k.key_scales else None for g, k in enumerate(keys)]
         self.state = {}
         for cid, (_, st) in cache_specs.items():
             if st is not None:
@@ -82,13 +87,14 @@ class CacheStorage:
         return len(self.group_keys)
 
     def bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in self.kv) + \
+        return sum(t.numel() * t.element_size() for t in self.kv + [t for t in self.key_scales if t is not None]) + \
             sum(t.numel() * t.element_size() for t in self.state.values())
 
     def layer_cache(self, cache_id: int, write: bool) -> LayerCache:
         g = self._group_of.get(cache_id)
         kv = self.kv[g][self._index_in_group[cache_id]] if g is not None else None
-        return LayerCache(g, kv, self.state.get(cache_id), self.page_size, write)
+        scales = self.key_scales[g][self._index_in_group[cache_id]] if g is not None and self.key_scales[g] is not None else None
+        return LayerCache(g, kv, self.state.get(cache_id), self.page_size, write, scales)
 
     def clear_pages(self, kernels, pages_per_group):
         """Pages that have just been handed out start at zero in every cache of their group: whatever the

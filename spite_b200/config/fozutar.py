@@ -197,8 +197,8 @@ class FozutarConfig:
                     raise ConfigError(f"{at}: heads, kv_heads, dim and mask.size must be positive, heads a multiple of kv_heads")
                 if not m.scale > 0 or not m.softcap > 0:
                     raise ConfigError(f"{at}: scale and softcap must be positive")
-                if m.table_rows < 2 or m.bias_max <= m.table_rows // 2:
-                    raise ConfigError(f"{at}: bias_max {m.bias_max} must lie beyond half of the table's {m.table_rows} rows")
+                if m.bias_max < 1 or m.table_rows < 1:
+                    raise ConfigError(f"{at}: bias_max and the rows of the table must be positive")
             else:
                 if min(m.heads, m.dim, m.vdim, m.decay_rank) < 1:
                     raise ConfigError(f"{at}: heads, dim, vdim and rank must be positive")

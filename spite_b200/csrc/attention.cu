@@ -144,13 +144,18 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkPrepareParams p
                 if (bias) { x0[r] += bias[e0[r]]; x1[r] += bias[e1[r]]; }
             }
         }
-        if (p.values_are_keys && !is_q) {                        // the key as projected is the value
+        if (p.values_are_keys && !is_q) {                        // (no rotation, no gains: checked by the host)
+            float ss = 0.f;
 #pragma unroll
             for (int r = 0; r < MAXP; ++r) {
-                if (2 * (lane + 32 * r) >= hd) continue;
-                if (halves) { dst[c.v_offset + e0[r]] = from_f32<T>(x0[r]); dst[c.v_offset + e1[r]] = from_f32<T>(x1[r]); }
-                else store_pair(dst + c.v_offset + e0[r], x0[r], x1[r]);
+                ss += x0[r] * x0[r] + x1[r] * x1[r];
+                if (2 * (lane + 32 * r) < hd) store_pair(dst + e0[r], x0[r], x1[r]);
             }
+            ss = warp_sum(ss);
+            if (lane == 0)
+                c.key_scale[((size_t)page * nkv + head - nq) * c.page_size + pos % c.page_size] =
+                    norm ? 1.0f / sqrtf(ss / norm_n + p.qk_norm_eps) : 1.0f;
+            continue;
         }
         if (norm_first) {
             float ss = 0.f;
@@ -267,7 +272,9 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const AttentionPar
             const T* k = kbase + row;
             float dot = 0.f;
             for (int d = 0; d < hd; ++d) dot = fmaf(q_s[warp][d], to_f32(k[d]), dot);
-            s = capped(p, dot * p.softmax_scale) - slope * (float)(pos - j);
+            s = dot * p.softmax_scale;
+            if (c.key_scale) s *= c.key_scale[row / hd];
+            s = capped(p, s) - slope * (float)(pos - j);
             if (dist) s += dist[min(pos - j, p.distance_len - 1)];
         }
         const float m_new = fmaxf(m, warp_max(s));
@@ -333,7 +340,8 @@ SPITE_API int spite_qk_prepare(int dtype, const QkPrepareParams* given, const St
     if (p->inv_freq && (p->rotary_dim < 2 || p->rotary_dim % 2 || p->rotary_dim > c->head_dim)) return SPITE_BAD_ARG;
     const int heads = p->num_heads + (p->q_only ? 0 : (p->values_are_keys ? 1 : 2) * c->num_kv_heads);
     if (p->q_only && (p->v_other || p->gates_out || p->values_are_keys)) return SPITE_BAD_ARG;
-    if (p->values_are_keys && (p->v_other || p->v_inv_freq || c->v_offset == 0)) return SPITE_BAD_ARG;
+    if (p->values_are_keys && (p->v_other || p->v_inv_freq || p->inv_freq || p->k_gain || c->v_offset != 0 || !c->key_scale))
+        return SPITE_BAD_ARG;
     if (p->qkv_stride < (long long)heads * c->head_dim || (p->qkv_stride & 1)) return SPITE_BAD_ARG;
     if (p->gates_out && p->qkv_stride < (long long)heads * c->head_dim + p->num_heads) return SPITE_BAD_ARG;
     if (p->v_inv_freq && (p->v_other || p->q_only || p->v_rotary_dim < 2 || p->v_rotary_dim % 2 || p->v_rotary_dim > c->head_dim ||

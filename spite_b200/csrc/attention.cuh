@@ -20,6 +20,8 @@ struct StepTokens {
 // One cache: keys at kv, values at kv + v_offset (elements); a page holds, for every
 // kv head, page_size rows of head_dim elements: [pages][kv heads][page_size][head_dim].
 // v_offset 0: the cache has keys only and a position's value is its key row.
+// key_scale, if given, holds a factor per cached key, [pages][kv heads][page_size]: the score of a key is the product with its row
+// times its factor (a norm of the keys whose rows are kept as projected, because they are the values too).
 struct PagedCache {
     void* kv;
     long long v_offset;
@@ -27,6 +29,7 @@ struct PagedCache {
     int page_size;
     int num_kv_heads;
     int head_dim;
+    float* key_scale;
 };
 
 #define SPITE_PAIR_NEIGHBOURS 0   // pair i of a head is elements (2i, 2i+1)
@@ -71,8 +74,8 @@ struct QkPrepareParams {
     // what inv_freq and v_inv_freq lost when they were rounded to float32 (null: the angle is the rounded product)
     const float* inv_freq_low;
     const float* v_inv_freq_low;
-    // the values are the projected keys (bias included), as they are before norm and rotation: a row of qkv holds q heads
-    // and k heads alone
+    // the values are the projected keys (bias included): a row of qkv holds q heads and k heads alone, a cache of one plane
+    // takes the keys as projected, and what the norm would multiply a key by goes to the cache's key_scale
     int values_are_keys;
 };
 
@@ -136,20 +139,27 @@ __device__ __forceinline__ float slope_of(const AttentionParams& p, int head) {
 __device__ __forceinline__ float capped(const AttentionParams& p, float s) {
     return p.score_softcap > 0.f ? p.score_softcap * tanhf(s / p.score_softcap) : s;
 }
-// The tensor-core kernels are compiled in three forms: scores as they are, capped, and with a number per distance (capped
-// if there is a cap).  With the choice made per score at run time, the decode kernel took a tenth longer without any cap.
-enum ScoreForm { FORM_PLAIN = 0, FORM_CAP = 1, FORM_DISTANCE = 2 };
-static inline int score_form_of(const AttentionParams& p) {
-    return p.distance_bias ? FORM_DISTANCE : p.score_softcap > 0.f ? FORM_CAP : FORM_PLAIN;
+// The tensor-core kernels are compiled in three forms: scores as they are, capped, and with everything else (a factor per key,
+// a number per distance, a cap or none) chosen at run time.  With the choice of the cap made per score at run time, the decode
+// kernel took a tenth longer without any cap.
+enum ScoreForm { FORM_PLAIN = 0, FORM_CAP = 1, FORM_ANY = 2 };
+static inline int score_form_of(const AttentionParams& p, const PagedCache& c) {
+    return p.distance_bias || c.key_scale ? FORM_ANY : p.score_softcap > 0.f ? FORM_CAP : FORM_PLAIN;
 }
 static inline bool distance_bias_ok(const AttentionParams* p) {
     return !p->distance_bias || (p->distance_runs && p->distance_len >= 1 && p->distance_len <= (1 << 24));
 }
-// The score of a visible key n positions before the query, from the scaled product `s`.
-template <int FORM> __device__ __forceinline__ float score_of(const AttentionParams& p, float s, float slope, const float* row, int n) {
+// The score of a visible key n positions before the query, from the product `s` scaled by the softmax's scale; `key` is the
+// key's own factor (1 without one).
+template <int FORM>
+__device__ __forceinline__ float score_of(const AttentionParams& p, float s, float key, float slope, const float* row, int n) {
     if constexpr (FORM == FORM_CAP) return p.score_softcap * tanhf(s / p.score_softcap) - slope * (float)n;
-    else if constexpr (FORM == FORM_DISTANCE) return capped(p, s) - slope * (float)n + row[min(n, p.distance_len - 1)];
+    else if constexpr (FORM == FORM_ANY) return capped(p, s * key) - slope * (float)n + (row ? row[min(n, p.distance_len - 1)] : 0.f);
     else return s - slope * (float)n;
+}
+// The factor of the first key of a tile that lies in one page (null without factors).
+__device__ __forceinline__ const float* key_scale_of(const PagedCache& c, int page, int kvh, int position) {
+    return c.key_scale ? c.key_scale + ((size_t)page * c.num_kv_heads + kvh) * c.page_size + position % c.page_size : nullptr;
 }
 // The factor on a finished output row.
 __device__ __forceinline__ float gate_of(const AttentionParams& p, int token, int head) {

@@ -84,6 +84,8 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
     extern __shared__ unsigned char smem_raw[];
     unsigned char* smem = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     Tail* tail = (Tail*)(smem + ring_bytes);               // the ring of stages, later the merge buffers, lie before it
+    __shared__ __align__(16) float key_scales[FORM == FORM_ANY ? MAX_STAGES * BN : 4];    // a stage's keys' factors
+    const bool scaled = FORM == FORM_ANY && c.key_scale != nullptr;
     volatile int* abort_flag = &tail->abort_flag;
     int* const err_word = waits.error_word ? waits.error_word : &g_attn_decode_error;
     const long long wait_limit = waits.limit_cycles;
@@ -134,7 +136,8 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
         const int page = max(table[j0 / c.page_size], 0);     // a tile with a visible key lies in a held page
         const int row = (page * nkv + kvh) * c.page_size + j0 % c.page_size;
         const unsigned bar = smem_u32(&tail->full[s]), dst = smem_u32(smem + (size_t)s * STAGE);
-        mbar_expect_tx(bar, STAGE);
+        mbar_expect_tx(bar, STAGE + (scaled ? BN * 4 : 0));
+        if (scaled) bulk_load(smem_u32(key_scales + s * BN), key_scale_of(c, page, kvh, j0), BN * 4, bar);
 #pragma unroll
         for (int kb = 0; kb < NKB; ++kb) {
             tma_load_2d_hint(dst + kb * BOX_BYTES, &map_k, kb * 64, row, bar, policy);
@@ -226,6 +229,14 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
                         mma16816(sc[n], qa[kk + 1][0], qa[kk + 1][1], qa[kk + 1][2], qa[kk + 1][3], kb[2], kb[3]);
                     }
                 }
+                float key[2][2] = {{1.f, 1.f}, {1.f, 1.f}};      // the keys' factors
+                if (scaled) {
+#pragma unroll
+                    for (int n = 0; n < 2; ++n) {
+                        const float2 f = *(const float2*)(key_scales + s * BN + 16 * warp + 8 * n + 2 * cc);
+                        key[n][0] = f.x; key[n][1] = f.y;
+                    }
+                }
                 // mask, running maximum and sum (float32)
                 float corr[2];
 #pragma unroll
@@ -237,7 +248,7 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
                         for (int e = 0; e < 2; ++e) {
                             const int j = j0 + 8 * n + 2 * cc + e;
                             const bool vis = row_ok[h] && j >= row_lo[h] && j <= row_pos[h];
-                            const float v = vis ? score_of<FORM>(p, sc[n][2 * h + e] * p.softmax_scale, row_slope[h], row_dist[h], row_pos[h] - j) : -INFINITY;
+                            const float v = vis ? score_of<FORM>(p, sc[n][2 * h + e] * p.softmax_scale, key[n][e], row_slope[h], row_dist[h], row_pos[h] - j) : -INFINITY;
                             sc[n][2 * h + e] = v;
                             mx = fmaxf(mx, v);
                         }
@@ -433,8 +444,8 @@ int launch(const AttentionParams& p, const StepTokens& b, const PagedCache& c, c
     ring = (ring + 15) & ~(size_t)15;
     const size_t smem = ring + sizeof(Tail) + 1024;
     if (smem > 227 * 1024) return SPITE_UNSUPPORTED;
-    const int form = score_form_of(p);
-    auto k = form == FORM_DISTANCE ? attn_decode_kernel<NKB, FORM_DISTANCE> : form == FORM_CAP ? attn_decode_kernel<NKB, FORM_CAP> : attn_decode_kernel<NKB, FORM_PLAIN>;
+    const int form = score_form_of(p, c);
+    auto k = form == FORM_ANY ? attn_decode_kernel<NKB, FORM_ANY> : form == FORM_CAP ? attn_decode_kernel<NKB, FORM_CAP> : attn_decode_kernel<NKB, FORM_PLAIN>;
     if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
         cudaFuncSetAttribute(k, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared) != cudaSuccess)
         return SPITE_LAUNCH_FAILED;
@@ -465,7 +476,7 @@ SPITE_API int spite_paged_attention_decode(const AttentionParams* p, const StepT
     if (x->tokens_per_block * G > 16) return SPITE_BAD_ARG;
     if (x->n_splits > 1 && (!x->partial || !x->tickets)) return SPITE_BAD_ARG;
     if (x->n_splits > 1024 || c->num_kv_heads > 65535 || x->n_splits > 65535) return SPITE_UNSUPPORTED;
-    if ((((uintptr_t)p->q | (uintptr_t)p->out | (uintptr_t)c->kv | (uintptr_t)x->partial) & 15) || (c->v_offset & 7))
+    if ((((uintptr_t)p->q | (uintptr_t)p->out | (uintptr_t)c->kv | (uintptr_t)x->partial | (uintptr_t)c->key_scale) & 15) || (c->v_offset & 7))
         return SPITE_UNSUPPORTED;                              // TMA, 16-byte loads of partial results, 8-byte stores
     if (b->n_tokens == 0 || n_blocks == 0) return SPITE_OK;
     cudaStream_t st = (cudaStream_t)stream;

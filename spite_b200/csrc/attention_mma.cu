@@ -125,9 +125,16 @@ __global__ void __launch_bounds__(WARPS * 32) attn_mma_kernel(const AttentionPar
     const __nv_bfloat16* vbase = kbase + c.v_offset;
 
     const unsigned long long kv_policy = l2_evict_first();
+    const bool scaled = FORM == FORM_ANY && c.key_scale != nullptr;
+    float2 next_scale[2] = {make_float2(1.f, 1.f), make_float2(1.f, 1.f)};     // the factors of this lane's keys of the tile asked for last
     auto issue = [&](int stage, int ti) {
         const int j0 = ti * TILE;
         const int page = table[j0 / c.page_size];
+        if (scaled) {
+            const float* f = key_scale_of(c, max(page, 0), kvh, j0) + 2 * cc;
+            next_scale[0] = make_float2(f[0], f[1]);
+            next_scale[1] = make_float2(f[8], f[9]);
+        }
         const size_t off = (((size_t)max(page, 0) * nkv + kvh) * c.page_size + j0 % c.page_size) * HD;
         const unsigned kdst = my_addr + stage * 2 * TILE_BYTES, vdst = kdst + TILE_BYTES;
 #pragma unroll
@@ -152,6 +159,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_mma_kernel(const AttentionPar
     cp_async_commit();
     int stage = 0;
     for (; ti < se; ti += WARPS, stage ^= 1) {
+        const float key[2][2] = {{next_scale[0].x, next_scale[0].y}, {next_scale[1].x, next_scale[1].y}};
         if (ti + WARPS < se) issue(stage ^ 1, ti + WARPS);
         cp_async_commit();
         cp_async_wait<1>();
@@ -192,7 +200,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_mma_kernel(const AttentionPar
                 for (int e = 0; e < 2; ++e) {
                     const int j = j0 + 8 * n + 2 * cc + e;
                     const bool ok = row_ok[h] && j >= row_lo[h] && j <= row_pos[h];
-                    const float v = ok ? score_of<FORM>(p, s[n][2 * h + e] * p.softmax_scale, row_slope[h], row_dist[h], row_pos[h] - j) : -INFINITY;
+                    const float v = ok ? score_of<FORM>(p, s[n][2 * h + e] * p.softmax_scale, key[n][e], row_slope[h], row_dist[h], row_pos[h] - j) : -INFINITY;
                     s[n][2 * h + e] = v;
                     mx = fmaxf(mx, v);
                 }
@@ -342,8 +350,8 @@ int launch(const AttentionParams& p, const StepTokens& b, const PagedCache& c, c
     const size_t tiles = (size_t)WARPS * 4 * TILE * 16 * NK * 2;
     const size_t merge = (size_t)WARPS * 16 * 16 * NK * 4 + WARPS * 16 * 2 * 4;
     const size_t smem = tiles > merge ? tiles : merge;
-    const int form = score_form_of(p);
-    auto k = form == FORM_DISTANCE ? attn_mma_kernel<NK, FORM_DISTANCE> : form == FORM_CAP ? attn_mma_kernel<NK, FORM_CAP> : attn_mma_kernel<NK, FORM_PLAIN>;
+    const int form = score_form_of(p, c);
+    auto k = form == FORM_ANY ? attn_mma_kernel<NK, FORM_ANY> : form == FORM_CAP ? attn_mma_kernel<NK, FORM_CAP> : attn_mma_kernel<NK, FORM_PLAIN>;
     if (smem > 48 * 1024 &&
         cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
         return SPITE_LAUNCH_FAILED;

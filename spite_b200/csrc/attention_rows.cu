@@ -117,6 +117,18 @@ __global__ void __launch_bounds__(WARPS * 32) attn_rows_kernel(const AttentionPa
     const __nv_bfloat16* kbase = (const __nv_bfloat16*)c.kv;
     const __nv_bfloat16* vbase = kbase + c.v_offset;
 
+    const bool scaled = FORM == FORM_ANY && c.key_scale != nullptr;
+    float2 next_scale[4];                                   // the factors of this lane's keys of the tile that comes next
+#pragma unroll
+    for (int n = 0; n < 4; ++n) next_scale[n] = make_float2(1.f, 1.f);
+    auto ask_scales = [&](int ti) {
+        if (!scaled || ti >= tile_hi) return;
+        const float* f = key_scale_of(c, max(table[ti * TILE / c.page_size], 0), kvh, ti * TILE) + 2 * cc;
+#pragma unroll
+        for (int n = 0; n < 4; ++n) next_scale[n] = make_float2(f[8 * n], f[8 * n + 1]);
+    };
+    ask_scales(tile_lo);
+
     auto issue = [&](int stage, int ti) {
         const int j0 = ti * TILE;
         const int page = table[j0 / c.page_size];
@@ -146,6 +158,10 @@ __global__ void __launch_bounds__(WARPS * 32) attn_rows_kernel(const AttentionPa
     }
     int stage = 0;
     for (int ti = tile_lo; ti < tile_hi; ++ti) {
+        float key[4][2];
+#pragma unroll
+        for (int n = 0; n < 4; ++n) { key[n][0] = next_scale[n].x; key[n][1] = next_scale[n].y; }
+        ask_scales(ti + 1);
         cp_async_wait<STAGES - 2>();
         __syncthreads();                                     // tile ti has landed; the stage refilled below is free
         {
@@ -189,7 +205,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_rows_kernel(const AttentionPa
                     for (int e = 0; e < 2; ++e) {
                         const int j = j0 + 8 * n + 2 * cc + e;
                         const bool ok = row_ok[h] && j >= row_lo[h] && j <= row_pos[h];
-                        const float v = ok ? score_of<FORM>(p, s[n][2 * h + e] * p.softmax_scale, row_slope[h], row_dist[h], row_pos[h] - j) : -INFINITY;
+                        const float v = ok ? score_of<FORM>(p, s[n][2 * h + e] * p.softmax_scale, key[n][e], row_slope[h], row_dist[h], row_pos[h] - j) : -INFINITY;
                         s[n][2 * h + e] = v;
                         mx = fmaxf(mx, v);
                     }
@@ -254,8 +270,8 @@ template <int NK>
 int launch(const AttentionParams& p, const StepTokens& b, const PagedCache& c, const AttnMmaExtra& x,
            int n_blocks, cudaStream_t st) {
     const size_t smem = (size_t)STAGES * 2 * TILE * 16 * NK * 2;
-    const int form = score_form_of(p);
-    auto k = form == FORM_DISTANCE ? attn_rows_kernel<NK, FORM_DISTANCE> : form == FORM_CAP ? attn_rows_kernel<NK, FORM_CAP> : attn_rows_kernel<NK, FORM_PLAIN>;
+    const int form = score_form_of(p, c);
+    auto k = form == FORM_ANY ? attn_rows_kernel<NK, FORM_ANY> : form == FORM_CAP ? attn_rows_kernel<NK, FORM_CAP> : attn_rows_kernel<NK, FORM_PLAIN>;
     if (smem > 48 * 1024 &&
         cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
         return SPITE_LAUNCH_FAILED;

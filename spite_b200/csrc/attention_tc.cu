@@ -92,6 +92,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
     constexpr int KT_BYTES = NKB * BN * 128;             // one K tile, one V tile
     extern __shared__ __align__(1024) unsigned char smem[];   // [Q0][Q1][K ring][V ring], each 1024-byte aligned
     __shared__ Barriers bars;
+    __shared__ __align__(16) float key_scales[FORM == FORM_ANY ? 8 : 1][BN];    // a softmax warp's copy of its tile's keys' factors
     pdl_wait();
     pdl_launch_dependents();
 
@@ -310,13 +311,31 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 const float cap_raw = p.score_softcap > 0.f ? p.score_softcap / p.softmax_scale : 0.f;
                 const float cap_arg = p.score_softcap > 0.f ? 2.f * LOG2E * p.softmax_scale / p.score_softcap : 0.f;
                 // a number per distance, brought into the units of the raw scores as it is added
-                const float* dist_row = FORM == FORM_DISTANCE ? distance_row_of(p, head) : nullptr;
+                const float* dist_row = FORM == FORM_ANY ? distance_row_of(p, head) : nullptr;
                 const float per_scale = 1.f / p.softmax_scale;
+                // the keys' factors: a lane asks for two of the next tile's while this tile is worked on
+                const bool scaled = FORM == FORM_ANY && c.key_scale != nullptr;
+                float* const scale_s = key_scales[FORM == FORM_ANY ? warp - 3 : 0];
+                float2 next_scale = make_float2(1.f, 1.f);
+                auto ask_scales = [&](int li) {
+                    if (!scaled || li >= n_own) return;
+                    const int j = k_begin + (first + li) * BN;
+                    int page = table[j / c.page_size];
+                    if (page < 0 || page >= c.n_pages) page = 0;        // (as the loader: behind every row's window)
+                    next_scale = *(const float2*)(key_scale_of(c, page, kvh, j) + 2 * lane);
+                };
+                ask_scales(0);
                 const unsigned lane_base = tmem_g + ((unsigned)(quarter * 32) << 16);
                 float m_ref = -INFINITY, l = 0.f;
                 bool ok = true;
                 for (int li = 0; li < n_own; ++li) {
                     const int sb = li & 1;
+                    if (scaled) {
+                        __syncwarp();                                   // every lane has read the tile before's
+                        *(float2*)(scale_s + 2 * lane) = next_scale;
+                        __syncwarp();
+                        ask_scales(li + 1);
+                    }
                     ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(&gb.s_full[sb]), (li >> 1) & 1, abort_flag, err_word, 3, wait_limit));
                     if (!ok) break;
                     fence_after();
@@ -330,7 +349,14 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                     // element with a constant that the compiler knows; the first is the same for the whole tile and joins
                     // the maximum and the exponent's offset below.
                     float tile_bias = biased ? bias_raw * (float)(j0 - pos) : 0.f;
-                    if (FORM == FORM_CAP || (FORM == FORM_DISTANCE && cap_raw > 0.f)) {
+                    if (scaled) {
+#pragma unroll
+                        for (int e = 0; e < BN; e += 4) {
+                            const float4 f = *(const float4*)(scale_s + e);
+                            s[e] *= f.x; s[e + 1] *= f.y; s[e + 2] *= f.z; s[e + 3] *= f.w;
+                        }
+                    }
+                    if (FORM == FORM_CAP || (FORM == FORM_ANY && cap_raw > 0.f)) {
                         // cap tanh(s scale / cap) in units of the raw scores: tanh(x) = 1 - 2 / (e^(2x) + 1), whose absolute
                         // error (a few float32 roundings of a number below one) times the cap is far below a bfloat16 weight's
 #pragma unroll
@@ -341,7 +367,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
 #pragma unroll
                         for (int e = 0; e < BN; ++e) s[e] = fmaf(bias_raw, (float)e, s[e]);
                     }
-                    if constexpr (FORM == FORM_DISTANCE) {
+                    if (FORM == FORM_ANY && dist_row) {
                         // The numbers change with the distance near the query and hardly further away: where every row of the
                         // warp has one number for its whole tile, that joins the tile's common term; else each key's is read
                         // (a row's distances lie side by side, the repeated ends take the tile's overhang).
@@ -477,8 +503,8 @@ int launch(const AttentionParams& p, const StepTokens& b, const PagedCache& c, c
         if (!make_map(&mv, (const __nv_bfloat16*)c.kv + c.v_offset, 2, dims, strides, box)) return SPITE_LAUNCH_FAILED;
     }
     const size_t smem = 2 * (size_t)NKB * BM * 128 + 2 * ST * (size_t)NKB * BN * 128;
-    const int form = score_form_of(p);
-    auto k = form == FORM_DISTANCE ? attn_tc_kernel<NKB, FORM_DISTANCE> : form == FORM_CAP ? attn_tc_kernel<NKB, FORM_CAP> : attn_tc_kernel<NKB, FORM_PLAIN>;
+    const int form = score_form_of(p, c);
+    auto k = form == FORM_ANY ? attn_tc_kernel<NKB, FORM_ANY> : form == FORM_CAP ? attn_tc_kernel<NKB, FORM_CAP> : attn_tc_kernel<NKB, FORM_PLAIN>;
     if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
         return SPITE_LAUNCH_FAILED;
     const long long items = (long long)n_blocks * nkv;
@@ -507,7 +533,7 @@ SPITE_API int spite_paged_attention_tc(const AttentionParams* p, const StepToken
     if (x->tokens_per_block * G > BM) return SPITE_BAD_ARG;
     if ((long long)n_blocks * c->num_kv_heads > 0x7fffffffll || p->num_heads > 256 * c->num_kv_heads) return SPITE_UNSUPPORTED;
     if ((long long)c->n_pages * c->num_kv_heads * c->page_size > 0x7fffffffll) return SPITE_UNSUPPORTED;   // TMA coordinates are int32
-    if ((((uintptr_t)p->q | (uintptr_t)p->out | (uintptr_t)c->kv) & 15) || (c->v_offset & 7)) return SPITE_UNSUPPORTED;
+    if ((((uintptr_t)p->q | (uintptr_t)p->out | (uintptr_t)c->kv | (uintptr_t)c->key_scale) & 15) || (c->v_offset & 7)) return SPITE_UNSUPPORTED;
     if (b->n_tokens == 0 || n_blocks == 0) return SPITE_OK;
     cudaStream_t st = (cudaStream_t)stream;
     return c->head_dim == 64 ? launch<1>(*p, *b, *c, *x, n_blocks, n_sm, st) : launch<2>(*p, *b, *c, *x, n_blocks, n_sm, st);

@@ -81,6 +81,11 @@ __device__ __forceinline__ void tma_load_2d_hint(unsigned dst, const CUtensorMap
     asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes.L2::cache_hint [%0], [%1, {%2, %3}], [%4], %5;\n"
                  ::"r"(dst), "l"((unsigned long long)map), "r"(x), "r"(y), "r"(bar), "l"(policy) : "memory");
 }
+// Untiled: `bytes` (a multiple of 16) from global memory, both addresses 16-byte aligned.
+__device__ __forceinline__ void bulk_load(unsigned dst, const void* src, unsigned bytes, unsigned bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];\n"
+                 ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
+}
 __device__ __forceinline__ unsigned long long l2_evict_first() {
     unsigned long long policy;
     asm volatile("createpolicy.fractional.L2::evict_first.b64 %0, 1.0;\n" : "=l"(policy));

@@ -106,10 +106,10 @@ class Model:
                 continue
             a, b = have[0], req[0]
             if a is not None and b is not None and a.window != b.window and have[1] == req[1] \
-                    and (a.num_kv_heads, a.head_dim, a.planes) == (b.num_kv_heads, b.head_dim, b.planes):
+                    and (a.num_kv_heads, a.head_dim, a.planes, a.key_scales) == (b.num_kv_heads, b.head_dim, b.planes, b.key_scales):
                 # layers that read one cache through different windows: every layer masks by its own, and the pages go
                 # back by the rule that keeps what either still reads
-                self._cache_specs[call.cache] = (PagedKV(a.window.union(b.window), a.num_kv_heads, a.head_dim, a.planes), have[1])
+                self._cache_specs[call.cache] = (PagedKV(a.window.union(b.window), a.num_kv_heads, a.head_dim, a.planes, a.key_scales), have[1])
             elif have != req:
                 raise ConfigError(
                     f"cache {call.cache} is shared by layers whose mixers need different caches: {have} vs {req}")

@@ -232,7 +232,9 @@ class KernelSet:
         the per-head norm takes its mean over them.
         `value_rotation`: a `parts.Rotation` over the leading elements of a value head: a value turns by its own position
         before it is cached.  `values_are_keys`: a row of qkv holds q and k heads alone ((nq + nkv) hd columns, `bias` too),
-        and the value of a position is its key as projected (with its bias, before norm and rotation)."""
+        and the value of a position is its key as projected, bias included; there is no rotation and no gain for k.  The cache has
+        one plane, which takes the keys as projected, and a factor per key (`cache.key_scale` [pages, nkv, page_size]), which
+        receives what the norm multiplies the key by (1 without a norm)."""
         raise NotImplementedError
 
     def paged_attention(self, q, out, batch, cache, *, num_heads, window, softmax_scale, cache_settled=False,
@@ -248,6 +250,8 @@ class KernelSet:
         `distance_bias`, a `DistanceBias`: a number per head and distance is added to a score (behind scale and cap).
         `head_gates` float32 [M, nq]: head h's output for token m is multiplied by head_gates[m, h].
         A cache with one plane (`cache.kv.shape[0] == 1`) holds keys only, and the value of a position is its key row.
+        A cache with `key_scale` (float32 [pages, nkv, page_size]): the product with a key row is multiplied by the key's factor
+        (ahead of scale and cap).
         `cache_settled`: the caller promises that the cache rows of positions before each request's first
         token of this step were written by earlier steps (not by the one or two kernels launched just
         before this call), so a kernel may fetch them while the kernel before still runs."""

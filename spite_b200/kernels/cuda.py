@@ -40,7 +40,7 @@ class StepTokens(C.Structure):
 
 class PagedCache(C.Structure):
     _fields_ = [("kv", C.c_void_p), ("v_offset", C.c_longlong), ("n_pages", C.c_int),
-                ("page_size", C.c_int), ("num_kv_heads", C.c_int), ("head_dim", C.c_int)]
+                ("page_size", C.c_int), ("num_kv_heads", C.c_int), ("head_dim", C.c_int), ("key_scale", C.c_void_p)]
 
 
 class QkPrepareParams(C.Structure):
@@ -856,7 +856,9 @@ class CudaKernels(KernelSet):
     def _paged(self, cache):
         kv = cache.kv                       # [planes, pages, nkv, page_size, hd]; one plane: the key rows are the values
         self._t(kv, self.dtype, "cache")
-        return PagedCache(kv=kv.data_ptr(), v_offset=kv.stride(0) if kv.shape[0] == 2 else 0, n_pages=kv.shape[1],
+        if cache.key_scale is not None and tuple(self._t(cache.key_scale, torch.float32, "key_scale").shape) != tuple(kv.shape[1:4]):
+            raise KernelError("a cache's key factors are [pages, kv heads, page_size]")
+        return PagedCache(key_scale=_ptr(cache.key_scale), kv=kv.data_ptr(), v_offset=kv.stride(0) if kv.shape[0] == 2 else 0, n_pages=kv.shape[1],
                           page_size=kv.shape[3], num_kv_heads=kv.shape[2], head_dim=kv.shape[4])
 
     def qk_prepare(self, qkv, q_out, batch, cache, *, num_heads, rotation, qk_norm, temperature,
@@ -864,8 +866,9 @@ class CudaKernels(KernelSet):
                    values_are_keys=False):
         self._t(qkv, self.dtype, "qkv"); self._t(q_out, self.dtype, "q_out")
         head_dim = cache.kv.shape[4]
-        if values_are_keys and (q_only or value_mix is not None or value_rotation is not None):
-            raise KernelError("qk_prepare: values that are the keys are neither borrowed, blended nor rotated")
+        if values_are_keys and (q_only or value_mix is not None or value_rotation is not None or rotation is not None
+                                or (qk_norm is not None and qk_norm.k_gain is not None)):
+            raise KernelError("qk_prepare: values that are the keys are neither borrowed, blended nor rotated, their norm has no gain")
         n_cols = (num_heads + (0 if q_only else (1 if values_are_keys else 2) * cache.kv.shape[2])) * head_dim
         if qkv.shape[1] < n_cols:
             raise KernelError(f"qk_prepare: rows of {qkv.shape[1]} elements cannot hold the heads' {n_cols}")
@@ -873,8 +876,9 @@ class CudaKernels(KernelSet):
             raise KernelError(f"qk_prepare: the bias has {bias.numel()} elements, the heads have {n_cols}")
         if q_only and cache.write:
             raise KernelError("qk_prepare: a layer without keys and values of its own cannot append to the cache")
-        if cache.kv.shape[0] != 2:
-            raise KernelError("qk_prepare appends keys and values: the cache needs both planes")
+        if cache.kv.shape[0] != (1 if values_are_keys else 2) or values_are_keys != (cache.key_scale is not None):
+            raise KernelError("qk_prepare appends keys and values: the cache needs both planes; keys that are the values need one, "
+                              "and a factor per key")
         inv_freq, pairing, rotary_dim, amplitude = None, 0, head_dim, 1.0
         v_other, v_stride, v_head, v_dim, v_lam = None, 0, 0, 0, 0.0
         if value_mix is not None:

@@ -27,7 +27,7 @@ from ..cache import FixedState, PagedKV, Window
 from ..config.specs import ConfigError, PartSpec
 from ..kernels.api import DistanceBias
 from .base import Mixer, ParamSpec, QkNorm, build_part, register_mixer
-from .position import distance_rows
+from .position import distance_reach, distance_rows
 
 
 @register_mixer("paged_attention")
@@ -63,7 +63,9 @@ class PagedAttention(Mixer):
         cached, and a head's result at position i is turned back by i before the output projection (so a value
         enters turned by its distance, and nothing else of the attention knows about it).
         `output_bias` (default: as `bias`): whether the output projection has one.  `values_are_keys`: there is no value
-        projection; a position's value is its key as projected, bias included, before norm and rotation.
+        projection; a position's value is its key as projected, bias included (no rotation, no gain for k).  The cache then holds
+        one row per position, the key as projected, and the factor that the norm multiplies it by: half the bytes of a key
+        and a value.
         `distance_table` (rows, far): the parameter `distance_bias` [rows, heads] is added to the scores (behind scale and cap),
         the row by the distance between query and key as `distance_rows` says."""
         super().__init__(ctx)
@@ -80,6 +82,8 @@ class PagedAttention(Mixer):
         self.values_are_keys = bool(values_are_keys)
         if self.values_are_keys and (kv_shared or value_mix or conv_taps is not None or value_rotation is not None):
             raise ConfigError("values that are the keys cannot be borrowed, blended, convolved or rotated")
+        if self.values_are_keys and qk_norm_gain:
+            raise ConfigError("values that are the keys go with a norm of the keys without a gain")
         if self.values_are_keys and value_dim not in (None, head_dim):
             raise ConfigError(f"values that are the keys have the keys' size {head_dim}, not {value_dim}")
         if self.kv_shared and value_mix:
@@ -121,6 +125,8 @@ class PagedAttention(Mixer):
         if rot is not None and (rot.rotary_dim or self.kd) > self.kd:
             raise ConfigError(f"{rot.rotary_dim} rotating elements in a head of {self.kd}")
         # (the per-head norm is told the key's own size and takes its mean over that)
+        if self.values_are_keys and rot is not None:
+            raise ConfigError("values that are the keys go without a rotation")
         may_pad = rot is None or rot.rotary_dim is not None
         if self.kd % 2 and not may_pad:
             raise ConfigError(f"head_dim {head_dim} must be even where heads rotate or are normed")
@@ -159,8 +165,12 @@ class PagedAttention(Mixer):
         self._distance_rows = self.distance_bias = None
         if self.distance_table is not None:
             rows, far = self.distance_table
-            # what lies beyond `far` shares its row; a window may end before that
-            self._distance_rows = distance_rows(rows, far, far + 1 if self.window.kind == "full" else min(self.window.size, far + 1))
+            # what lies beyond some distance shares its row; a window may end before that
+            reach = distance_reach(rows, far)
+            sizes = [n for n in (None if reach is None else reach + 1, None if self.window.kind == "full" else self.window.size) if n]
+            if not sizes:
+                raise ConfigError(f"a table by distance of {rows} rows and a far distance of {far} never ends; give the layer a window")
+            self._distance_rows = distance_rows(rows, far, min(sizes))
         self.wqkv = self.wo = None
 
     def param_specs(self):
@@ -264,6 +274,8 @@ class PagedAttention(Mixer):
         state = None
         if self.conv_taps is not None and self.conv_taps > 1:
             state = FixedState(((self.conv_taps - 1) * (self.nq + 2 * self.nkv) * self.hd,), torch.float32)
+        if self.values_are_keys:
+            return PagedKV(self.window, self.nkv, self.hd, planes=1, key_scales=True), state
         return PagedKV(self.window, self.nkv, self.hd), state
 
     @property

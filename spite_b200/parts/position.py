@@ -112,19 +112,26 @@ class RotaryYarn(PositionEncoding):
 def distance_rows(rows: int, far: int, length: int) -> list[int]:
     """Which row of a table serves each distance 0 .. length - 1 (the T5 kind of buckets, one-sided): the first half of the
     rows one distance each, the others ranges that grow geometrically up to the distance `far`, the last row everything
-    beyond.  With h = rows // 2: n < h: n; else min(rows - 1, h + floor(ln(n / h) / ln(far / h) (rows - h)))."""
+    beyond.  With h = rows // 2: n < h: n; else min(rows - 1, h + floor(ln(n / h) / ln(far / h) (rows - h))).  (Where `far` does
+    not lie beyond h the second half has no ranges to speak of: from h on the last row, if `far` is h, or what the formula's
+    negative logarithm gives.)"""
+    if rows < 1 or far < 1:
+        raise ConfigError(f"a table by distance needs rows ({rows}) and a far distance ({far})")
     half = rows // 2
-    if rows < 2 or far <= half:
-        raise ConfigError(f"a table of {rows} rows by distance needs two rows and a far distance ({far}) beyond half of them")
     out = []
     for n in range(length):
-        if n < half:
-            out.append(n)
+        if n < half or half in (0, far):
+            out.append(n if n < half else rows - 1)
             continue
         x = math.log(n / half) / math.log(far / half) * (rows - half)
         # (a border that falls on a whole number belongs to the row above it, whichever way the logarithms were rounded)
-        out.append(min(rows - 1, half + math.floor(x + 1e-9)))
+        out.append(max(0, min(rows - 1, half + math.floor(x + 1e-9))))
     return out
+
+
+def distance_reach(rows: int, far: int) -> int | None:
+    """The distance from which on `distance_rows` stays the same (None: nowhere)."""
+    return far if far >= rows // 2 else None
 
 
 @register_position("rotary_halves")

@@ -403,7 +403,7 @@ class TorchReferenceKernels(KernelSet):
         if bias is not None:
             x = x + bias.to(self.acc)[None, :]
         x = x.reshape(M, -1, hd)
-        q, k, v = x[:, :nq], x[:, nq:nq + nkv], x[:, nq:] if values_are_keys else x[:, nq + nkv:]
+        q, k, v = x[:, :nq], x[:, nq:nq + nkv], x[:, nq + nkv:]
         if q_only:
             assert not cache.write
             k = q[:, :0]
@@ -424,6 +424,7 @@ class TorchReferenceKernels(KernelSet):
             t = t * (1.0 / torch.sqrt(t.pow(2).sum(-1, keepdim=True) / (norm_dim or hd) + qk_norm.eps))
             return t if gain is None else t * gain.to(t.device, self.acc)
 
+        raw = k
         if qk_norm is not None and qk_norm.before_rotation:
             q, k = norm(q, qk_norm.q_gain), norm(k, qk_norm.k_gain)
         if rotation is not None:
@@ -458,6 +459,12 @@ class TorchReferenceKernels(KernelSet):
                 p = int(pos[t])
                 page = int(bt[seg[t], p // P])
                 assert page >= 0, "write into a page that is not held"
+                if values_are_keys:                              # the row as projected, what the norm makes of it beside it
+                    assert rotation is None and kv.shape[0] == 1
+                    kv[0, page, :, p % P, :] = raw[t].to(kv.dtype)
+                    rms = torch.sqrt(raw[t].pow(2).sum(-1) / (norm_dim or hd) + qk_norm.eps) if qk_norm is not None else torch.ones(nkv)
+                    cache.key_scale[page, :, p % P] = (1.0 / rms).to(torch.float32)
+                    continue
                 kv[0, page, :, p % P, :] = k[t].to(kv.dtype)
                 kv[1, page, :, p % P, :] = v[t].to(kv.dtype)
 
@@ -540,8 +547,12 @@ class TorchReferenceKernels(KernelSet):
             assert bool((pages >= 0).all()), "read from a page that was given back"
             K = kv[0, pages, :, js % P, :].to(self.acc)          # [n, nkv, hd]
             V = kv[kv.shape[0] - 1, pages, :, js % P, :].to(self.acc)     # (one plane: the key rows are the values)
+            if cache.key_scale is not None:
+                factor = cache.key_scale[pages, :, js % P].to(self.acc)          # [n, nkv]
             for h in range(nq):
                 s = (K[:, h // group, :] @ qf[t, h]) * softmax_scale
+                if cache.key_scale is not None:
+                    s = s * factor[:, h // group]
                 if score_softcap is not None:
                     s = score_softcap * torch.tanh(s / score_softcap)
                 if head_slopes is not None:

@@ -183,7 +183,7 @@ def test_router_entry_point(libs):
                  offs=ptr(offs), rows=ptr(rows))
         a.update(kw)
         return lib.spite_moe_route(1, a["x"], a["w"], a["M"], a["d"], a["E"], a["k"], a["ids"], a["wts"],
-                                   a["logits"], a["offs"], a["rows"], a.get("scoring", 0), None, None, None)
+                                   a["logits"], a["offs"], a["rows"], a.get("scoring", 0), None, None, None, None)
     for kw in (dict(x=None), dict(w=None), dict(ids=None), dict(wts=None), dict(offs=None), dict(rows=None),
                dict(M=-1), dict(d=0), dict(E=0), dict(k=0), dict(k=E + 1), dict(scoring=2), dict(scoring=3)):
         assert call(**kw) == BAD_ARG, kw
@@ -205,8 +205,18 @@ def test_scan_stream_and_shift_entry_points(libs):
                 dim=N, vdim=P)
     ss = lambda **c: scan.spite_state_space_scan(C.byref(ScanParams(**dict(good, **c))), ptr(a), C.c_longlong(H), ptr(one), ptr(one), None)
     dec = lambda **c: scan.spite_decay_scan(C.byref(ScanParams(**dict(good, skip=None, w=w.data_ptr(), w_stride=H * N, **c))), ptr(one), ptr(one), None)
+    gla = lambda rank=3, tau=4.0, a2=one, b=one, low=a, stride=4, **c: scan.spite_gated_linear_scan(
+        C.byref(ScanParams(**dict(good, scalars=None, skip=None, w=w.data_ptr(), w_stride=H * N, out_scale=1.0, **c))), ptr(low),
+        C.c_longlong(stride), ptr(a2), ptr(b), rank, C.c_float(tau), None)
     for call in (ss, dec):
-        for c in (dict(q=None), dict(k=None), dict(v=None), dict(out=None), dict(state=None), dict(scalars=None), dict(cu_seqlens=None),
+        assert call(scalars=None) == BAD_ARG
+    for c in (dict(rank=0), dict(rank=5), dict(tau=0.0), dict(tau=float("nan")), dict(a2=None), dict(b=None), dict(low=None), dict(kv_heads=1)):
+        assert gla(**c) == BAD_ARG, c
+    assert scan.spite_gated_linear_scan(None, ptr(a), C.c_longlong(4), ptr(one), ptr(one), 3, C.c_float(4.0), None) == BAD_ARG
+    assert scan.spite_gated_linear_scan(C.byref(ScanParams(**dict(good, skip=None))), ptr(a), C.c_longlong(4), ptr(one), ptr(one), 3,
+                                        C.c_float(4.0), None) == BAD_ARG                      # no room for the decays
+    for call in (ss, dec, gla):
+        for c in (dict(q=None), dict(k=None), dict(v=None), dict(out=None), dict(state=None), dict(cu_seqlens=None),
                   dict(slots=None), dict(heads=0), dict(heads=3, kv_heads=2), dict(dim=0), dict(vdim=0), dict(slot_stride=7), dict(out_stride=3),
                   dict(n_tokens=-1), dict(n_segments=-1), dict(q_stride=0)):
             assert call(**c) == BAD_ARG, c
@@ -400,6 +410,11 @@ def test_attention_refuses_malformed_calls(libs, which):
     k = attention_case()
     k["p"].window_kind, k["p"].window_size = 1, 0                        # a chunk window of no keys
     assert call(k) == BAD_ARG and untouched(k["out"]), name
+    table = torch.zeros((4, 132), dtype=torch.float32, device=DEV)          # numbers by distance without their runs, without a length
+    for runs, n in ((None, 4), (table.data_ptr(), 0), (table.data_ptr(), -3)):
+        k = attention_case()
+        k["p"].distance_bias, k["p"].distance_runs, k["p"].distance_len = table.data_ptr(), runs, n
+        assert call(k) == BAD_ARG and untouched(k["out"]), name
 
 
 def test_attention_refuses_sizes_outside_its_domain(libs):
@@ -469,6 +484,19 @@ def test_prepare_refuses_malformed_calls(libs):
         setattr(k[struct], field, value)
         assert lib.spite_qk_prepare(1, C.byref(k["qp"]), C.byref(k["b"]), C.byref(k["c"]), None) == BAD_ARG, (struct, field)
         torch.cuda.synchronize()
+        assert untouched(k["out"]) and float(k["kv"].float().abs().sum()) == 0.0
+    some = torch.ones(1 << 12, dtype=torch.float32, device=DEV)
+    for edits in (dict(q_only=1), dict(v_other=some.data_ptr()), dict(v_inv_freq=some.data_ptr(), v_rotary_dim=8), dict(qkv_stride=5 * 64),
+                  dict(inv_freq=some.data_ptr(), rotary_dim=8), dict(k_gain=some.data_ptr()), dict(two_planes=1), dict(no_factors=1)):
+        k = attention_case()                                     # values that are the keys, and what does not go with them
+        k["c"].v_offset, k["c"].key_scale = 0, some.data_ptr()
+        if edits.pop("two_planes", 0):
+            k["c"].v_offset = k["kv"].stride(0)
+        if edits.pop("no_factors", 0):
+            k["c"].key_scale = None
+        for field, value in dict(edits, values_are_keys=1).items():
+            setattr(k["qp"], field, value)
+        assert lib.spite_qk_prepare(1, C.byref(k["qp"]), C.byref(k["b"]), C.byref(k["c"]), None) == BAD_ARG, edits
         assert untouched(k["out"]) and float(k["kv"].float().abs().sum()) == 0.0
     k = attention_case()
     assert lib.spite_qk_prepare(9, C.byref(k["qp"]), C.byref(k["b"]), C.byref(k["c"]), None) == BAD_ARG
