@@ -56,6 +56,8 @@ def main(argv=None):
     ap.add_argument("--sink", type=float, default=None, help="attention cases run with a sink of this score in the softmax")
     ap.add_argument("--bias", action="store_true", help="attention cases run with a distance bias, a learned sink and a gate per head")
     ap.add_argument("--cap", type=float, default=None, help="attention cases run with scores capped at this")
+    ap.add_argument("--wide", action="store_true", help="decode attention in its form of sixteen rows whatever the heads a kv head")
+    ap.add_argument("--factors", action="store_true", help="attention cases run on keys that are the values, with a factor per key, alone")
     ap.add_argument("--distance", action="store_true", help="attention cases run with a number per head and distance (32 buckets up to "
                                                           "the context) over keys that are the values, with a factor per key")
     ap.add_argument("--latent", action="store_true", help="attention cases run on a cache of one plane: 16 query heads on one kv head "
@@ -64,6 +66,8 @@ def main(argv=None):
     dev = "cuda:0"
     torch.cuda.set_device(0)
     ks = CudaKernels(torch.bfloat16, dev)
+    if args.wide:
+        ks.attention_narrow_rows = 0
     pk, src = peaks()
     flush = torch.empty(256 * 1024 * 1024, dtype=torch.uint8, device=dev)       # larger than L2
     bf = torch.bfloat16
@@ -226,9 +230,10 @@ def main(argv=None):
 
     # ---- attention over the paged cache
     P = 64
+    keys_alone = args.distance or args.factors
+    one_plane = args.latent or keys_alone
     sink = "" if args.sink is None else f" sink={args.sink}"
-    sink += ("" if args.cap is None else f" cap={args.cap}") + (" distance, keys as values" if args.distance else "")
-    one_plane = args.latent or args.distance
+    sink += ("" if args.cap is None else f" cap={args.cap}") + (" distance" if args.distance else "") + (" keys as values" if keys_alone else "")
     sink += (" bias+sinks+gates" if args.bias else "") + (" one plane, 16 heads on 1" if args.latent else "")
     if args.latent:
         nq, nkv, hd = 16, 1, 128
@@ -244,7 +249,7 @@ def main(argv=None):
         def make():
             kv = (torch.randn((1 if one_plane else 2, n_req * pages_per, nkv, P, hd), device=dev) * 0.5).to(bf)
             q, out = rnd(off, nq * hd), torch.empty((off, nq * hd), dtype=bf, device=dev)
-            factors = torch.rand((n_req * pages_per, nkv, P), device=dev) + 0.5 if args.distance else None
+            factors = torch.rand((n_req * pages_per, nkv, P), device=dev) + 0.5 if keys_alone else None
             cache = LayerCache(0, kv, None, P, False, factors)
             more = {} if args.cap is None else {"score_softcap": args.cap}
             if args.distance:
@@ -261,7 +266,7 @@ def main(argv=None):
         seen = sum(min(p + 1, ctx) - win.lowest_visible(p) for p in range(ctx - n_new, ctx)) / n_new
         if n_new == 1:
             # short launches: back to back over rotating copies of the cache, so no launch gap is counted
-            nbytes = int(n_req * seen * nkv * (hd * 2 * (1 if one_plane else 2) + (4 if args.distance else 0)))
+            nbytes = int(n_req * seen * nkv * (hd * 2 * (1 if one_plane else 2) + (4 if keys_alone else 0)))
             report(fam, f"requests={n_req} context={ctx} window={window[0]}{sink}", timed_rotating(make, nbytes), nbytes=nbytes)
             return
         report(fam, f"tokens={n_new} context={ctx} window={window[0]}{sink}", timed(make()),

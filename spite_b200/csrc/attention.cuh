@@ -139,6 +139,32 @@ __device__ __forceinline__ float slope_of(const AttentionParams& p, int head) {
 __device__ __forceinline__ float capped(const AttentionParams& p, float s) {
     return p.score_softcap > 0.f ? p.score_softcap * tanhf(s / p.score_softcap) : s;
 }
+// The same for the tensor-core kernels, without a division or a call: with t = s / cap, s (1 - t^2/3 + 2 t^4/15 - ...), the
+// Taylor series of the hyperbolic tangent to t^11, where |t| <= CAP_SERIES (what is left out is below 1e-7 of the result), and
+// cap (1 - 2 / (e^(2t) + 1)) beyond, whose absolute error is a few float32 roundings of the cap.
+#define CAP_SERIES 0.4f
+#define CAP_C1 (-1.f / 3.f)
+#define CAP_C2 (2.f / 15.f)
+#define CAP_C3 (-17.f / 315.f)
+#define CAP_C4 (62.f / 2835.f)
+#define CAP_C5 (-1382.f / 155925.f)
+__device__ __forceinline__ float reciprocal_approx(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float exp2_approx(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float capped_series(float s, float cap, float inv_cap) {
+    const float t = s * inv_cap, y = t * t;
+    float r = s * fmaf(y, fmaf(y, fmaf(y, fmaf(y, fmaf(y, CAP_C5, CAP_C4), CAP_C3), CAP_C2), CAP_C1), 1.f);
+    if (fabsf(t) > CAP_SERIES)
+        r = fmaf(-2.f * cap, reciprocal_approx(exp2_approx(t * 2.8853900817779268f) + 1.f), cap);      // (e^(2t) = 2^(2t / ln 2))
+    return r;
+}
 // The tensor-core kernels are compiled in three forms: scores as they are, capped, and with everything else (a factor per key,
 // a number per distance, a cap or none) chosen at run time.  With the choice of the cap made per score at run time, the decode
 // kernel took a tenth longer without any cap.
@@ -150,12 +176,21 @@ static inline bool distance_bias_ok(const AttentionParams* p) {
     return !p->distance_bias || (p->distance_runs && p->distance_len >= 1 && p->distance_len <= (1 << 24));
 }
 // The score of a visible key n positions before the query, from the product `s` scaled by the softmax's scale; `key` is the
-// key's own factor (1 without one).
+// key's own factor (1 without one), `inv_cap` 1 / score_softcap (0 without a cap), `number` what the distance adds.
 template <int FORM>
-__device__ __forceinline__ float score_of(const AttentionParams& p, float s, float key, float slope, const float* row, int n) {
-    if constexpr (FORM == FORM_CAP) return p.score_softcap * tanhf(s / p.score_softcap) - slope * (float)n;
-    else if constexpr (FORM == FORM_ANY) return capped(p, s * key) - slope * (float)n + (row ? row[min(n, p.distance_len - 1)] : 0.f);
-    else return s - slope * (float)n;
+__device__ __forceinline__ float score_of(const AttentionParams& p, float s, float key, float inv_cap, float slope, float number, int n) {
+    if constexpr (FORM == FORM_PLAIN) return s - slope * (float)n;
+    else {
+        if constexpr (FORM == FORM_ANY) s *= key;
+        if (FORM == FORM_CAP || inv_cap > 0.f) s = capped_series(s, p.score_softcap, inv_cap);
+        s -= slope * (float)n;
+        return FORM == FORM_ANY ? s + number : s;
+    }
+}
+__device__ __forceinline__ float inverse_cap(const AttentionParams& p) { return p.score_softcap > 0.f ? 1.f / p.score_softcap : 0.f; }
+// What the distance n (of either sign; a key behind the query is masked anyway) adds to a score.
+__device__ __forceinline__ float number_at(const AttentionParams& p, const float* row, int n) {
+    return row ? row[min(max(n, 0), p.distance_len - 1)] : 0.f;
 }
 // The factor of the first key of a tile that lies in one page (null without factors).
 __device__ __forceinline__ const float* key_scale_of(const PagedCache& c, int page, int kvh, int position) {

@@ -8,7 +8,9 @@
 // into a ring of shared-memory stages with TMA (cp.async.bulk.tensor, 128-byte swizzle, no cluster
 // multicast) and marks them to leave L2 first; four consumer warps take 16 keys of every tile each
 // (ldmatrix + mma.sync m16n8k16, float32 running maximum and sum per warp) and merge their states in
-// shared memory at the end.  With several splits a block leaves its unnormalised partial result in a
+// shared memory at the end.  Blocks of up to 8 rows (NARROW) have the operands swapped: keys, then elements of the values,
+// are the instruction's 16 rows and the (token, head) rows its 8 columns, so that nothing is computed for rows that are not
+// there: half the instructions and registers of the 16-row form, and half again as many blocks on a multiprocessor.  With several splits a block leaves its unnormalised partial result in a
 // scratch buffer and takes a ticket; the block that takes a (request block, kv head)'s last ticket
 // merges the splits in split order, so no second kernel runs and the order of the additions does
 // not depend on which block came last.
@@ -56,6 +58,12 @@ __device__ __forceinline__ void ldmatrix_x4_trans(unsigned (&r)[4], unsigned add
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
+// An 8 x 8 matrix of 16-bit elements held as lane l's two elements of row l / 4, transposed across the warp.
+__device__ __forceinline__ unsigned transpose_8x8(unsigned v) {
+    unsigned t;
+    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;\n" : "=r"(t) : "r"(v));
+    return t;
+}
 __device__ __forceinline__ unsigned pack_bf16(float a, float b) {
     __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
     return *(unsigned*)&v;
@@ -69,8 +77,8 @@ __device__ __forceinline__ unsigned tile_addr(unsigned base, int r, int ch) {
 }
 
 // NKB = head_dim / 64.  grid (blocks over the served segments, kv heads, splits).
-template <int NKB, int FORM>
-__global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_constant__ CUtensorMap map_k,
+template <int NKB, int FORM, bool NARROW>
+__global__ void __launch_bounds__(THREADS, NARROW ? 3 : 2) attn_decode_kernel(const __grid_constant__ CUtensorMap map_k,
                                                               const __grid_constant__ CUtensorMap map_v,
                                                               const AttentionParams p, const StepTokens b,
                                                               const PagedCache c, const AttnDecodeExtra x,
@@ -153,7 +161,9 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
     pdl_wait();
     pdl_launch_dependents();
 
-    float o[2 * NK][4];
+    // wide: o[n] is rows g and g + 8 of output elements 8 n + 2 cc, + 1; narrow: o[n] is output elements 16 n + g and + 8 of rows
+    // 2 cc, + 1
+    float o[NARROW ? NK : 2 * NK][4];
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
     bool ok = true;
 
@@ -173,6 +183,135 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
                 for (int j = max(0, issued - n_stages); j < issued; ++j)
                     mbar_drain(smem_u32(&tail->full[j % n_stages]), (j / n_stages) & 1, wait_limit);
             }
+        }
+    } else if constexpr (NARROW) {
+        // ---- consumers: warp w takes keys 16 w .. 16 w + 15 of every tile; this lane works on keys g and g + 8 of them for the
+        //      rows 2 cc and 2 cc + 1
+        const int g = lane >> 2, cc = lane & 3;
+        int row_pos[2], row_lo[2];
+        float row_slope[2];
+        const float* row_dist[2];
+        bool row_ok[2];
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            const int row = 2 * cc + h;
+            row_ok[h] = row < n_rows;
+            const int tok = t0 + (row_ok[h] ? row / G : 0), head = kvh * G + (row_ok[h] ? row % G : 0);
+            row_pos[h] = b.positions[tok];
+            row_slope[h] = slope_of(p, head);
+            row_dist[h] = distance_row_of(p, head);
+            row_lo[h] = window_lowest(p.window_kind, p.window_size, row_pos[h]);
+        }
+        unsigned qb[NK][2];                                      // row g of q
+        {
+            const bool q_ok = g < n_rows;
+            const __nv_bfloat16* qrow = (const __nv_bfloat16*)p.q + ((size_t)(t0 + (q_ok ? g / G : 0)) * nq + kvh * G + (q_ok ? g % G : 0)) * HD;
+#pragma unroll
+            for (int kk = 0; kk < NK; ++kk) {
+                const unsigned* src = (const unsigned*)(qrow + 16 * kk + 2 * cc);
+                qb[kk][0] = q_ok ? src[0] : 0u;
+                qb[kk][1] = q_ok ? src[4] : 0u;
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < NK; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
+        const float inv_cap = inverse_cap(p);
+        // What the distances to this lane's keys add, asked for ahead of the wait.  A row's distances fall from tile to tile, and
+        // far from the query one number serves many tiles: it is kept, with the smallest distance it is right for.
+        float number[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
+        int right_from[2] = {0x7fffffff, 0x7fffffff};
+        int s = 0;
+        unsigned ph = 0;
+        for (int ti = sb; ti < se; ++ti, s = (s + 1 == n_stages ? 0 : s + 1), ph ^= (s == 0)) {
+            const int j0 = ti * BN + 16 * warp;                  // this warp's first key
+            if (FORM == FORM_ANY && p.distance_bias) {
+                const int len1 = p.distance_len - 1;
+                int near[2], far[2];                             // the distances of this warp's last and first key of the tile
+#pragma unroll
+                for (int h = 0; h < 2; ++h) {
+                    near[h] = min(max(row_pos[h] - j0 - 15, 0), len1);
+                    far[h] = min(max(row_pos[h] - j0, 0), len1);
+                }
+                if (__any_sync(0xffffffffu, near[0] < right_from[0] || near[1] < right_from[1])) {
+#pragma unroll
+                    for (int h = 0; h < 2; ++h) {
+                        const int from = p.distance_runs[far[h]];
+                        right_from[h] = from <= near[h] ? from : 0x7fffffff;      // one number for all 16 keys, or one each
+#pragma unroll
+                        for (int i = 0; i < 2; ++i) number[h][i] = number_at(p, row_dist[h], row_pos[h] - (j0 + g + 8 * i));
+                    }
+                }
+            }
+            ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(&tail->full[s]), ph, abort_flag, err_word, 2, wait_limit));
+            if (!ok) break;
+            const unsigned kbase = smem_u32(smem + (size_t)s * STAGE), vbase = one_plane ? kbase : kbase + NKB * BOX_BYTES;
+            // a warp whose 16 keys no row may see skips them (the first and the last tile of a window)
+            if (j0 + 15 >= lo_first && j0 <= p_last) {
+                float sc[4] = {0.f, 0.f, 0.f, 0.f}, sc2[4] = {0.f, 0.f, 0.f, 0.f};      // two chains of products
+#pragma unroll
+                for (int kk = 0; kk < NK; kk += 2) {
+                    unsigned ka[4];
+                    const int row = 16 * warp + (lane & 7) + 8 * ((lane >> 3) & 1);
+                    ldmatrix_x4(ka, tile_addr(kbase, row, 2 * kk + (lane >> 4)));
+                    mma16816(sc, ka[0], ka[1], ka[2], ka[3], qb[kk][0], qb[kk][1]);
+                    ldmatrix_x4(ka, tile_addr(kbase, row, 2 * kk + 2 + (lane >> 4)));
+                    mma16816(sc2, ka[0], ka[1], ka[2], ka[3], qb[kk + 1][0], qb[kk + 1][1]);
+                }
+                float key[2] = {1.f, 1.f};                       // the keys' factors
+                if (scaled) { key[0] = key_scales[s * BN + 16 * warp + g]; key[1] = key_scales[s * BN + 16 * warp + g + 8]; }
+                float pv[2][2], corr[2];
+#pragma unroll
+                for (int h = 0; h < 2; ++h) {
+                    float mx = -INFINITY;
+#pragma unroll
+                    for (int i = 0; i < 2; ++i) {
+                        const int j = j0 + g + 8 * i;
+                        const bool vis = row_ok[h] && j >= row_lo[h] && j <= row_pos[h];
+                        const float v = vis ? score_of<FORM>(p, (sc[2 * i + h] + sc2[2 * i + h]) * p.softmax_scale, key[i], inv_cap, row_slope[h],
+                                                             FORM == FORM_ANY ? number[h][i] : 0.f, row_pos[h] - j) : -INFINITY;
+                        pv[h][i] = v;
+                        mx = fmaxf(mx, v);
+                    }
+                    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 4));
+                    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
+                    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 16));
+                    const float m_new = fmaxf(m_run[h], mx);
+                    corr[h] = (m_new == -INFINITY) ? 1.f : expf(m_run[h] - m_new);
+                    float sum = 0.f;
+#pragma unroll
+                    for (int i = 0; i < 2; ++i) {
+                        pv[h][i] = (m_new == -INFINITY) ? 0.f : expf(pv[h][i] - m_new);
+                        sum += pv[h][i];
+                    }
+                    l_run[h] = l_run[h] * corr[h] + sum;
+                    m_run[h] = m_new;
+                }
+                if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
+#pragma unroll
+                    for (int n = 0; n < NK; ++n) {
+                        o[n][0] *= corr[0]; o[n][2] *= corr[0];
+                        o[n][1] *= corr[1]; o[n][3] *= corr[1];
+                    }
+                }
+                // values: O^T += V^T P^T
+                const unsigned pb0 = transpose_8x8(pack_bf16(pv[0][0], pv[1][0])), pb1 = transpose_8x8(pack_bf16(pv[0][1], pv[1][1]));
+#pragma unroll
+                for (int jj = 0; jj < NK; ++jj) {
+                    unsigned va[4];
+                    ldmatrix_x4_trans(va, tile_addr(vbase, 16 * warp + (lane & 7) + 8 * (lane >> 4), 2 * jj + ((lane >> 3) & 1)));
+                    mma16816(o[jj], va[0], va[1], va[2], va[3], pb0, pb1);
+                }
+            }
+            __syncwarp();
+            if (lane == 0) mbar_arrive(smem_u32(&tail->empty[s]));
+        }
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 4);
+            l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 8);
+            l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 16);
         }
     } else {
         // ---- consumers: warp w takes keys 16 w .. 16 w + 15 of every tile
@@ -205,9 +344,43 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
 #pragma unroll
             for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
 
+        const float inv_cap = inverse_cap(p);
+        const bool upper = n_rows > 8;                       // rows 8 .. 15 hold a (token, head) at all
+        // What the distances to this lane's keys add, asked for ahead of the wait.  A row's distances fall from tile to tile, and
+        // far from the query one number serves many tiles: it is kept, with the smallest distance it is right for.
+        float number[2][2][2] = {{{0.f, 0.f}, {0.f, 0.f}}, {{0.f, 0.f}, {0.f, 0.f}}};
+        int right_from[2] = {0x7fffffff, 0x7fffffff};
         int s = 0;
         unsigned ph = 0;
         for (int ti = sb; ti < se; ++ti, s = (s + 1 == n_stages ? 0 : s + 1), ph ^= (s == 0)) {
+            if (FORM == FORM_ANY && p.distance_bias) {
+                const int len1 = p.distance_len - 1, j0 = ti * BN + 16 * warp;
+                int near[2], far[2];                         // the distances of this warp's last and first key of the tile
+#pragma unroll
+                for (int h = 0; h < 2; ++h) {
+                    near[h] = min(max(row_pos[h] - j0 - 15, 0), len1);
+                    far[h] = min(max(row_pos[h] - j0, 0), len1);
+                }
+                if (__any_sync(0xffffffffu, near[0] < right_from[0] || (upper && near[1] < right_from[1]))) {
+                    const int from0 = p.distance_runs[far[0]], from1 = upper ? p.distance_runs[far[1]] : 0;
+                    const bool one = __all_sync(0xffffffffu, from0 <= near[0] && (!upper || from1 <= near[1]));
+                    right_from[0] = one ? from0 : 0x7fffffff;
+                    right_from[1] = one ? from1 : 0x7fffffff;
+#pragma unroll
+                    for (int h = 0; h < 2; ++h) {
+                        if (h == 1 && !upper) continue;
+                        if (one) {
+                            number[h][0][0] = number[h][0][1] = number[h][1][0] = number[h][1][1] = row_dist[h][near[h]];
+                            continue;
+                        }
+#pragma unroll
+                        for (int n = 0; n < 2; ++n)
+#pragma unroll
+                            for (int e = 0; e < 2; ++e)
+                                number[h][n][e] = number_at(p, row_dist[h], row_pos[h] - (j0 + 8 * n + 2 * cc + e));
+                    }
+                }
+            }
             ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(&tail->full[s]), ph, abort_flag, err_word, 2, wait_limit));
             if (!ok) break;
             const unsigned kbase = smem_u32(smem + (size_t)s * STAGE), vbase = one_plane ? kbase : kbase + NKB * BOX_BYTES;
@@ -238,9 +411,13 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
                     }
                 }
                 // mask, running maximum and sum (float32)
-                float corr[2];
+                float corr[2] = {1.f, 1.f};
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {
+                    if (FORM != FORM_PLAIN && h == 1 && !upper) {          // (their weights stay zero)
+                        sc[0][2] = sc[0][3] = sc[1][2] = sc[1][3] = 0.f;
+                        continue;
+                    }
                     float mx = -INFINITY;
 #pragma unroll
                     for (int n = 0; n < 2; ++n)
@@ -248,7 +425,7 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
                         for (int e = 0; e < 2; ++e) {
                             const int j = j0 + 8 * n + 2 * cc + e;
                             const bool vis = row_ok[h] && j >= row_lo[h] && j <= row_pos[h];
-                            const float v = vis ? score_of<FORM>(p, sc[n][2 * h + e] * p.softmax_scale, key[n][e], row_slope[h], row_dist[h], row_pos[h] - j) : -INFINITY;
+                            const float v = vis ? score_of<FORM>(p, sc[n][2 * h + e] * p.softmax_scale, key[n][e], inv_cap, row_slope[h], FORM == FORM_ANY ? number[h][n][e] : 0.f, row_pos[h] - j) : -INFINITY;
                             sc[n][2 * h + e] = v;
                             mx = fmaxf(mx, v);
                         }
@@ -268,10 +445,12 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
                     l_run[h] = l_run[h] * corr[h] + sum;
                     m_run[h] = m_new;
                 }
+                if (FORM == FORM_PLAIN || __any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
 #pragma unroll
-                for (int n = 0; n < 2 * NK; ++n) {
-                    o[n][0] *= corr[0]; o[n][1] *= corr[0];
-                    o[n][2] *= corr[1]; o[n][3] *= corr[1];
+                    for (int n = 0; n < 2 * NK; ++n) {
+                        o[n][0] *= corr[0]; o[n][1] *= corr[0];
+                        o[n][2] *= corr[1]; o[n][3] *= corr[1];
+                    }
                 }
                 // values: O += P V
                 const unsigned pa0 = pack_bf16(sc[0][0], sc[0][1]), pa1 = pack_bf16(sc[0][2], sc[0][3]);
@@ -303,13 +482,26 @@ __global__ void __launch_bounds__(THREADS) attn_decode_kernel(const __grid_const
     float* o_s = (float*)smem;                               // [CONSUMERS][16][HD]
     float* m_s = o_s + CONSUMERS * 16 * HD;                  // [CONSUMERS][16]
     float* l_s = m_s + CONSUMERS * 16;
+    if constexpr (NARROW) {
 #pragma unroll
-    for (int n = 0; n < 2 * NK; ++n) {
-        float* dst = o_s + ((size_t)warp * 16 + g) * HD + 8 * n + 2 * cc;
-        dst[0] = o[n][0]; dst[1] = o[n][1];
-        dst[8 * HD] = o[n][2]; dst[8 * HD + 1] = o[n][3];
+        for (int n = 0; n < NK; ++n) {
+            float* dst = o_s + ((size_t)warp * 16 + 2 * cc) * HD + 16 * n + g;
+            dst[0] = o[n][0]; dst[HD] = o[n][1];
+            dst[8] = o[n][2]; dst[HD + 8] = o[n][3];
+        }
+        if (g == 0) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h) { m_s[warp * 16 + 2 * cc + h] = m_run[h]; l_s[warp * 16 + 2 * cc + h] = l_run[h]; }
+        }
+    } else {
+#pragma unroll
+        for (int n = 0; n < 2 * NK; ++n) {
+            float* dst = o_s + ((size_t)warp * 16 + g) * HD + 8 * n + 2 * cc;
+            dst[0] = o[n][0]; dst[1] = o[n][1];
+            dst[8 * HD] = o[n][2]; dst[8 * HD + 1] = o[n][3];
+        }
     }
-    if (cc == 0) {
+    if (!NARROW && cc == 0) {
         m_s[warp * 16 + g] = m_run[0]; m_s[warp * 16 + g + 8] = m_run[1];
         l_s[warp * 16 + g] = l_run[0]; l_s[warp * 16 + g + 8] = l_run[1];
     }
@@ -445,7 +637,10 @@ int launch(const AttentionParams& p, const StepTokens& b, const PagedCache& c, c
     const size_t smem = ring + sizeof(Tail) + 1024;
     if (smem > 227 * 1024) return SPITE_UNSUPPORTED;
     const int form = score_form_of(p, c);
-    auto k = form == FORM_ANY ? attn_decode_kernel<NKB, FORM_ANY> : form == FORM_CAP ? attn_decode_kernel<NKB, FORM_CAP> : attn_decode_kernel<NKB, FORM_PLAIN>;
+    const bool narrow = x.tokens_per_block * (p.num_heads / c.num_kv_heads) <= 8;
+#define SPITE_DECODE_FORM(F) (narrow ? attn_decode_kernel<NKB, F, true> : attn_decode_kernel<NKB, F, false>)
+    auto k = form == FORM_ANY ? SPITE_DECODE_FORM(FORM_ANY) : form == FORM_CAP ? SPITE_DECODE_FORM(FORM_CAP) : SPITE_DECODE_FORM(FORM_PLAIN);
+#undef SPITE_DECODE_FORM
     if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
         cudaFuncSetAttribute(k, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared) != cudaSuccess)
         return SPITE_LAUNCH_FAILED;

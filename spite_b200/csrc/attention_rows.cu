@@ -143,6 +143,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_rows_kernel(const AttentionPa
         }
     };
 
+    const float inv_cap = inverse_cap(p);
     float o[2 * NK][4];
 #pragma unroll
     for (int n = 0; n < 2 * NK; ++n)
@@ -205,7 +206,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_rows_kernel(const AttentionPa
                     for (int e = 0; e < 2; ++e) {
                         const int j = j0 + 8 * n + 2 * cc + e;
                         const bool ok = row_ok[h] && j >= row_lo[h] && j <= row_pos[h];
-                        const float v = ok ? score_of<FORM>(p, s[n][2 * h + e] * p.softmax_scale, key[n][e], row_slope[h], row_dist[h], row_pos[h] - j) : -INFINITY;
+                        const float v = ok ? score_of<FORM>(p, s[n][2 * h + e] * p.softmax_scale, key[n][e], inv_cap, row_slope[h], FORM == FORM_ANY ? number_at(p, row_dist[h], row_pos[h] - j) : 0.f, row_pos[h] - j) : -INFINITY;
                         s[n][2 * h + e] = v;
                         mx = fmaxf(mx, v);
                     }

@@ -75,6 +75,23 @@ __device__ __forceinline__ float ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
     return y;
 }
+typedef unsigned long long f2;                            // two packed floats
+__device__ __forceinline__ f2 pack2(float lo, float hi) {
+    f2 v;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(lo), "f"(hi));
+    return v;
+}
+__device__ __forceinline__ void unpack2(f2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
+    f2 v;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(v) : "l"(a), "l"(b), "l"(c));
+    return v;
+}
+__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
+    f2 v;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(v) : "l"(a), "l"(b));
+    return v;
+}
 __device__ __forceinline__ unsigned pack_bf16(float a, float b) {
     __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
     return *(unsigned*)&v;
@@ -310,6 +327,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 // a cap on the scaled scores, in units of the raw ones; the argument of 2^x that gives e^(2 s scale / cap)
                 const float cap_raw = p.score_softcap > 0.f ? p.score_softcap / p.softmax_scale : 0.f;
                 const float cap_arg = p.score_softcap > 0.f ? 2.f * LOG2E * p.softmax_scale / p.score_softcap : 0.f;
+                const float inv_cap_raw = p.score_softcap > 0.f ? p.softmax_scale / p.score_softcap : 0.f;
                 // a number per distance, brought into the units of the raw scores as it is added
                 const float* dist_row = FORM == FORM_ANY ? distance_row_of(p, head) : nullptr;
                 const float per_scale = 1.f / p.softmax_scale;
@@ -352,16 +370,31 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                     if (scaled) {
 #pragma unroll
                         for (int e = 0; e < BN; e += 4) {
-                            const float4 f = *(const float4*)(scale_s + e);
-                            s[e] *= f.x; s[e + 1] *= f.y; s[e + 2] *= f.z; s[e + 3] *= f.w;
+                            const ulonglong2 f = *(const ulonglong2*)(scale_s + e);
+                            unpack2(mul2(pack2(s[e], s[e + 1]), f.x), s[e], s[e + 1]);
+                            unpack2(mul2(pack2(s[e + 2], s[e + 3]), f.y), s[e + 2], s[e + 3]);
                         }
                     }
                     if (FORM == FORM_CAP || (FORM == FORM_ANY && cap_raw > 0.f)) {
-                        // cap tanh(s scale / cap) in units of the raw scores: tanh(x) = 1 - 2 / (e^(2x) + 1), whose absolute
-                        // error (a few float32 roundings of a number below one) times the cap is far below a bfloat16 weight's
+                        // cap tanh(s scale / cap) in units of the raw scores: where every score of the warp's rows is small against
+                        // the cap the series (multiply-adds, two scores an instruction), else 1 - 2 / (e^(2x) + 1), whose two
+                        // special-function operations a score would bind the kernel; the errors are far below a bfloat16 weight's
+                        float big[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-                        for (int e = 0; e < BN; ++e)
-                            s[e] = fmaf(-2.f * cap_raw, __frcp_rn(ex2(s[e] * cap_arg) + 1.f), cap_raw);
+                        for (int e = 0; e < BN; ++e) big[e & 3] = fmaxf(big[e & 3], fabsf(s[e]));
+                        if (__all_sync(0xffffffffu, fmaxf(fmaxf(big[0], big[1]), fmaxf(big[2], big[3])) <= CAP_SERIES * cap_raw)) {
+                            const f2 inv = pack2(inv_cap_raw, inv_cap_raw), one = pack2(1.f, 1.f), c1 = pack2(CAP_C1, CAP_C1),
+                                     c2 = pack2(CAP_C2, CAP_C2), c3 = pack2(CAP_C3, CAP_C3), c4 = pack2(CAP_C4, CAP_C4), c5 = pack2(CAP_C5, CAP_C5);
+#pragma unroll
+                            for (int e = 0; e < BN; e += 2) {
+                                const f2 v = pack2(s[e], s[e + 1]), t = mul2(v, inv), y = mul2(t, t);
+                                unpack2(mul2(v, fma2(y, fma2(y, fma2(y, fma2(y, fma2(y, c5, c4), c3), c2), c1), one)), s[e], s[e + 1]);
+                            }
+                        } else {
+#pragma unroll
+                            for (int e = 0; e < BN; ++e)
+                                s[e] = fmaf(-2.f * cap_raw, reciprocal_approx(ex2(s[e] * cap_arg) + 1.f), cap_raw);
+                        }
                     }
                     if (biased) {
 #pragma unroll

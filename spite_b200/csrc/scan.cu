@@ -373,8 +373,9 @@ __global__ void __launch_bounds__(128) memory_gates_kernel(float* __restrict__ w
 }
 
 // gated linear attention: w[t, c] = sigmoid(z)^(1/tau) with z = sum_r a[t, r] A_2[r, c] + b[c] for the channels c of all heads.
-// A thread has one channel of DECAY_TOKENS tokens; the sum runs over r in ascending order.
-constexpr int DECAY_TOKENS = 8, DECAY_RANK = 64;          // (the short vectors of a block's tokens pass through in pieces)
+// A thread has one channel of DECAY_TOKENS tokens (8 in prompts, 1 in steps of few tokens); the sum runs over r in ascending order.
+constexpr int DECAY_RANK = 64;                            // (the short vectors of a block's tokens pass through in pieces)
+template <int DECAY_TOKENS>
 __global__ void __launch_bounds__(128) channel_decays_kernel(const float* __restrict__ a, long long a_stride, const float* __restrict__ a2,
                                                              const float* __restrict__ b, float* __restrict__ w, long long w_stride,
                                                              int n_tokens, int n, int rank, float inv_tau) {
@@ -394,7 +395,7 @@ __global__ void __launch_bounds__(128) channel_decays_kernel(const float* __rest
         }
         __syncthreads();
         if (c < n) {
-#pragma unroll 4
+#pragma unroll 16
             for (int r = 0; r < nr; ++r) {
                 const float v = a2[(size_t)(r0 + r) * n + c];
 #pragma unroll
@@ -498,9 +499,11 @@ SPITE_API int spite_gated_linear_scan(const ScanParams* p, const float* a, long 
     if (p->n_segments == 0 || p->n_tokens == 0) return SPITE_OK;
     cudaStream_t st = (cudaStream_t)stream;
     const int n = p->heads * p->dim;
-    dim3 grid((n + 127) / 128, (p->n_tokens + DECAY_TOKENS - 1) / DECAY_TOKENS);
+    const bool few = p->n_tokens <= 64;
+    dim3 grid((n + 127) / 128, few ? p->n_tokens : (p->n_tokens + 7) / 8);
     if (grid.y > 65535) return SPITE_UNSUPPORTED;
-    SPITE_LAUNCH(channel_decays_kernel, grid, 128, 0, st, a, a_stride, a2, b, (float*)p->w, p->w_stride, p->n_tokens, n, rank, 1.f / tau);
+    auto decays = few ? channel_decays_kernel<1> : channel_decays_kernel<8>;
+    SPITE_LAUNCH(decays, grid, 128, 0, st, a, a_stride, a2, b, (float*)p->w, p->w_stride, p->n_tokens, n, rank, 1.f / tau);
     if (cudaGetLastError() != cudaSuccess) return SPITE_LAUNCH_FAILED;
     return choose_scan<PER_CHANNEL>(*p, st);
 }

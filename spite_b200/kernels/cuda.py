@@ -255,6 +255,7 @@ class CudaKernels(KernelSet):
         # most key splits of decode attention: beyond about twenty the merge by the last block costs more than the
         # extra blocks bring (one request at 8,192 keys: 22 us with 37 splits, 17.6 us with 18)
         self.attention_max_splits = 24
+        self.attention_narrow_rows = 8         # decoded tokens of up to so many heads a kv head take its form of eight rows (0: never)
         self.use_decode_attention = True       # the TMA-fed decode kernel (head sizes 64 and 128, pages of a multiple of 64 keys)
         # row counts up to which the weight-streaming kernel is preferred over the tcgen05 one
         self.skinny_max_rows = 16
@@ -1032,6 +1033,8 @@ class CudaKernels(KernelSet):
             if batch.context_bucket:            # fixed launch shape for a captured step
                 longest = batch.context_bucket if window.kind == "full" else min(batch.context_bucket, window.size)
             if c.head_dim in (64, 128) and c.page_size % 64 == 0 and self.use_decode_attention:
+                if group <= self.attention_narrow_rows and all(seg.n_tokens == 1 for seg in batch.segments if seg.n_tokens < big_from):
+                    tpb = 1                     # one token a block: up to eight rows, the kernel's narrow form
                 self._attention_decode(p, b, c, batch, n_small, tpb, big_from - 1, longest, num_heads, cache_settled)
                 return
             tiles = -(-longest // 16) + 1
@@ -1069,10 +1072,12 @@ class CudaKernels(KernelSet):
     def _attention_decode(self, p, b, c, batch, n_small, tpb, seg_max, longest, num_heads, cache_settled):
         """Decoded tokens (and portions too short for the row kernels) on the TMA-fed decode kernel: as many
         key splits as fill the resident blocks once, partial results merged by the last block of a split set."""
-        stage = 2 * c.head_dim * 64 * 2                         # 64 keys and 64 values of one kv head
+        # 64 keys and 64 values of one kv head; keys that are the values, with a factor each, are one tile
+        stage = (1 if c.key_scale else 2) * c.head_dim * 64 * 2
         tiles = -(-longest // 64) + 1
         base = n_small * c.num_kv_heads
-        per_sm = max(1, min(4, (225 * 1024) // (3 * stage + 2048)))
+        narrow = tpb * (num_heads // c.num_kv_heads) <= 8
+        per_sm = max(1, min(4 if not c.key_scale else 3 if narrow else 2, (225 * 1024) // (3 * stage + 2048)))
         slots = per_sm * self.sm_count
         if base <= slots:
             splits = slots // base
@@ -1081,7 +1086,8 @@ class CudaKernels(KernelSet):
         else:
             splits = max(range(1, 5), key=lambda s: (base * s / slots) / -(-base * s // slots))
         splits = max(1, min(splits, tiles // 2, self.attention_max_splits))
-        n_stages = max(2, min(3 if per_sm > 1 else 6, -(-tiles // splits)))
+        deep = 6 if per_sm == 1 or (c.key_scale and per_sm == 2) else 4 if c.key_scale else 3
+        n_stages = max(2, min(deep, -(-tiles // splits)))
         partial = tickets = None
         if splits > 1:
             if base > self._tickets_n:
