@@ -15,9 +15,9 @@
 //   weight of the token at place i (for a product that scales its rows in the sorted order).
 //   No host round trip: the grouped products read these arrays on the device.
 //
-// Two kernels.  The first computes the logits (8 tokens x 2 experts at a time, the block's 8
-// warps splitting the width), one pair of experts a block, so that a few tokens still spread over
-// several multiprocessors.  The second, one block per choice slot, selects and sorts.
+// The first kernel computes the logits (8 tokens x 2 experts at a time, the block's 8 warps splitting the width), one pair of
+// experts a block, so that a few tokens still spread over several multiprocessors.  A second one, a warp a token, chooses
+// the experts, a third, one block per choice slot, sorts; in steps of few tokens the third chooses, too.
 // A logit is summed in an order fixed by the width alone.
 #include "common.cuh"
 
@@ -27,6 +27,7 @@ constexpr int MAX_EXPERTS = 1024;
 constexpr int TB = 8;                  // tokens per block of the logits kernel
 constexpr int EB = 2;                  // experts per block
 constexpr int WARPS = 8;
+constexpr int SELECT_IN_SORT = 64;     // steps of up to so many tokens choose and sort in one kernel
 constexpr int SCORE_SIGMOID = 0, SCORE_SOFTMAX_RENORM = 1, SCORE_SOFTMAX_BIASED = 2;
 
 __device__ __forceinline__ void load4(const float* p, float (&v)[4]) {
@@ -117,15 +118,89 @@ __global__ void __launch_bounds__(WARPS * 32) route_logits_kernel(const T* __res
     }
 }
 
-// grid top_k, block 1024: block `slot` picks every token's slot-th expert and sorts the tokens by it.
-__global__ void __launch_bounds__(1024) select_and_sort_kernel(const float* __restrict__ logits, int n_tokens,
-                                                               int n_experts, int top_k,
-                                                               int* __restrict__ expert_ids, float* __restrict__ weights,
-                                                               int* __restrict__ offsets,
-                                                               int* __restrict__ sorted_rows, int scoring,
-                                                               float* __restrict__ sorted_weights,
-                                                               const float* __restrict__ choice_bias) {
+// One token's choices, made by a warp: `take(slot, expert, weight)` is called by lane 0 for slot 0, 1, ... below `slots` in the
+// order (value descending, expert id ascending).  A lane looks at experts lane, lane + 32, ...; every sum is made in an order
+// that the number of experts fixes, so a token's weights do not depend on what else is in the step.
+struct Choice { float v; int e; };
+__device__ __forceinline__ Choice better(Choice a, Choice b) {          // (an id of -1: none)
+    if (b.e < 0) return a;
+    return a.e < 0 || b.v > a.v || (b.v == a.v && b.e < a.e) ? b : a;
+}
+template <typename F>
+__device__ __forceinline__ void choose_experts(const float* __restrict__ l, int n_experts, int top_k, int slots, int scoring,
+                                               const float* __restrict__ choice_bias, int lane, F take) {
+    const bool biased = scoring == SCORE_SOFTMAX_BIASED, renorm = scoring == SCORE_SOFTMAX_RENORM;
+    float mx = -INFINITY, z = 1.f, inv_z = 1.f;
+    if (biased || renorm) {
+        for (int e = lane; e < n_experts; e += 32) mx = fmaxf(mx, l[e]);
+        mx = warp_max(mx);
+        z = 0.f;
+        for (int e = lane; e < n_experts; e += 32) z += expf(l[e] - mx);
+        z = warp_sum(z);
+        inv_z = 1.0f / z;                                    // (one rounding for every share of the token, choice and weight alike)
+    }
+    float chosen_sum = 0.f;                                  // of exp(logit - largest logit) over the chosen experts
+    Choice prev = {INFINITY, -1};
+    float keep_v = 0.f;                                      // renorm: lane s keeps the logit and the id of choice s until the sum is known
+    int keep_e = 0;
+    const int rounds = renorm ? top_k : slots;
+    for (int s = 0; s < rounds; ++s) {
+        Choice best = {-INFINITY, -1};
+        for (int e = lane; e < n_experts; e += 32) {
+            const float v = biased ? expf(l[e] - mx) * inv_z + choice_bias[e] : l[e];
+            if (v < prev.v || (v == prev.v && e > prev.e)) best = better(best, Choice{v, e});
+        }
+#pragma unroll
+        for (int h = 16; h >= 1; h >>= 1) {
+            Choice other;
+            other.v = __shfl_xor_sync(0xffffffffu, best.v, h);
+            other.e = __shfl_xor_sync(0xffffffffu, best.e, h);
+            best = better(best, other);
+        }
+        if (best.e < 0) { best.e = 0; best.v = biased ? 0.f : l[0]; }     // values that do not compare (NaN): still a valid id
+        prev = best;
+        if (renorm) {
+            chosen_sum += expf(best.v - mx);
+            if (lane == s) { keep_v = best.v; keep_e = best.e; }          // (at most 32 choices: the caller's limit)
+            continue;
+        }
+        if (lane == 0) take(s, best.e, biased ? expf(l[best.e] - mx) * inv_z : 1.0f / (1.0f + expf(-best.v)));
+    }
+    if (renorm) {
+        // share_e = exp(l_e - max) / Z with Z over all experts; w = share / (sum of chosen shares + 1e-20)
+        const float w = (expf(keep_v - mx) / z) / (chosen_sum / z + 1e-20f);
+        for (int s = 0; s < slots; ++s) {
+            const int e = __shfl_sync(0xffffffffu, keep_e, s);
+            const float ws = __shfl_sync(0xffffffffu, w, s);
+            if (lane == 0) take(s, e, ws);
+        }
+    }
+}
+
+// grid ceil(tokens / 8), block 256: a warp chooses one token's experts for every slot.
+__global__ void __launch_bounds__(256) select_kernel(const float* __restrict__ logits, int n_tokens, int n_experts, int top_k,
+                                                     int* __restrict__ expert_ids, float* __restrict__ weights, int scoring,
+                                                     const float* __restrict__ choice_bias) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t = blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (t >= n_tokens) return;
+    choose_experts(logits + (size_t)t * n_experts, n_experts, top_k, top_k, scoring, choice_bias, threadIdx.x & 31, [&](int s, int e, float w) {
+        expert_ids[(size_t)s * n_tokens + t] = e;
+        weights[(size_t)s * n_tokens + t] = w;
+    });
+}
+
+// grid top_k, block 1024: block `slot` sorts the tokens by their slot-th expert.  SELECT (steps of few tokens): it first chooses
+// that expert for every token itself, which spares a kernel.
+constexpr int SORT_TOKENS = 4096;                            // ids kept in shared memory, if they fit
+template <bool SELECT>
+__global__ void __launch_bounds__(1024) sort_kernel(const float* __restrict__ logits, int n_tokens, int n_experts, int top_k,
+                                                    int* __restrict__ expert_ids, float* __restrict__ weights,
+                                                    int* __restrict__ offsets, int* __restrict__ sorted_rows, int scoring,
+                                                    float* __restrict__ sorted_weights, const float* __restrict__ choice_bias) {
     __shared__ int counts[MAX_EXPERTS + 1];
+    __shared__ int ids_s[SORT_TOKENS];
     pdl_wait();
     pdl_launch_dependents();
     const int slot = blockIdx.x;
@@ -133,81 +208,48 @@ __global__ void __launch_bounds__(1024) select_and_sort_kernel(const float* __re
     for (int e = threadIdx.x; e <= n_experts; e += blockDim.x) counts[e] = 0;
     __syncthreads();
     int* ids = expert_ids + (size_t)slot * n_tokens;
-    for (int t = threadIdx.x; t < n_tokens; t += blockDim.x) {
-        // the slot-th element in the order (logit descending, expert id ascending)
-        const float* l = logits + (size_t)t * n_experts;
-        if (scoring == SCORE_SOFTMAX_BIASED) {
-            // share_e = exp(l_e - max) / Z; the slot-th expert in the order (share + bias descending, expert id ascending)
-            float mx = -INFINITY, z = 0.f;
-            for (int e = 0; e < n_experts; ++e) mx = fmaxf(mx, l[e]);
-            for (int e = 0; e < n_experts; ++e) z += expf(l[e] - mx);
-            const float inv_z = 1.0f / z;                    // (one rounding for every share of the token, choice and weight alike)
-            float pv = INFINITY, bv = 0.f;
-            int pe = -1, be = 0;
-            for (int s = 0; s <= slot; ++s) {
-                bv = -INFINITY;
-                be = -1;
-                for (int e = 0; e < n_experts; ++e) {
-                    const float v = expf(l[e] - mx) * inv_z + choice_bias[e];
-                    const bool after_prev = v < pv || (v == pv && e > pe);
-                    if (after_prev && (be < 0 || v > bv)) { bv = v; be = e; }
-                }
-                if (be < 0) { be = 0; bv = 0.f; }
-                pv = bv;
-                pe = be;
-            }
-            ids[t] = be;
-            weights[(size_t)slot * n_tokens + t] = expf(l[be] - mx) * inv_z;
-            atomicAdd(&counts[be + 1], 1);
-            continue;
+    const bool in_shared = n_tokens <= SORT_TOKENS;
+    if (SELECT) {
+        for (int t = warp; t < n_tokens; t += nwarps)
+            choose_experts(logits + (size_t)t * n_experts, n_experts, top_k, slot + 1, scoring, choice_bias, lane, [&](int s, int e, float w) {
+                if (s != slot) return;
+                ids[t] = e;
+                if (in_shared) ids_s[t] = e;
+                weights[(size_t)slot * n_tokens + t] = w;
+                atomicAdd(&counts[e + 1], 1);
+            });
+    } else {
+        for (int t = threadIdx.x; t < n_tokens; t += blockDim.x) {
+            const int e = ids[t];
+            if (in_shared) ids_s[t] = e;
+            atomicAdd(&counts[e + 1], 1);
         }
-        float prev_v = INFINITY;
-        int prev_e = -1;
-        float best_v = 0.f, mine_v = 0.f;
-        int best_e = 0, mine_e = 0;
-        float chosen_max = 0.f, chosen_sum = 0.f;            // of exp(logit - largest logit) over the chosen experts
-        const int picks = scoring == SCORE_SOFTMAX_RENORM ? top_k : slot + 1;
-        for (int s = 0; s < picks; ++s) {
-            best_v = -INFINITY;
-            best_e = -1;
-            for (int e = 0; e < n_experts; ++e) {
-                const float v = l[e];
-                const bool after_prev = v < prev_v || (v == prev_v && e > prev_e);
-                if (after_prev && (best_e < 0 || v > best_v)) { best_v = v; best_e = e; }
-            }
-            if (best_e < 0) { best_e = 0; best_v = l[0]; }    // logits that do not compare (NaN): still a valid id
-            prev_v = best_v;
-            prev_e = best_e;
-            if (s == 0) chosen_max = best_v;                 // the largest logit of all
-            chosen_sum += expf(best_v - chosen_max);
-            if (s == slot) { mine_v = best_v; mine_e = best_e; }
-        }
-        ids[t] = mine_e;
-        float w;
-        if (scoring == SCORE_SOFTMAX_RENORM) {
-            // share_e = exp(l_e - max) / Z with Z over all experts; w = share / (sum of chosen shares + 1e-20)
-            float z = 0.f;
-            for (int e = 0; e < n_experts; ++e) z += expf(l[e] - chosen_max);
-            w = (expf(mine_v - chosen_max) / z) / (chosen_sum / z + 1e-20f);
-        } else {
-            w = 1.0f / (1.0f + expf(-mine_v));
-        }
-        weights[(size_t)slot * n_tokens + t] = w;
-        atomicAdd(&counts[mine_e + 1], 1);
     }
     __syncthreads();
-    if (threadIdx.x == 0)
-        for (int e = 0; e < n_experts; ++e) counts[e + 1] += counts[e];
+    if (warp == 0) {                                         // running sums, 32 experts at a time
+        int before = 0;
+        for (int e0 = 1; e0 <= n_experts; e0 += 32) {
+            int v = e0 + lane <= n_experts ? counts[e0 + lane] : 0;
+#pragma unroll
+            for (int h = 1; h < 32; h <<= 1) {
+                const int up = __shfl_up_sync(0xffffffffu, v, h);
+                if (lane >= h) v += up;
+            }
+            if (e0 + lane <= n_experts) counts[e0 + lane] = before + v;
+            before += __shfl_sync(0xffffffffu, v, 31);
+        }
+    }
     __syncthreads();
     int* off = offsets + (size_t)slot * (n_experts + 1);
     for (int e = threadIdx.x; e <= n_experts; e += blockDim.x) off[e] = counts[e];
     int* rows = sorted_rows + (size_t)slot * n_tokens;
+    const int* from = in_shared ? ids_s : ids;
     for (int e = warp; e < n_experts; e += nwarps) {
         int base = counts[e];
-        if (counts[e + 1] == base) continue;
-        for (int t0 = 0; t0 < n_tokens; t0 += 32) {
+        const int end = counts[e + 1];
+        for (int t0 = 0; t0 < n_tokens && base < end; t0 += 32) {
             const int t = t0 + lane;
-            const bool mine = t < n_tokens && ids[t] == e;
+            const bool mine = t < n_tokens && from[t] == e;
             const unsigned mask = __ballot_sync(0xffffffffu, mine);
             if (mine) {
                 const int at = base + __popc(mask & ((1u << lane) - 1u));
@@ -230,7 +272,7 @@ SPITE_API int spite_moe_route(int dtype, const void* x, const float* w_router, i
     if (scoring != SCORE_SIGMOID && scoring != SCORE_SOFTMAX_RENORM && scoring != SCORE_SOFTMAX_BIASED) return SPITE_BAD_ARG;
     if (scoring == SCORE_SOFTMAX_BIASED && !choice_bias) return SPITE_BAD_ARG;
     if (n_tokens < 0 || d <= 0 || n_experts < 1 || top_k < 1 || top_k > n_experts) return SPITE_BAD_ARG;
-    if (n_experts > MAX_EXPERTS) return SPITE_UNSUPPORTED;
+    if (n_experts > MAX_EXPERTS || (scoring == SCORE_SOFTMAX_RENORM && top_k > 32)) return SPITE_UNSUPPORTED;
     cudaStream_t st = (cudaStream_t)stream;
     if (n_tokens > 0) {
         // one pair of experts a block: measured faster than blocks that take several pairs and reuse
@@ -248,8 +290,16 @@ SPITE_API int spite_moe_route(int dtype, const void* x, const float* w_router, i
             return SPITE_BAD_ARG;
         if (cudaGetLastError() != cudaSuccess) return SPITE_LAUNCH_FAILED;
     }
-    SPITE_LAUNCH(select_and_sort_kernel, top_k, 1024, 0, st, (const float*)logits, n_tokens, n_experts, top_k,
-                 expert_ids, weights, offsets, sorted_rows, scoring, sorted_weights, choice_bias);
+    if (n_tokens <= SELECT_IN_SORT) {
+        SPITE_LAUNCH(sort_kernel<true>, top_k, 1024, 0, st, (const float*)logits, n_tokens, n_experts, top_k, expert_ids, weights, offsets,
+                     sorted_rows, scoring, sorted_weights, choice_bias);
+        return spite_launch_status();
+    }
+    SPITE_LAUNCH(select_kernel, (n_tokens + 7) / 8, 256, 0, st, (const float*)logits, n_tokens, n_experts, top_k, expert_ids, weights, scoring,
+                 choice_bias);
+    if (cudaGetLastError() != cudaSuccess) return SPITE_LAUNCH_FAILED;
+    SPITE_LAUNCH(sort_kernel<false>, top_k, 1024, 0, st, (const float*)logits, n_tokens, n_experts, top_k, expert_ids, weights, offsets,
+                 sorted_rows, scoring, sorted_weights, choice_bias);
     return spite_launch_status();
 }
 

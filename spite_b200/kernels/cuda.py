@@ -1316,7 +1316,7 @@ class CudaKernels(KernelSet):
             C.c_void_p(ids.data_ptr()), C.c_void_p(wts.data_ptr()), C.c_void_p(_ptr(logits)),
             C.c_void_p(offsets.data_ptr()), C.c_void_p(rows.data_ptr()), int(renorm), C.c_void_p(_ptr(sorted_w)),
             C.c_void_p(_ptr(choice_bias)), C.c_void_p(_ptr(logit_bias)), self._stream())
-        self._count("moe", 2)
+        self._count("moe", 2 if M <= 64 else 3)
         _check(st, "moe_route")
         return Routing(ids, wts, offsets, rows, logits if want_logits else None, sorted_w)
 

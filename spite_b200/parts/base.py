@@ -209,6 +209,12 @@ class FeedForward(Part):
     #: float32 [hidden]: a bias on the output that an arrangement may add itself (fused with what it does to the output):
     #: `forward(..., accumulate=False, add_bias=False)` then leaves it out
     output_bias = None
+    #: `begin(x, batch)` does what needs the input alone (a router, the first products) and returns a list of tensors;
+    #: `forward(..., begun=that list)` does the rest.  An arrangement may run it on another stream beside a mixer.
+    can_begin = False
+
+    def begin(self, x, batch) -> list:
+        raise NotImplementedError
 
     def forward(self, x, h, batch):
         raise NotImplementedError

@@ -24,7 +24,7 @@ from __future__ import annotations
 import torch
 
 from ..config.specs import ConfigError
-from .base import Block, register_block
+from .base import Block, register_block, side_stream
 
 
 @register_block("prenorm_residual")
@@ -48,12 +48,32 @@ class ParallelResidual(Block):
     places = {"norm": "norm", "mixer": "mixer", "ffn": "feed_forward"}
     optional = ("ffn",)
 
+    #: in steps of up to so many tokens what the feed-forward does before it adds to the stream runs beside the mixer
+    beside_max_tokens = 64
+
     def forward(self, h, batch, cache):
         x = torch.empty(h.shape, dtype=self.ctx.dtype, device=h.device)
         self.norm.forward(h, x)
+        begun = None
+        side = side_stream(x) if self.ffn is not None and self.ffn.can_begin and x.shape[0] <= self.beside_max_tokens else None
+        if side is not None:
+            main = torch.cuda.current_stream(x.device)
+            forked, done = torch.cuda.Event(), torch.cuda.Event()
+            forked.record(main)
+            with torch.cuda.stream(side):
+                side.wait_event(forked)
+                begun = self.ffn.begin(x, batch)
+                done.record(side)
         self.mixer.forward(x, h, batch, cache)
-        if self.ffn is not None:
+        if self.ffn is None:
+            return
+        if side is None:
             self.ffn.forward(x, h, batch)
+            return
+        main.wait_event(done)
+        for t in begun:
+            t.record_stream(main)                                # made on the side stream, read on this one
+        self.ffn.forward(x, h, batch, begun=begun)
 
 
 @register_block("sandwich_residual")

@@ -44,9 +44,15 @@ class DenseSwiGLU(FeedForward):
     def weight_bytes(self):
         return (self.w_gate_up.numel() + self.w_down.numel()) * self.w_down.element_size()
 
-    def forward(self, x, h, batch):
+    can_begin = True
+
+    def begin(self, x, batch):
         a = torch.empty((x.shape[0], self.f), dtype=x.dtype, device=x.device)
         self.k.linear_swiglu(x, self.w_gate_up, a, activation=self.activation)
+        return [a]
+
+    def forward(self, x, h, batch, begun=None):
+        a, = begun or self.begin(x, batch)
         self.k.linear(a, self.w_down, h, accumulate=True)
 
 
@@ -294,9 +300,10 @@ class MoESoftmaxTopK(FeedForward):
         per = 3 * self.f * self.d * self.w_down.element_size()
         return int(per * n_distinct_experts) + self.router.numel() * 4
 
-    def forward(self, x, h, batch, accumulate=True):
+    can_begin = True
+
+    def _route(self, x):
         k = self.k
-        M = x.shape[0]
         more = {} if self.router_bias is None else dict(logit_bias=self.router_bias)
         if self.renormalize:
             routing = k.moe_route(x, self.router, self.top_k, want_logits=self.keep_router_logits, scoring="softmax_renorm", **more)
@@ -304,6 +311,24 @@ class MoESoftmaxTopK(FeedForward):
             routing = k.moe_route(x, self.router, self.top_k, want_logits=self.keep_router_logits, scoring="softmax_biased",
                                   choice_bias=self.choice_bias, **more)
         self.last_routing = routing
+        return routing
+
+    def _first_product(self, x, routing, slot):
+        a = torch.empty((x.shape[0], self.f), dtype=x.dtype, device=x.device)
+        # (the experts' ranges of the sorted order come first; the places behind them belong to identity experts)
+        self.k.grouped_linear_swiglu(x, self.w_gate_up, routing.sorted_rows[slot], routing.offsets[slot][:self.E + 1], None, a)
+        return a
+
+    def begin(self, x, batch):
+        """The router and every choice slot's first product."""
+        routing = self._route(x)
+        firsts = [self._first_product(x, routing, slot) for slot in range(self.top_k)] if self.E else []
+        return firsts + [t for t in (routing.expert_ids, routing.weights, routing.offsets, routing.sorted_rows, routing.logits,
+                                     routing.sorted_weights) if t is not None]
+
+    def forward(self, x, h, batch, accumulate=True, begun=None):
+        k = self.k
+        routing = self._route(x) if begun is None else self.last_routing
         if self.identity:
             # the tokens that drew an identity expert get their input back, times the weight; without `accumulate` this
             # also starts every row of the sum that the experts then add to
@@ -313,9 +338,6 @@ class MoESoftmaxTopK(FeedForward):
         if not self.E:
             return
         for slot in range(self.top_k):
-            a = torch.empty((M, self.f), dtype=x.dtype, device=x.device)
-            # (the experts' ranges of the sorted order come first; the places behind them belong to identity experts)
-            offsets = routing.offsets[slot][:self.E + 1]
-            k.grouped_linear_swiglu(x, self.w_gate_up, routing.sorted_rows[slot], offsets, None, a)
-            k.grouped_linear_accumulate(a, self.w_down, routing.sorted_rows[slot], offsets, h,
+            a = self._first_product(x, routing, slot) if begun is None else begun[slot]
+            k.grouped_linear_accumulate(a, self.w_down, routing.sorted_rows[slot], routing.offsets[slot][:self.E + 1], h,
                                         row_scale=routing.sorted_weights[slot])
