@@ -254,10 +254,14 @@ __global__ void __launch_bounds__(1024) sort_kernel(const float* __restrict__ lo
             if (mine) {
                 const int at = base + __popc(mask & ((1u << lane) - 1u));
                 rows[at] = t;
-                if (sorted_weights) sorted_weights[(size_t)slot * n_tokens + at] = weights[(size_t)slot * n_tokens + t];
             }
             base += __popc(mask);
         }
+    }
+    if (sorted_weights) {                                    // (a pass of its own: in the loop above every round would wait for its loads)
+        __syncthreads();
+        for (int i = threadIdx.x; i < n_tokens; i += blockDim.x)
+            sorted_weights[(size_t)slot * n_tokens + i] = weights[(size_t)slot * n_tokens + rows[i]];
     }
 }
 
