@@ -545,12 +545,12 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const TX* __restric
     }
 }
 
-// The same for a float32 x whose heads are whole groups of four elements and at most 512: 16-byte loads, gates and gain asked for
+// The same for a float32 x and a bfloat16 out whose heads are whole groups of four elements and at most 512: 16-byte loads, gates and gain asked for
 // ahead of the sum, the head's elements held in registers.  Q: groups a lane.
-template <typename TO, int Q>
+template <int Q>
 __global__ void __launch_bounds__(128) head_norm_gate_vec_kernel(const float* __restrict__ x, const float* __restrict__ gates,
                                                                  long long gate_stride, const float* __restrict__ gain,
-                                                                 TO* __restrict__ out, long long out_stride, int n_tokens, int heads,
+                                                                 __nv_bfloat16* __restrict__ out, long long out_stride, int n_tokens, int heads,
                                                                  int size, float eps, int gate_silu, int gain_per_head) {
     pdl_wait();
     pdl_launch_dependents();
@@ -562,7 +562,7 @@ __global__ void __launch_bounds__(128) head_norm_gate_vec_kernel(const float* __
     const float* in = x + (size_t)row * size;
     const float* g = gates ? gates + (size_t)m * gate_stride + (size_t)h * size : nullptr;
     const float* w = gain ? gain + (gain_per_head ? (size_t)h * size : 0) : nullptr;
-    TO* o = out + (size_t)m * out_stride + (size_t)h * size;
+    __nv_bfloat16* o = out + (size_t)m * out_stride + (size_t)h * size;
     float4 v[Q], z[Q], b[Q];
     float s = 0.f;
 #pragma unroll
@@ -594,21 +594,17 @@ __global__ void __launch_bounds__(128) head_norm_gate_vec_kernel(const float* __
         if (j >= size) continue;
         const float y0 = gate(v[q].x * mul * b[q].x, z[q].x), y1 = gate(v[q].y * mul * b[q].y, z[q].y);
         const float y2 = gate(v[q].z * mul * b[q].z, z[q].z), y3 = gate(v[q].w * mul * b[q].w, z[q].w);
-        if constexpr (sizeof(TO) == 4) *(float4*)(o + j) = make_float4(y0, y1, y2, y3);
-        else {
-            const __nv_bfloat162 lo = __floats2bfloat162_rn(y0, y1), hi = __floats2bfloat162_rn(y2, y3);
-            *(uint2*)(o + j) = make_uint2(*(const unsigned*)&lo, *(const unsigned*)&hi);
-        }
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(y0, y1), hi = __floats2bfloat162_rn(y2, y3);
+        *(uint2*)(o + j) = make_uint2(*(const unsigned*)&lo, *(const unsigned*)&hi);
     }
 }
 
-template <typename TO>
-static bool head_norm_gate_vec(const void* x, const void* gates, long long gate_stride, const float* gain, void* out, long long out_stride,
+static bool head_norm_gate_vec(const void* x, const void* gates, long long gate_stride, const float* gain, __nv_bfloat16* out, long long out_stride,
                                int n_tokens, int heads, int size, float eps, int gate_silu, int gain_per_head, int blocks, cudaStream_t st) {
     const uintptr_t at = (uintptr_t)x | (uintptr_t)gates | (uintptr_t)gain | (uintptr_t)out;
-    if (size % 4 || size > 512 || (at & 15) || gate_stride % 4 || out_stride % 4 || x == out) return false;
-#define SPITE_HEADS(Q) SPITE_LAUNCH((head_norm_gate_vec_kernel<TO, Q>), blocks, 128, 0, st, (const float*)x, (const float*)gates, gate_stride, \
-                                    gain, (TO*)out, out_stride, n_tokens, heads, size, eps, gate_silu, gain_per_head)
+    if (size % 4 || size > 512 || (at & 15) || gate_stride % 4 || out_stride % 4) return false;
+#define SPITE_HEADS(Q) SPITE_LAUNCH((head_norm_gate_vec_kernel<Q>), blocks, 128, 0, st, (const float*)x, (const float*)gates, gate_stride, \
+                                    gain, out, out_stride, n_tokens, heads, size, eps, gate_silu, gain_per_head)
     if (size <= 128) SPITE_HEADS(1);
     else if (size <= 256) SPITE_HEADS(2);
     else SPITE_HEADS(4);
@@ -631,12 +627,10 @@ SPITE_API int spite_head_norm_gate(int x_dtype, int out_dtype, const void* x, co
     const long long blocks = (rows + 3) / 4;
     if (blocks > 0x7fffffffLL) return SPITE_UNSUPPORTED;
     cudaStream_t st = (cudaStream_t)stream;
-    if (x_dtype == SPITE_DT_F32) {
-        const bool done = out_dtype == SPITE_DT_F32
-            ? head_norm_gate_vec<float>(x, gates, gate_stride, gain, out, out_stride, n_tokens, heads, size, eps, gate_silu, gain_per_head, (int)blocks, st)
-            : head_norm_gate_vec<__nv_bfloat16>(x, gates, gate_stride, gain, out, out_stride, n_tokens, heads, size, eps, gate_silu, gain_per_head, (int)blocks, st);
-        if (done) return spite_launch_status();
-    }
+    if (x_dtype == SPITE_DT_F32 && out_dtype == SPITE_DT_BF16 &&
+        head_norm_gate_vec(x, gates, gate_stride, gain, (__nv_bfloat16*)out, out_stride, n_tokens, heads, size, eps, gate_silu, gain_per_head,
+                           (int)blocks, st))
+        return spite_launch_status();
     if (x_dtype == SPITE_DT_F32 && out_dtype == SPITE_DT_F32)
         SPITE_LAUNCH((head_norm_gate_kernel<float, float>), (int)blocks, 128, 0, st, (const float*)x, (const float*)gates,
                      gate_stride, gain, (float*)out, out_stride, n_tokens, heads, size, eps, gate_silu, gain_per_head);

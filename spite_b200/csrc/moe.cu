@@ -200,7 +200,9 @@ __global__ void __launch_bounds__(1024) sort_kernel(const float* __restrict__ lo
                                                     int* __restrict__ offsets, int* __restrict__ sorted_rows, int scoring,
                                                     float* __restrict__ sorted_weights, const float* __restrict__ choice_bias) {
     __shared__ int counts[MAX_EXPERTS + 1];
-    __shared__ int ids_s[SORT_TOKENS];
+    // (few bytes in steps of few tokens: the kernel then runs beside products that leave a multiprocessor little shared memory)
+    constexpr int KEPT = SELECT ? SELECT_IN_SORT : SORT_TOKENS;
+    __shared__ int ids_s[KEPT];
     pdl_wait();
     pdl_launch_dependents();
     const int slot = blockIdx.x;
@@ -208,7 +210,7 @@ __global__ void __launch_bounds__(1024) sort_kernel(const float* __restrict__ lo
     for (int e = threadIdx.x; e <= n_experts; e += blockDim.x) counts[e] = 0;
     __syncthreads();
     int* ids = expert_ids + (size_t)slot * n_tokens;
-    const bool in_shared = n_tokens <= SORT_TOKENS;
+    const bool in_shared = n_tokens <= KEPT;
     if (SELECT) {
         for (int t = warp; t < n_tokens; t += nwarps)
             choose_experts(logits + (size_t)t * n_experts, n_experts, top_k, slot + 1, scoring, choice_bias, lane, [&](int s, int e, float w) {
